@@ -15,7 +15,7 @@ before the window, except the pages of the first ``keep_first`` positions when t
 keep those.  A run that reads another run's cache (``cache_of``) gets a view of that
 run's plane and writes nothing; what the owner's group keeps is then the union of what the owner
 and its readers see (the widest window, the most kept first positions).  Runs that ask for fixed-size state get one tensor
-``[slots, ...]`` each, zeroed when a slot is opened (the reference keeps recurrent state of
+``[slots, ...]`` each (or several by name), zeroed when a slot is opened (the reference keeps recurrent state of
 this kind in its run state, include/model_run_state.h:21-23, zeroed on reset,
 src/session.c:145-167).  The reference's own key/value arrays are per session and
 [layers, seq_len, kv_dim] (src/transformer/kv.c:123-131).
@@ -196,11 +196,20 @@ class Cache:
                 raise CacheError(f"schedule entry {i} cannot read entry {src}'s cache: "
                                  f"{a.n_kv_heads}x{a.head_dim}/{a.v_dim} against {b.n_kv_heads}x{b.head_dim}/{b.v_dim}")
             self._reader[i] = src
-        self.states: Dict[int, torch.Tensor] = {}
-        self.state_requests = {i: r for i, r in enumerate(state_requests) if r is not None}
+        # schedule entry -> its state; an entry that keeps several by name has one for each (entry, name)
+        self.states: Dict[object, torch.Tensor] = {}
+        self._named: Dict[int, Dict[str, torch.Tensor]] = {}
+        self.state_requests: Dict[object, StateRequest] = {}
+        for i, r in enumerate(state_requests):
+            if isinstance(r, dict):
+                self.state_requests.update({(i, name): one for name, one in r.items()})
+            elif r is not None:
+                self.state_requests[i] = r
         if allocate:
             for i, r in self.state_requests.items():
                 self.states[i] = torch.zeros((n_slots,) + tuple(r.shape), dtype=r.dtype, device=device)
+                if isinstance(i, tuple):
+                    self._named.setdefault(i[0], {})[i[1]] = self.states[i]
 
     # ---- slots ----------------------------------------------------------------------------
     def open(self) -> int:
@@ -275,8 +284,10 @@ class Cache:
                       head_dim=g.request.head_dim, window=g.request.window, owner=owner,
                       v_head_dim=g.request.v_head_dim)
 
-    def state(self, entry: int) -> Optional[torch.Tensor]:
-        return self.states.get(entry)
+    def state(self, entry: int):
+        """The entry's state tensor, or a dict of them by name if it keeps several, or None."""
+        named = self._named.get(entry)
+        return named if named is not None else self.states.get(entry)
 
     # ---- accounting -----------------------------------------------------------------------
     def tokens_free(self) -> int:

@@ -3,6 +3,7 @@ from .spec import (BiasAttentionSpec, MlstmSpec, MoeSpec, PostNormBlockSpec)  # 
 from .spec import (DeltaRuleSpec, LatentAttentionSpec, ParallelBlockSpec, RotaryPairsSpec, TokenSideSpec)  # noqa: F401
 from .spec import (LimitedMlpSpec, SigmoidAttentionSpec)  # noqa: F401
 from .spec import (NormedAttentionSpec, RotaryBlendSpec, SandwichBlockSpec)  # noqa: F401
+from .spec import (HeadDeltaSpec, LayerNormSpec, Mamba2Spec, PolyMlpSpec, StreamsBlockSpec)  # noqa: F401
 from .spec import (AttentionSpec, BlockSpec, ConfigError, GatedMlpSpec, LinearHeadSpec, ModelSpec, NoPositionSpec,
                    RmsNormSpec, RotarySpec, ScheduleEntry)
 from .registry import (Architecture, architecture, architecture_of, known_architectures,
@@ -70,7 +71,20 @@ register_architecture(Architecture(
     config_to_dict=NetanexConfig.to_dict,
 ))
 
+from . import rudolix as _rudolix
+from .rudolix import RudolixConfig
+
+register_architecture(Architecture(
+    name=_rudolix.ARCHITECTURE,
+    read_config=RudolixConfig.from_dict,
+    to_spec=RudolixConfig.to_spec,
+    tensor_name=_rudolix.tensor_name,
+    cap_positions=RudolixConfig.with_max_positions,
+    config_to_dict=RudolixConfig.to_dict,
+))
+
 __all__ = [
+    "RudolixConfig", "HeadDeltaSpec", "LayerNormSpec", "Mamba2Spec", "PolyMlpSpec", "StreamsBlockSpec",
     "NetanexConfig", "NormedAttentionSpec", "RotaryBlendSpec", "SandwichBlockSpec",
     "AttentionSpec", "BlockSpec", "ConfigError", "GatedMlpSpec", "LinearHeadSpec", "ModelSpec", "NoPositionSpec",
     "RmsNormSpec", "RotarySpec", "ScheduleEntry", "Architecture", "architecture", "architecture_of",

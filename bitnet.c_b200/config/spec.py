@@ -31,6 +31,15 @@ class RmsNormSpec:
 
 
 @dataclass(frozen=True)
+class LayerNormSpec:
+    """(x - mean) / sqrt(mean((x - mean)^2) + eps) over the last axis, with a learned gain and bias."""
+
+    width: int
+    eps: float
+    kind: str = "layernorm"
+
+
+@dataclass(frozen=True)
 class RotarySpec:
     """Rotary position encoding in the rotate-half pairing (i, i + rotary_dims/2)."""
 
@@ -133,6 +142,7 @@ class BiasAttentionSpec:
     chunk: int = 0  # c > 0 (in place of a window): a token sees the earlier keys of its own chunk of c positions
     position: Any = None  # a position spec whose encoding q and k get (after the unit norm, if any); None: none
     values_are_keys: bool = False  # no value projection: the values are the keys as projected, before any encoding
+    sink: bool = False  # a learned score per head in the softmax's denominator, without a key or a value
     kind: str = "bias_attention"
 
 
@@ -243,6 +253,40 @@ class DeltaRuleSpec:
 
 
 @dataclass(frozen=True)
+class HeadDeltaSpec:
+    """Gated delta rule with one decay per head: short causal convolutions and SiLU on q, k, v; unit q and k; beta and
+    the decays from the mixer's input, one number per head each; a per-head unit norm with a shared gain and a SiLU
+    gate of full width on the output."""
+
+    width: int
+    n_heads: int
+    n_kv_heads: int
+    head_dim: int
+    v_head_dim: int
+    conv_taps: int
+    norm_eps: float
+    kind: str = "head_delta"
+
+
+@dataclass(frozen=True)
+class Mamba2Spec:
+    """Mamba-2 state-space layer: one input projection [z | x | B | C | dt]; a causal convolution with a bias and SiLU
+    on x, B and C; a state of ``state`` x ``v_head_dim`` numbers per head under one decay per head and token, B and C
+    shared by the heads of a group; a skip per head; the output gated by silu(z) and then RMS-normed, the row cut into
+    ``norm_groups`` parts that are normed apart, with a gain."""
+
+    width: int
+    n_heads: int
+    n_groups: int
+    state: int
+    v_head_dim: int
+    conv_taps: int
+    norm_groups: int
+    norm_eps: float
+    kind: str = "mamba2"
+
+
+@dataclass(frozen=True)
 class MlstmSpec:
     """mLSTM: a matrix memory per head with exponential gating, a soft cap on the gates' pre-activations,
     a unit norm per head, a gain over all heads and a logistic output gate."""
@@ -277,6 +321,7 @@ class MoeSpec:
     weight_scale: float = 1.0  # factor on the (renormalised) weights
     renormalise_eps: float = 0.0  # added to the sum the weights are divided by
     activation: str = "limited"  # "limited": the clamped unit above; "silu" / "gelu_tanh": act(g) * u, no clamps
+    router_bias: bool = False  # a learned number per expert added to the router's logits before the choice
     kind: str = "moe"
 
 
@@ -301,6 +346,17 @@ class LimitedMlpSpec:
     limit: float
     slope: float = 1.702
     kind: str = "limited_mlp"
+
+
+@dataclass(frozen=True)
+class PolyMlpSpec:
+    """Dense feed-forward without a gate: down(act(up x)), act(z) = c1 z/r1 + c2 z^2/r2 + c3 z^3/r3 + c0 where rk is the
+    root mean square of z^k over the token's ``intermediate`` numbers (eps inside) and the four factors are learned."""
+
+    width: int
+    intermediate: int
+    eps: float
+    kind: str = "poly_mlp"
 
 
 @dataclass(frozen=True)
@@ -374,6 +430,25 @@ class ParallelBlockSpec:
 
 
 @dataclass(frozen=True)
+class StreamsBlockSpec:
+    """A block on a residual of ``streams`` streams.  With X the streams as rows of a matrix, sublayer q
+    reads h = norm_q(in_q^T X), plus (``input_taps`` > 0) a per-channel causal convolution of h along the sequence, and
+    with y its result, times one number per channel (``layer_scale``), X becomes
+    mix_q^T X + ``residual_mult`` out_q y^T.  ``ffn`` may be None."""
+
+    mixer: Any
+    ffn: Any
+    mixer_norm: Any
+    ffn_norm: Any
+    width: int
+    streams: int
+    residual_mult: float = 1.0
+    input_taps: int = 0
+    layer_scale: bool = True
+    kind: str = "streams"
+
+
+@dataclass(frozen=True)
 class LinearHeadSpec:
     """The output head: logits = scale * (W h), then optionally ``softcap * tanh(logits / softcap)``
     (the reference's final soft-cap, src/transformer/logits.c:325-333; 0 means none).  W is the
@@ -411,12 +486,16 @@ class ModelSpec:
     embedding_norm: Any = None  # a norm spec: the embedding rows are normed before the first block reads them
     stop_ids: Tuple[int, ...] = field(default_factory=tuple)
     head: Any = field(default_factory=LinearHeadSpec)  # a head spec; its part turns normed rows into logits
+    streams: int = 1  # the residual holds so many streams of ``width`` side by side, which start alike (the embedding row)
 
     def validate(self) -> None:
         if self.vocab_size <= 0 or self.width <= 0 or self.max_positions <= 0:
             raise ConfigError("vocab_size, width and max_positions must be positive")
         if not self.blocks or not self.schedule:
             raise ConfigError("a model needs at least one block and one schedule entry")
+        for i, b in enumerate(self.blocks):
+            if getattr(b, "streams", 1) != self.streams:
+                raise ConfigError(f"block {i} works on {getattr(b, 'streams', 1)} streams, the model has {self.streams}")
         for i, e in enumerate(self.schedule):
             if not 0 <= e.block < len(self.blocks):
                 raise ConfigError(f"schedule entry {i} names block {e.block}, "

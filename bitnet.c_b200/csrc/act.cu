@@ -260,3 +260,100 @@ extern "C" int bn_gate_rows(void* x, int x_stride, const void* g, int g_stride, 
     return BN_ERR_BAD_ARG;
   return BN_OK;
 }
+
+// A polynomial of normed powers over the rows of z: with r_k = sqrt(mean over the row of z^(2k) + eps),
+//   out = coef[0] z / r_1 + coef[1] z^2 / r_2 + coef[2] z^3 / r_3 + coef[3]
+// for the first `len` numbers of a row; up to `row_len` zeros follow (a padded width).  One block per row; the row
+// waits in shared memory between its two passes; sums in float32.
+template <typename T, typename Z, int V>
+__global__ void poly_norm_kernel(const Z* __restrict__ z, const float* __restrict__ coef, float eps, T* __restrict__ out, int len,
+                                 int row_len) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float row[];  // row_len
+  __shared__ float scratch[32];
+  const Z* zr = z + (size_t)blockIdx.x * row_len;
+  float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+  for (int i = threadIdx.x * V; i < len; i += blockDim.x * V) {
+    float v[V];
+    if (V == 4) {
+      if (sizeof(Z) == 4) {
+        const float4 a = *reinterpret_cast<const float4*>(zr + i);
+        v[0] = a.x; v[1 % V] = a.y; v[2 % V] = a.z; v[3 % V] = a.w;
+      } else {
+        const uint2 raw = *reinterpret_cast<const uint2*>(zr + i);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        v[0] = a.x; v[1 % V] = a.y; v[2 % V] = b.x; v[3 % V] = b.y;
+      }
+      *reinterpret_cast<float4*>(row + i) = make_float4(v[0], v[1 % V], v[2 % V], v[3 % V]);
+    } else {
+      row[i] = v[0] = to_f32<Z>(zr[i]);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const float q = v[e] * v[e];
+      s1 += q;
+      s2 = fmaf(q, q, s2);
+      s3 = fmaf(q * q, q, s3);
+    }
+  }
+  s1 = block_sum(s1, scratch);
+  s2 = block_sum(s2, scratch);
+  s3 = block_sum(s3, scratch);
+  const float n = (float)len;
+  const float a = coef[0] / sqrtf(s1 / n + eps), b = coef[1] / sqrtf(s2 / n + eps), c = coef[2] / sqrtf(s3 / n + eps), e0 = coef[3];
+  T* dst = out + (size_t)blockIdx.x * row_len;
+  for (int i = threadIdx.x * V; i < row_len; i += blockDim.x * V) {
+    float v[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const float x = i + e < len ? row[i + e] : 0.f;
+      v[e] = i + e < len ? fmaf(x, fmaf(x, fmaf(x, c, b), a), e0) : 0.f;
+    }
+    if (V == 4 && sizeof(T) == 4) {
+      *reinterpret_cast<float4*>(dst + i) = make_float4(v[0], v[1 % V], v[2 % V], v[3 % V]);
+    } else if (V == 4) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1 % V]), hi = __floats2bfloat162_rn(v[2 % V], v[3 % V]);
+      uint2 raw;
+      raw.x = *reinterpret_cast<const unsigned*>(&lo);
+      raw.y = *reinterpret_cast<const unsigned*>(&hi);
+      *reinterpret_cast<uint2*>(dst + i) = raw;
+    } else {
+      dst[i] = from_f32<T>(v[0]);
+    }
+  }
+}
+
+template <typename T, typename Z, int V>
+static int launch_poly_norm(const void* z, const float* coef, float eps, void* out, int n_rows, int len, int row_len, cudaStream_t stream) {
+  const size_t smem = ((size_t)row_len + 3) / 4 * 4 * sizeof(float);
+  if (smem > 200 * 1024) return BN_ERR_BAD_ARG;
+  if (smem > 48 * 1024) {
+    static size_t granted = 0;
+    if (smem > granted) {
+      cudaError_t e = cudaFuncSetAttribute(poly_norm_kernel<T, Z, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) return BN_ERR_LAUNCH + (int)e;
+      granted = smem;
+    }
+  }
+  const int threads = row_len >= 8192 ? 1024 : (row_len >= 2048 ? 512 : (row_len >= 512 ? 256 : 128));
+  BN_LAUNCH((poly_norm_kernel<T, Z, V>), n_rows, threads, smem, stream, (const Z*)z, coef, eps, (T*)out, len, row_len);
+  return BN_OK;
+}
+
+// z and out [n_rows, row_len]; coef: four float32 numbers on the device
+extern "C" int bn_poly_norm(const void* z, int z_dtype, const float* coef, float eps, void* out, int out_dtype, int n_rows, int len,
+                            int row_len, cudaStream_t stream) {
+  if (n_rows <= 0) return BN_OK;
+  if (!z || !coef || !out || len <= 0 || row_len < len || !(eps > 0.f)) return BN_ERR_BAD_ARG;
+  const bool vec = len % 4 == 0 && row_len % 4 == 0 && !(((uintptr_t)z | (uintptr_t)out) & 15);
+#define BN_POLY(TT, ZZ)                                                                                   \
+  return vec ? launch_poly_norm<TT, ZZ, 4>(z, coef, eps, out, n_rows, len, row_len, stream)               \
+             : launch_poly_norm<TT, ZZ, 1>(z, coef, eps, out, n_rows, len, row_len, stream)
+  if (z_dtype == BN_F32 && out_dtype == BN_F32) BN_POLY(float, float);
+  if (z_dtype == BN_F32 && out_dtype == BN_BF16) BN_POLY(__nv_bfloat16, float);
+  if (z_dtype == BN_BF16 && out_dtype == BN_BF16) BN_POLY(__nv_bfloat16, __nv_bfloat16);
+#undef BN_POLY
+  return BN_ERR_BAD_ARG;
+}

@@ -49,6 +49,8 @@ SOURCES: Dict[str, str] = {
     "moe": "moe.cu",
     "rotary_pairs": "rotary_pairs.cu",
     "delta_rule": "delta_rule.cu",
+    "streams": "streams.cu",
+    "gated_state": "gated_state.cu",
     "sigmoid_attention": "sigmoid_attention.cu",
     "sigmoid_attention_prefill": "sigmoid_attention_prefill.cu",
 }

@@ -5,33 +5,37 @@
 
 template <typename T>
 __global__ void embed_gather_kernel(const T* __restrict__ table, const int* __restrict__ tokens,
-                                    float* __restrict__ out, int width, int vocab, float scale,
+                                    float* __restrict__ out, int width, int vocab, float scale, int copies,
                                     int* __restrict__ bad_token) {
   pdl_launch_dependents();  // the next kernel in the stream may begin its prologue
   pdl_wait();               // the kernels before this one have completed and their writes are visible
   int t = blockIdx.x;
   int id = tokens[t];
-  float* o = out + (size_t)t * width;
+  float* o = out + (size_t)t * copies * width;
   if (id < 0 || id >= vocab) {
     if (threadIdx.x == 0) atomicExch(bad_token, 1);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = 0.f;
+    for (int i = threadIdx.x; i < copies * width; i += blockDim.x) o[i] = 0.f;
     return;
   }
   const T* row = table + (size_t)id * width;
-  for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = to_f32<T>(row[i]) * scale;
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    const float v = to_f32<T>(row[i]) * scale;
+    for (int s = 0; s < copies; ++s) o[(size_t)s * width + i] = v;
+  }
 }
 
-// bad_token: one int on the device, set to 1 when an id lies outside [0, vocab).
+// bad_token: one int on the device, set to 1 when an id lies outside [0, vocab).  copies: the row is written so many
+// times side by side, out [n_tokens, copies * width] (a residual of several streams that start alike).
 extern "C" int bn_embed_gather(const void* table, int table_dtype, const int* tokens, float* out,
-                               int n_tokens, int width, int vocab, float scale, int* bad_token,
+                               int n_tokens, int width, int vocab, float scale, int copies, int* bad_token,
                                cudaStream_t stream) {
   if (n_tokens <= 0) return BN_OK;
-  if (width <= 0 || vocab <= 0) return BN_ERR_BAD_ARG;
+  if (width <= 0 || vocab <= 0 || copies <= 0) return BN_ERR_BAD_ARG;
   int threads = width >= 1024 ? 256 : 128;
   if (table_dtype == BN_F32)
-    BN_LAUNCH((embed_gather_kernel<float>), n_tokens, threads, 0, stream, (const float*)table, tokens, out, width, vocab, scale, bad_token);
+    BN_LAUNCH((embed_gather_kernel<float>), n_tokens, threads, 0, stream, (const float*)table, tokens, out, width, vocab, scale, copies, bad_token);
   else if (table_dtype == BN_BF16)
-    BN_LAUNCH((embed_gather_kernel<__nv_bfloat16>), n_tokens, threads, 0, stream, (const __nv_bfloat16*)table, tokens, out, width, vocab, scale, bad_token);
+    BN_LAUNCH((embed_gather_kernel<__nv_bfloat16>), n_tokens, threads, 0, stream, (const __nv_bfloat16*)table, tokens, out, width, vocab, scale, copies, bad_token);
   else
     return BN_ERR_BAD_ARG;
   BN_CHECK_LAUNCH();

@@ -22,7 +22,8 @@
 #define MOE_MAX_EXPERTS 1024
 
 template <typename T, typename W>
-__global__ void moe_route_kernel(const T* __restrict__ h, int width, const W* __restrict__ w, int n_experts, int top,
+__global__ void moe_route_kernel(const T* __restrict__ h, int width, const W* __restrict__ w, const float* __restrict__ bias,
+                                 int n_experts, int top,
                                  int renormalise, int softmax, float weight_scale, float sum_eps, int* __restrict__ ids,
                                  float* __restrict__ weights) {
   pdl_launch_dependents();
@@ -36,7 +37,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, int width, const W* __
   __syncthreads();
   for (int e = warp; e < n_experts; e += n_warps) {
     float dot = warp_dot(xs, w + (size_t)e * width, width, lane);
-    if (lane == 0) z[e] = dot;
+    if (lane == 0) z[e] = bias ? dot + bias[e] : dot;
   }
   __syncthreads();
   if (warp == 0) {
@@ -79,8 +80,9 @@ __global__ void moe_route_kernel(const T* __restrict__ h, int width, const W* __
 }
 
 // softmax: the scores are the softmax over all experts instead of each logit's logistic function; the chosen
-// experts' scores are divided by their sum + sum_eps with `renormalise`, then multiplied by weight_scale
-extern "C" int bn_moe_route_ex(const void* h, int h_dtype, int n_tokens, int width, const void* w, int w_dtype,
+// experts' scores are divided by their sum + sum_eps with `renormalise`, then multiplied by weight_scale.  bias
+// [n_experts] float32 (or null) is added to the logits before anything is chosen.
+extern "C" int bn_moe_route_ex(const void* h, int h_dtype, int n_tokens, int width, const void* w, int w_dtype, const float* bias,
                                int n_experts, int top, int renormalise, int softmax, float weight_scale, float sum_eps,
                                int* ids, float* weights, cudaStream_t stream) {
   if (n_tokens <= 0) return BN_OK;
@@ -89,14 +91,14 @@ extern "C" int bn_moe_route_ex(const void* h, int h_dtype, int n_tokens, int wid
     return BN_ERR_BAD_ARG;
   const size_t smem = (size_t)width * sizeof(float);
   if (h_dtype == BN_F32 && w_dtype == BN_F32)
-    BN_LAUNCH((moe_route_kernel<float, float>), n_tokens, 256, smem, stream, (const float*)h, width, (const float*)w,
+    BN_LAUNCH((moe_route_kernel<float, float>), n_tokens, 256, smem, stream, (const float*)h, width, (const float*)w, bias,
               n_experts, top, renormalise, softmax, weight_scale, sum_eps, ids, weights);
   else if (h_dtype == BN_BF16 && w_dtype == BN_BF16)
     BN_LAUNCH((moe_route_kernel<__nv_bfloat16, __nv_bfloat16>), n_tokens, 256, smem, stream, (const __nv_bfloat16*)h, width,
-              (const __nv_bfloat16*)w, n_experts, top, renormalise, softmax, weight_scale, sum_eps, ids, weights);
+              (const __nv_bfloat16*)w, bias, n_experts, top, renormalise, softmax, weight_scale, sum_eps, ids, weights);
   else if (h_dtype == BN_BF16 && w_dtype == BN_F32)
     BN_LAUNCH((moe_route_kernel<__nv_bfloat16, float>), n_tokens, 256, smem, stream, (const __nv_bfloat16*)h, width,
-              (const float*)w, n_experts, top, renormalise, softmax, weight_scale, sum_eps, ids, weights);
+              (const float*)w, bias, n_experts, top, renormalise, softmax, weight_scale, sum_eps, ids, weights);
   else
     return BN_ERR_BAD_ARG;
   BN_CHECK_LAUNCH();
@@ -105,7 +107,7 @@ extern "C" int bn_moe_route_ex(const void* h, int h_dtype, int n_tokens, int wid
 
 extern "C" int bn_moe_route(const void* h, int h_dtype, int n_tokens, int width, const void* w, int w_dtype,
                             int n_experts, int top, int renormalise, int* ids, float* weights, cudaStream_t stream) {
-  return bn_moe_route_ex(h, h_dtype, n_tokens, width, w, w_dtype, n_experts, top, renormalise, 0, 1.0f, 0.0f, ids, weights, stream);
+  return bn_moe_route_ex(h, h_dtype, n_tokens, width, w, w_dtype, nullptr, n_experts, top, renormalise, 0, 1.0f, 0.0f, ids, weights, stream);
 }
 
 #define MOE_THREADS 256

@@ -106,17 +106,18 @@ _F0 = c_float(0.0)
 
 # ---- embedding ----------------------------------------------------------------------------
 def embed_gather(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, bad_token: torch.Tensor,
-                 scale: float = 1.0) -> torch.Tensor:
-    """out[t] = float32(table[tokens[t]]) * scale; sets bad_token[0] = 1 on an id outside the table."""
+                 scale: float = 1.0, copies: int = 1) -> torch.Tensor:
+    """out[t] = float32(table[tokens[t]]) * scale, ``copies`` times side by side; sets bad_token[0] = 1 on an id
+    outside the table."""
     _need(table, "table", dims=2)
     _need(tokens, "tokens", torch.int32, 1)
     _need(out, "out", torch.float32, 2)
     _need(bad_token, "bad_token", torch.int32)
     n, width = tokens.shape[0], table.shape[1]
-    if out.shape[0] < n or out.shape[1] != width:
-        raise KernelError(f"out {tuple(out.shape)} does not hold {n} rows of width {width}")
+    if out.shape[0] < n or out.shape[1] != copies * width:
+        raise KernelError(f"out {tuple(out.shape)} does not hold {n} rows of width {copies} x {width}")
     _check(_fn("embed", "bn_embed_gather")(_ptr(table), _code(table), _ptr(tokens), _ptr(out), int(n),
-                                           int(width), int(table.shape[0]), c_float(scale),
+                                           int(width), int(table.shape[0]), c_float(scale), int(copies),
                                            _ptr(bad_token), _stream()), "embed_gather")
     return out
 
@@ -281,6 +282,21 @@ def glu_halves(h: torch.Tensor, out: torch.Tensor, act: int = 0) -> torch.Tensor
         raise KernelError(f"glu_halves: h {tuple(h.shape)} and out {tuple(out.shape)} do not fit")
     _check(_fn("act", "bn_glu_halves")(_ptr(h), _ptr(out), int(_code(h)), int(h.shape[0]), int(inter), int(act), _stream()),
            "glu_halves")
+    return out
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float, out_dtype: torch.dtype, length: int = 0) -> torch.Tensor:
+    """coef[0] z/r1 + coef[1] z^2/r2 + coef[2] z^3/r3 + coef[3] over the rows of z, rk the root mean square of z^k over the
+    row's first ``length`` numbers (0: all; eps inside the root); zeros behind them.  ``coef``: four float32 numbers."""
+    _need(z, "z", dims=2)
+    _need(coef, "coef", torch.float32, 1)
+    n, row = z.shape
+    length = length or row
+    if coef.shape[0] != 4 or length > row:
+        raise KernelError("poly_norm: four coefficients, and a length within the row")
+    out = torch.empty((n, row), dtype=out_dtype, device=z.device)
+    _check(_fn("act", "bn_poly_norm")(_ptr(z), int(_code(z)), _ptr(coef), c_float(eps), _ptr(out), int(_code(out)), int(n), int(length),
+                                      int(row), _stream()), "poly_norm")
     return out
 
 
@@ -1596,6 +1612,175 @@ def delta_output(o: torch.Tensor, gain: torch.Tensor, gate: torch.Tensor, heads:
     return out
 
 
+# ---- matrix states under one decay per head ------------------------------------------------------
+GATED_STATE_MAX_DIM = 256
+GATED_STATE_MAX_TAPS = 16
+
+
+def gated_state_floats(heads: int, groups: int, dim: int, vdim: int, taps: int) -> int:
+    """Floats of one sequence's state: the heads' matrices, then a ring of the convolutions' last ``taps`` inputs."""
+    n = heads * dim * vdim + (taps * (2 * groups * dim + heads * vdim) if taps > 1 else 0)
+    return (n + 3) // 4 * 4
+
+
+def gated_state(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: torch.Tensor, a_off: int, b_off: int,
+                conv_w: torch.Tensor, conv_b: Optional[torch.Tensor], dt_bias: torch.Tensor, a_log: torch.Tensor,
+                skip: Optional[torch.Tensor], state: torch.Tensor, tok_seq: torch.Tensor, seq_start: torch.Tensor,
+                seq_pos0: torch.Tensor, slots: torch.Tensor, n_seqs: int, heads: int, groups: int, dim: int, vdim: int,
+                one_token: bool) -> torch.Tensor:
+    """A matrix state per head over the new tokens of every sequence, from and into ``state`` ``[slots,
+    gated_state_floats]`` (float32), under one decay per head and token.  ``proj`` ``[T, n]``: rows with the channels of
+    q and k (``groups * dim`` each) and v (``heads * vdim``) at their offsets; each channel passes a causal convolution
+    (``conv_w`` float32 ``[taps, channels]``, channels in the order q, k, v; ``conv_b`` or None) and SiLU.  ``gates``:
+    a float32 matrix (or view with unit inner stride) with the heads' pre-activations.
+    ``b_off`` >= 0, the gated delta rule: q and k made unit vectors per group, q times dim^-1/2; l = -exp(``a_log``)
+    softplus(a + ``dt_bias``), b = sigmoid(.); S <- e^l S; u = b (v - S^T k); S <- S + k u^T; o = S^T q.
+    ``b_off`` < 0, the state-space update: b = softplus(a + ``dt_bias``), l = -exp(``a_log``) b;
+    S <- e^l S + b k v^T; o = S^T q + ``skip`` v.
+    ``one_token``: every sequence brings one token (one launch does it all).  Returns o, float32 ``[T, heads * vdim]``."""
+    _need(proj, "proj", dims=2)
+    _need(conv_w, "conv_w", torch.float32, 2)
+    _need(state, "state", torch.float32, 2)
+    for t, nm, n in ((dt_bias, "dt_bias", heads), (a_log, "a_log", heads), (skip, "skip", heads), (conv_b, "conv_b", conv_w.shape[1])):
+        if t is not None:
+            _need(t, nm, torch.float32, 1)
+            if t.shape[0] != n:
+                raise KernelError(f"gated_state: {nm} holds {t.shape[0]} numbers, {n} are needed")
+    for t, nm in ((tok_seq, "tok_seq"), (seq_start, "seq_start"), (seq_pos0, "seq_pos0"), (slots, "slots")):
+        _need(t, nm, torch.int32, 1)
+    T, taps = tok_seq.shape[0], conv_w.shape[0]
+    n_qk, n_v = groups * dim, heads * vdim
+    if (not gates.is_cuda or gates.dtype != torch.float32 or gates.dim() != 2 or gates.stride(1) != 1 or gates.shape[0] < T
+            or max(a_off, b_off) + heads > gates.shape[1]):
+        raise KernelError("gated_state: gates must be a float32 CUDA matrix with unit inner stride that holds the pre-activations")
+    if (conv_w.shape[1] != 2 * n_qk + n_v or proj.shape[0] < T or state.shape[1] != gated_state_floats(heads, groups, dim, vdim, taps)
+            or seq_start.shape[0] < n_seqs + 1 or seq_pos0.shape[0] < n_seqs or slots.shape[0] < n_seqs or heads % groups
+            or (one_token and T != n_seqs)):
+        raise KernelError("gated_state: sizes do not fit")
+    if dim > GATED_STATE_MAX_DIM or taps > GATED_STATE_MAX_TAPS:
+        raise KernelError(f"gated_state: dim={dim} (at most {GATED_STATE_MAX_DIM}) or {taps} taps (at most {GATED_STATE_MAX_TAPS})")
+    dev = proj.device
+    out = torch.empty((T, n_v), dtype=torch.float32, device=dev)
+    args = (_ptr(proj), int(_code(proj)), int(T), int(proj.shape[1]), int(q_off), int(k_off), int(v_off), c_void_p(gates.data_ptr()),
+            int(gates.stride(0)), int(a_off), int(b_off), int(groups), int(heads), int(dim), int(vdim), int(taps), _ptr(conv_w),
+            _ptr(conv_b), _ptr(dt_bias), _ptr(a_log), _ptr(skip), c_float(dim ** -0.5), _ptr(state),
+            ctypes.c_longlong(state.shape[1]), _ptr(tok_seq), _ptr(seq_start), _ptr(seq_pos0), _ptr(slots), int(n_seqs))
+    if one_token:
+        _check(_fn("gated_state", "bn_gated_state_token")(*args, _ptr(out), _stream()), "gated_state_token")
+        return out
+    qn = torch.empty((T, n_qk), dtype=torch.float32, device=dev)
+    kn = torch.empty((T, n_qk), dtype=torch.float32, device=dev)
+    vc = torch.empty((T, n_v), dtype=torch.float32, device=dev)
+    lb = torch.empty((T, heads, 2), dtype=torch.float32, device=dev)
+    between = (_ptr(qn), _ptr(kn), _ptr(vc), _ptr(lb))
+    _check(_fn("gated_state", "bn_gated_state_prepare")(*args, *between, _stream()), "gated_state_prepare")
+    _check(_fn("gated_state", "bn_gated_state_run")(*args, *between, _ptr(out), _stream()), "gated_state_run")
+    return out
+
+
+def state_output(o: torch.Tensor, z: torch.Tensor, gain: torch.Tensor, parts: int, eps: float, gate_first: bool,
+                 dtype: torch.dtype) -> torch.Tensor:
+    """Rows of o (float32) in ``parts`` equal parts: o silu(z) divided by its root mean square per part, times ``gain``
+    (``gate_first``), or o divided by its root mean square per part, times ``gain``, times silu(z).  ``z``: a view of
+    o's width with unit inner stride; ``gain`` float32, as long as a row or as a part (shared by the parts)."""
+    _need(o, "o", torch.float32, 2)
+    _need(gain, "gain", torch.float32, 1)
+    n, row = o.shape
+    if (not z.is_cuda or z.dim() != 2 or z.stride(1) != 1 or z.shape[1] != row or z.shape[0] < n or row % parts
+            or gain.shape[0] not in (row, row // parts)):
+        raise KernelError("state_output: gate or gain does not fit")
+    out = torch.empty((n, row), dtype=dtype, device=o.device)
+    _check(_fn("gated_state", "bn_state_output")(_ptr(o), c_void_p(z.data_ptr()), int(_code(z)), int(z.stride(0)), _ptr(gain),
+                                                 int(gain.shape[0]), int(_DT[dtype]), int(n), int(parts), int(row // parts),
+                                                 c_float(eps), int(bool(gate_first)), _ptr(out), _stream()), "state_output")
+    return out
+
+
+# ---- a residual of several streams ----------------------------------------------------------------
+MAX_STREAMS = 16
+STREAMS_MAX_TAPS = 16
+STREAMS_MAX_WIDTH = (200 * 1024) // 4
+
+
+def streams_norm(x: torch.Tensor, streams: int, w: torch.Tensor, b: Optional[torch.Tensor], eps: float, out_dtype: torch.dtype, *,
+                 delta: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None, scale: Optional[torch.Tensor] = None,
+                 mult: float = 1.0, read: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+                 taps: Optional[torch.Tensor] = None, hist: Optional[torch.Tensor] = None,
+                 slots: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """On the float32 residual x ``[T, streams * width]``: with ``delta`` ``[T, width]``, a token's
+    streams as the rows of X become M^T X + mult out (scale delta)^T (``mix``: M row by row, then the numbers out; None with
+    one stream: a plain sum); then the layer norm (``w``, ``b``) of read^T X (None: the rows' plain
+    sum) in ``out_dtype``.  With ``rows`` only those rows are normed, and x is left alone.  ``taps`` (float32 ``[n, width]``):
+    the causal convolution of the normed rows is added to them; every row is then the one new token of the slot
+    ``slots`` names, ``hist`` ``[slots, n - 1, width]`` (in ``out_dtype``) holds the inputs before it and is brought up to date."""
+    _need(x, "x", torch.float32, 2)
+    _need(w, "w", dims=1)
+    width = w.shape[0]
+    if not 1 <= streams <= MAX_STREAMS or x.shape[1] != streams * width or width > STREAMS_MAX_WIDTH:
+        raise KernelError(f"streams_norm: x {tuple(x.shape)} is not {streams} streams of width {width}")
+    if b is not None:
+        _need(b, "b", dims=1)
+        if b.shape[0] != width:
+            raise KernelError("streams_norm: the norm's bias does not fit")
+    if delta is not None:
+        _need(delta, "delta", dims=2)
+        if delta.shape[1] != width or delta.shape[0] != x.shape[0] or (mix is None and streams > 1):
+            raise KernelError("streams_norm: the delta does not fit, or several streams have no mixing matrix")
+    for t, nm, n in ((mix, "mix", streams * streams + streams), (scale, "scale", width), (read, "read", streams)):
+        if t is not None:
+            _need(t, nm, torch.float32, 1)
+            if t.shape[0] != n:
+                raise KernelError(f"streams_norm: {nm} holds {t.shape[0]} numbers, {n} are needed")
+    n_rows = x.shape[0]
+    if rows is not None:
+        _need(rows, "rows", torch.int32, 1)
+        n_rows = rows.shape[0]
+    n_taps, hist_stride = 0, 0
+    if taps is not None:
+        _need(taps, "taps", torch.float32, 2)
+        _need(slots, "slots", torch.int32, 1)
+        n_taps = taps.shape[0]
+        if taps.shape[1] != width or n_taps > STREAMS_MAX_TAPS or rows is not None or slots.shape[0] < n_rows:
+            raise KernelError("streams_norm: the convolution's taps do not fit")
+        if n_taps > 1:
+            _need(hist, "hist", out_dtype, 3)
+            if tuple(hist.shape[1:]) != (n_taps - 1, width):
+                raise KernelError(f"streams_norm: the history {tuple(hist.shape)} is not [slots, {n_taps - 1}, {width}]")
+            hist_stride = hist.stride(0)
+    out = torch.empty((n_rows, width), dtype=out_dtype, device=x.device)
+    _check(_fn("streams", "bn_streams_norm")(
+        _ptr(x), int(n_rows), int(width), int(streams), _ptr(delta), int(_code(delta)) if delta is not None else 0, _ptr(mix),
+        _ptr(scale), c_float(mult), _ptr(read), _ptr(w), int(_code(w)), _ptr(b), int(_code(b)) if b is not None else 0, c_float(eps),
+        _ptr(rows), int(rows is None), _ptr(out), int(_code(out)), _ptr(taps), int(n_taps), _ptr(hist if n_taps > 1 else None),
+        ctypes.c_longlong(hist_stride), _ptr(slots if taps is not None else None), _stream()), "streams_norm")
+    return out
+
+
+def input_convolution(h: torch.Tensor, taps: torch.Tensor, hist: Optional[torch.Tensor], tok_seq: torch.Tensor,
+                      seq_start: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
+    """h + its causal convolution along the sequence, channel by channel (``taps`` float32 ``[n, width]``, the last row the current token's)
+    over runs of new tokens; inputs before the step come from ``hist`` ``[slots, n - 1, width]`` (h's type), which then
+    holds each sequence's last n - 1 inputs."""
+    _need(h, "h", dims=2)
+    _need(taps, "taps", torch.float32, 2)
+    for t, nm in ((tok_seq, "tok_seq"), (seq_start, "seq_start"), (slots, "slots")):
+        _need(t, nm, torch.int32, 1)
+    n, width = taps.shape
+    if h.shape[1] != width or h.shape[0] != tok_seq.shape[0] or n > STREAMS_MAX_TAPS:
+        raise KernelError("input_convolution: sizes do not fit")
+    stride = 0
+    if n > 1:
+        _need(hist, "hist", h.dtype, 3)
+        if tuple(hist.shape[1:]) != (n - 1, width):
+            raise KernelError(f"input_convolution: the history {tuple(hist.shape)} is not [slots, {n - 1}, {width}]")
+        stride = hist.stride(0)
+    out = torch.empty_like(h)
+    _check(_fn("streams", "bn_input_convolution")(_ptr(h), _ptr(out), int(_code(h)), int(h.shape[0]), int(width), _ptr(taps), int(n),
+                                                  _ptr(hist if n > 1 else None), ctypes.c_longlong(stride), _ptr(tok_seq),
+                                                  _ptr(seq_start), _ptr(slots), _stream()), "input_convolution")
+    return out
+
+
 # ---- mixture of experts -----------------------------------------------------------------------
 def sigmoid_attention_prefill_fits(n_heads: int, n_kv_heads: int, head_dim: int, v_dim: int) -> bool:
     """Whether the tensor-core kernel for runs of new tokens takes these sizes (bfloat16 only)."""
@@ -1665,8 +1850,8 @@ def sigmoid_attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor,
 
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, top: int, renormalise: bool = False, softmax: bool = False,
-              weight_scale: float = 1.0, sum_eps: float = 0.0):
-    """Per token the ``top`` experts with the largest router logits (float32 products), and their scores as
+              weight_scale: float = 1.0, sum_eps: float = 0.0, bias: Optional[torch.Tensor] = None):
+    """Per token the ``top`` experts with the largest router logits (float32 products, plus ``bias``), and their scores as
     weights: the logistic function of each logit, or with ``softmax`` the softmax over all experts; divided by
     the chosen ones' sum (+ ``sum_eps``) with ``renormalise``, then times ``weight_scale``:
     ``(ids int32 [T, top], weights float32 [T, top])``."""
@@ -1674,10 +1859,14 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, top: int, renormalise: bo
     _need(w_router, "w_router", dims=2)
     if w_router.shape[1] != h.shape[1] or not 0 < top <= min(w_router.shape[0], 32) or w_router.shape[0] > 1024:
         raise KernelError(f"moe_route: router {tuple(w_router.shape)}, top {top} do not fit rows of width {h.shape[1]}")
+    if bias is not None:
+        _need(bias, "bias", torch.float32, 1)
+        if bias.shape[0] != w_router.shape[0]:
+            raise KernelError(f"moe_route: {bias.shape[0]} biases for {w_router.shape[0]} experts")
     ids = torch.empty((h.shape[0], top), dtype=torch.int32, device=h.device)
     weights = torch.empty((h.shape[0], top), dtype=torch.float32, device=h.device)
     _check(_fn("moe", "bn_moe_route_ex")(_ptr(h), int(_code(h)), int(h.shape[0]), int(h.shape[1]), _ptr(w_router),
-                                         int(_code(w_router)), int(w_router.shape[0]), int(top), int(bool(renormalise)),
+                                         int(_code(w_router)), _ptr(bias), int(w_router.shape[0]), int(top), int(bool(renormalise)),
                                          int(bool(softmax)), c_float(weight_scale), c_float(sum_eps), _ptr(ids), _ptr(weights),
                                          _stream()), "moe_route")
     return ids, weights

@@ -18,7 +18,7 @@ from ..config import ConfigError, ModelSpec, architecture_of, read_config_json
 from ..csrc import build as kernel_build
 from ..csrc import ops
 from ..parts import BuildContext, ParamSpec, Part, build_part
-from ..parts.base import Cast, Normed
+from ..parts.base import Cast, Normed, StreamDelta
 from .batch import SeqStep, StepContext, pack_step
 
 _DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16, "float32": torch.float32, "fp32": torch.float32,
@@ -47,6 +47,8 @@ def _walk(prefix: str, part: Part, out: Dict[str, tuple]) -> None:
 class Model:
     def __init__(self, spec: ModelSpec, dtype="bfloat16", device="cuda:0", arch=None, config=None):
         spec.validate()
+        if getattr(spec, "streams", 1) > 1 and getattr(spec, "embedding_norm", None) is not None:
+            raise ConfigError("a normed embedding and a residual of several streams are not built together")
         self.spec, self.arch, self.config = spec, arch, config
         self.dtype = resolve_dtype(dtype)
         self.device = torch.device(device) if device is not None else None
@@ -235,11 +237,12 @@ class Model:
 
     def forward(self, cache: Cache, ctx: StepContext) -> Optional[torch.Tensor]:
         """Embedding, every scheduled run, final norm and head at the wanted rows."""
-        x = torch.empty((ctx.n_tokens, self.spec.width), dtype=torch.float32, device=self.device)
+        streams = getattr(self.spec, "streams", 1)
+        x = torch.empty((ctx.n_tokens, streams * self.spec.width), dtype=torch.float32, device=self.device)
         sched = self.spec.schedule
         pending = None
         if self.embedding_norm is None:
-            ops.embed_gather(self.embedding, ctx.tokens, x, self._bad_token, self.spec.embedding_scale)
+            ops.embed_gather(self.embedding, ctx.tokens, x, self._bad_token, self.spec.embedding_scale, copies=streams)
         elif self.spec.width > ops.EMBED_NORMED_MAX_WIDTH:
             ops.embed_gather(self.embedding, ctx.tokens, x, self._bad_token, self.spec.embedding_scale)
             ops.scaled_add_rmsnorm(x, 1.0, None, self.embedding_norm.weight, self.embedding_norm.spec.eps)
@@ -295,7 +298,9 @@ class Model:
 
 def _residual_after(x: torch.Tensor, pending) -> torch.Tensor:
     """The residual stream with a block's last delta added (the delta is otherwise added by the next
-    norm; a product that prepared that norm in its epilogue has added it already)."""
+    norm; a product that prepared that norm in its epilogue has added it already).  Of several streams: their sum."""
+    if isinstance(pending, StreamDelta):
+        return pending.summed(x)
     if pending is None or isinstance(pending, (Normed, Cast)):
         return x
     return x + (pending.sum(0) if pending.dim() == 3 else pending).float()

@@ -43,7 +43,8 @@ class ParamSpec:
 
     shape: Tuple[int, ...]
     # "normal": N(0, std) matrix; "ones": gain around 1; "around_zero": gain stored as its distance from 1; "zeros";
-    # "distinct": integer rows of different numbers below ``high``
+    # "distinct": integer rows of different numbers below ``high``; "identity": a square matrix near the identity;
+    # "unused": an optional tensor that is read past (random models do not have it)
     init: str = "normal"
     integer: bool = False
     high: int = 0
@@ -89,7 +90,8 @@ class KvRequest:
 @dataclass(frozen=True)
 class StateRequest:
     """Fixed-size state per sequence: one tensor of ``shape`` and ``dtype`` for every slot,
-    zero when a sequence starts."""
+    zero when a sequence starts.  A part that keeps several answers a dict of them by name and is
+    handed the tensors in a dict by the same names."""
 
     shape: Tuple[int, ...]
     dtype: torch.dtype = torch.float32
@@ -171,6 +173,23 @@ class Cast:
 
     def __init__(self, value):
         self.value = value
+
+
+class StreamDelta:
+    """A sublayer's result that is not in the residual yet, where the residual holds several streams: with a token's
+    streams as the rows of X, X <- M^T X + ``mult`` out (``scale`` ``delta``)^T.  ``mix`` holds M row by row and then
+    the numbers out, float32; ``scale`` one number per channel, or None."""
+
+    def __init__(self, delta, streams, mix, scale, mult):
+        self.delta, self.streams, self.mix, self.scale, self.mult = delta, streams, mix, scale, mult
+
+    def summed(self, x):
+        """All streams of ``x`` [T, streams * width] added up once this is in them (for diagnostics; x stays)."""
+        S = self.streams
+        xs = x.view(x.shape[0], S, -1)
+        y = self.delta.float() if self.scale is None else self.delta.float() * self.scale
+        into = self.mix[: S * S].view(S, S).sum(1)  # how much of stream s reaches the sum
+        return (xs * into[None, :, None]).sum(1) + self.mult * self.mix[S * S:].sum() * y
 
 
 class Norm(Part):

@@ -1,5 +1,5 @@
 """Softmax attention in its general form: a value width of its own, unit-norm queries and keys, a
-learned bias by distance, a window that keeps the first tokens, a gate per head, shared keys and values."""
+learned bias by distance, a window that keeps the first tokens, a gate per head, a sink, shared keys and values."""
 from __future__ import annotations
 
 import math
@@ -33,7 +33,8 @@ class BiasAttention(Mixer):
     output times the logistic function of its gate; output projection.  A run without projections of
     keys and values reads the cache of the run its schedule entry names.  Optional: a position encoding on q
     and k (``position``); chunks in place of the window (``chunk``); no value projection, the values being the
-    keys as projected, before the encoding (``values_are_keys``)."""
+    keys as projected, before the encoding (``values_are_keys``); a learned score per head that only enlarges the softmax's
+    denominator (``sink``)."""
 
     kernels = ("linear", "linear_mma", "linear_tc", "gemm_tc", "attention", "attention_prefill", "unit_norm", "rotary_pairs")
     TILED_MIN_TOKENS = 16  # runs of new tokens from this many on take the tensor-core kernel (bfloat16)
@@ -55,6 +56,7 @@ class BiasAttention(Mixer):
         self.w_in: Optional[torch.Tensor] = None
         self.w_o: Optional[torch.Tensor] = None
         self.rel: Optional[torch.Tensor] = None
+        self.sink: Optional[torch.Tensor] = None
 
     def children(self):
         return {"position": self.position} if self.position is not None else {}
@@ -82,6 +84,8 @@ class BiasAttention(Mixer):
             p["rel"] = ParamSpec((s.bias_buckets, s.n_heads))
         if s.head_gate:
             p["g"] = ParamSpec((s.n_heads, s.width))
+        if s.sink:
+            p["sink"] = ParamSpec((s.n_heads,))
         return p
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
@@ -109,6 +113,7 @@ class BiasAttention(Mixer):
         self.w_in = torch.cat([t.to(dt) for t in parts], dim=0).contiguous()
         self.row = at + pad
         self.w_o = tensors["o"]
+        self.sink = tensors["sink"].float().contiguous() if s.sink else None
         if s.bias_buckets:
             # the table by distance instead of by bucket: row n serves distance n, the last row every longer one
             buckets = distance_buckets(s.bias_buckets, s.bias_max_distance).to(tensors["rel"].device)
@@ -154,11 +159,12 @@ class BiasAttention(Mixer):
             # softmax weights with 16 bits of mantissa
             ops.attention_prefill(proj, self.row, out, s.n_heads, s.n_kv_heads, s.head_dim, s.scale, s.window, ctx.tile_seq,
                                   ctx.tile_row0, ctx.seq_start, ctx.seq_pos0, ctx.slots, kv.page_table, kv.k, kv.v,
-                                  keep_first=keep, rel=self.rel, gate=gate, gate_stride=self.row, precise=True, chunk=s.chunk)
+                                  keep_first=keep, rel=self.rel, gate=gate, gate_stride=self.row, precise=True, chunk=s.chunk,
+                                  sink=self.sink)
         else:
             ops.attention_general(proj, self.row, out, n, s.n_heads, s.n_kv_heads, s.head_dim, s.scale, s.window, ctx.tok_seq,
                                   ctx.tok_pos, ctx.slots, kv.page_table, kv.k, kv.v, keep_first=keep,
-                                  rel=self.rel, gate=gate, gate_stride=self.row, chunk=s.chunk,
+                                  rel=self.rel, gate=gate, gate_stride=self.row, chunk=s.chunk, sink=self.sink,
                                   max_keys=min(ctx.max_len, s.chunk or (s.window + keep)) if (s.window > 0 or s.chunk > 0) else ctx.max_len)
         ctx.tap("attn_out", out)
         return ops.linear(out, self.w_o, out_dtype=torch.float32)

@@ -1,8 +1,10 @@
 """How a mixer, a feed-forward and their norms are arranged into one block."""
 from __future__ import annotations
 
+import torch
+
 from ..csrc import ops
-from .base import Block, Cast, Normed
+from .base import Block, Cast, Normed, ParamSpec, StateRequest, StreamDelta
 from .registry import build_part, register_block
 
 
@@ -257,3 +259,100 @@ class SandwichBlock(Block):
         ctx.tap("ffn_out", f)
         h = self._add(x, f, self.ffn_post_norm, next_norm)
         return Normed(h) if h is not None else None
+
+
+@register_block("streams")
+class StreamsBlock(Block):
+    """A block on a residual of several streams: with X a token's streams as rows, sublayer q reads h_q = norm_q(in_q^T X)
+    plus the causal convolution of h_q along the sequence (its last inputs are per-sequence state), and with y its result,
+    scaled channel by channel, X becomes mix_q^T X + residual_mult out_q y^T.  An update waits as
+    ``StreamDelta`` for whoever norms next, so that update, reading, norm and (in steps of one token per sequence)
+    convolution are one pass over the streams; steps with runs of tokens take the convolution in a second pass.  Without
+    a feed-forward the second sublayer is left out; tensors that a file may hold for it are not used."""
+
+    graph_safe = True  # as far as its parts are
+    kernels = ("streams",)
+
+    def __init__(self, spec, build):
+        super().__init__(spec, build)
+        if not 1 <= spec.streams <= ops.MAX_STREAMS or not 0 <= spec.input_taps <= ops.STREAMS_MAX_TAPS:
+            raise ValueError(f"a streams block takes 1 to {ops.MAX_STREAMS} streams and up to {ops.STREAMS_MAX_TAPS} taps, "
+                             f"not {spec.streams} and {spec.input_taps}")
+        self.mixer_norm = build_part("norm", spec.mixer_norm, build)
+        self.mixer = build_part("mixer", spec.mixer, build)
+        self.ffn = build_part("ffn", spec.ffn, build) if spec.ffn is not None else None
+        self.ffn_norm = build_part("norm", spec.ffn_norm, build) if spec.ffn is not None else None
+        self.sublayers = (1, 2) if self.ffn is not None else (1,)
+
+    def children(self):
+        c = {"mixer_norm": self.mixer_norm, "mixer": self.mixer}
+        if self.ffn is not None:
+            c.update(ffn_norm=self.ffn_norm, ffn=self.ffn)
+        return c
+
+    def params(self):
+        s = self.spec
+        p = {}
+        for q in (1, 2):
+            used = q in self.sublayers  # of a sublayer that is left out the file may hold tensors or not; they are not used
+            one = lambda shape, init: ParamSpec(shape, init=init if used else "unused", optional=not used)
+            if not used:
+                p.update({f"norm{q}": one((s.width,), "ones"), f"norm{q}.b": one((s.width,), "around_zero")})
+            if s.layer_scale:
+                p[f"ls{q}"] = one((s.width,), "ones")
+            p.update({f"hc{q}.in": one((s.streams,), "ones"), f"hc{q}.out": one((s.streams,), "ones"),
+                      f"hc{q}.mix": one((s.streams, s.streams), "identity")})
+            if s.input_taps:
+                p[f"canon{q}"] = one((s.width, s.input_taps), "normal")
+        return p
+
+    def bind(self, tensors) -> None:
+        f32 = lambda t: t.float().contiguous()
+        self.read, self.mix, self.scale, self.taps = {}, {}, {}, {}
+        for q in self.sublayers:
+            self.read[q] = f32(tensors[f"hc{q}.in"])
+            self.mix[q] = torch.cat([f32(tensors[f"hc{q}.mix"]).flatten(), f32(tensors[f"hc{q}.out"])]).contiguous()
+            self.scale[q] = f32(tensors[f"ls{q}"]) if self.spec.layer_scale else None
+            self.taps[q] = f32(tensors[f"canon{q}"].t()) if self.spec.input_taps else None
+
+    def cache_request(self):
+        return self.mixer.cache_request()
+
+    def state_request(self):
+        s = self.spec
+        states = {}
+        own = self.mixer.state_request()
+        if own is not None:
+            states["mixer"] = own
+        if s.input_taps > 1:
+            for q in self.sublayers:
+                states[f"canon{q}"] = StateRequest((s.input_taps - 1, s.width), self.build.dtype)
+        return states or None
+
+    def _input(self, q, norm, x, pending, ctx, state):
+        taps = self.taps[q]
+        if taps is None:
+            return norm.streams_norm(x, pending, read=self.read[q])
+        hist = state.get(f"canon{q}") if state else None
+        if ctx.decode:
+            return norm.streams_norm(x, pending, read=self.read[q], taps=taps, hist=hist, slots=ctx.slots)
+        h = norm.streams_norm(x, pending, read=self.read[q])
+        return ops.input_convolution(h, taps, hist, ctx.tok_seq, ctx.seq_start, ctx.slots)
+
+    def _update(self, q, y):
+        s = self.spec
+        return StreamDelta(y, s.streams, self.mix[q], self.scale[q], s.residual_mult)
+
+    def forward(self, x, pending, ctx, kv, state):
+        h = self._input(1, self.mixer_norm, x, pending, ctx, state)
+        ctx.tap("attn_norm", h)
+        d = self.mixer.forward(h, ctx, kv, state.get("mixer") if state else None)
+        ctx.tap("attn_proj", d)
+        pending = self._update(1, d)
+        if self.ffn is None:
+            return pending
+        h = self._input(2, self.ffn_norm, x, pending, ctx, state)
+        ctx.tap("ffn_norm", h)
+        d = self.ffn.forward(h, ctx)
+        ctx.tap("ffn_out", d)
+        return self._update(2, d)

@@ -84,3 +84,32 @@ class LimitedMlp(FeedForward):
         act = torch.empty((h.shape[0], self.inter), dtype=gu.dtype, device=gu.device)
         ops.glu_limited(gu, act, s.limit, s.slope)
         return ops.linear(act, self.w_down, out_dtype=torch.float32)
+
+
+@register_ffn("poly_mlp")
+class PolyMlp(FeedForward):
+    """y = W_down p(W_up h) without a gate, p(z) = c1 z/r1 + c2 z^2/r2 + c3 z^3/r3 + c0 with rk the root mean square of z^k
+    over a token's numbers (eps inside the root) and four learned factors.  z and the norms are float32;
+    the delta leaves the last product in float32.  A width that is no multiple of 8 is filled up with zeros."""
+
+    kernels = ("linear", "linear_mma", "linear_tc", "gemm_tc", "act")
+    graph_safe = True
+
+    def params(self) -> Dict[str, ParamSpec]:
+        s = self.spec
+        return {"up": ParamSpec((s.intermediate, s.width)), "down": ParamSpec((s.width, s.intermediate)), "act": ParamSpec((4,))}
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        up, down = tensors["up"], tensors["down"]
+        pad = -up.shape[0] % 8
+        if pad:
+            up = torch.cat([up, torch.zeros((pad, up.shape[1]), dtype=up.dtype, device=up.device)])
+            down = torch.cat([down, torch.zeros((down.shape[0], pad), dtype=down.dtype, device=down.device)], dim=1)
+        self.w_up, self.w_down = up.contiguous(), down.contiguous()
+        self.coef = tensors["act"].float().contiguous()
+
+    def forward(self, h, ctx):
+        s = self.spec
+        z = ops.linear(h, self.w_up, out_dtype=torch.float32)
+        act = ops.poly_norm(z, self.coef, s.eps, self.build.dtype, length=s.intermediate)
+        return ops.linear(act, self.w_down, out_dtype=torch.float32)

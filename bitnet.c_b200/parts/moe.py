@@ -19,7 +19,7 @@ class Moe(FeedForward):
     g = min(gate x, limit), u = clamp(up x, -limit, limit); a shared expert of the same form (sizes and
     limit of its own) runs for every token and is added.  By the spec: ``scores`` "softmax" takes the softmax
     over all experts as scores; ``renormalise`` divides the chosen ones' by their sum (+ ``renormalise_eps``);
-    ``weight_scale`` multiplies the weights; ``activation`` "silu" / "gelu_tanh" makes an expert
+    ``router_bias`` adds a number per expert to the logits; ``weight_scale`` multiplies the weights; ``activation`` "silu" / "gelu_tanh" makes an expert
     down(act(gate x) * (up x)) without clamps; ``scores`` "table": no router, a table of expert ids by token id
     chooses and every chosen expert weighs 1 / top.
 
@@ -60,6 +60,8 @@ class Moe(FeedForward):
             p = {"table": ParamSpec((s.table_rows, s.top), init="distinct", integer=True, high=s.n_experts)}
         else:
             p = {"router": ParamSpec((s.n_experts, s.width))}
+            if s.router_bias:
+                p["router.b"] = ParamSpec((s.n_experts,))
         for e in range(s.n_experts):
             p[f"e{e}.gate"] = ParamSpec((s.expert_ff, s.width))
             p[f"e{e}.up"] = ParamSpec((s.expert_ff, s.width))
@@ -74,6 +76,7 @@ class Moe(FeedForward):
         s = self.spec
         dt = self.build.dtype
         self.w_router = tensors.get("router")
+        self.b_router = tensors["router.b"].float().contiguous() if s.router_bias else None
         self.table = tensors.get("table")
         # the table on the host too: how many tokens of a step take each expert is then known without asking the device
         self.table_host = self.table.cpu().numpy() if self.table is not None else None
@@ -103,7 +106,8 @@ class Moe(FeedForward):
             ids, weights = ctx.memo[key]
         else:
             ids, weights = ops.moe_route(h, self.w_router, s.top, s.renormalise, softmax=self.softmax,
-                                         weight_scale=getattr(s, "weight_scale", 1.0), sum_eps=getattr(s, "renormalise_eps", 0.0))
+                                         weight_scale=getattr(s, "weight_scale", 1.0), sum_eps=getattr(s, "renormalise_eps", 0.0),
+                                         bias=self.b_router)
         if ctx.diag is not None:
             ctx.tap("moe_ids", lambda: ids.float())
         if self.few_fits and (ctx.decode or T * s.top <= self.FEW_ITEMS):

@@ -1,4 +1,4 @@
-"""RMSNorm with the residual add fused in front of it."""
+"""Norms with the residual add fused in front of them."""
 from __future__ import annotations
 
 from typing import Dict
@@ -6,7 +6,7 @@ from typing import Dict
 import torch
 
 from ..csrc import ops
-from .base import Norm, ParamSpec
+from .base import Norm, ParamSpec, StreamDelta
 from .registry import register_norm
 
 
@@ -51,3 +51,36 @@ class RmsNorm(Norm):
             return x
         out = torch.empty(x.shape, dtype=self.build.dtype, device=x.device)
         return ops.scaled_add_rmsnorm(x, alpha, delta, self.weight, self.spec.eps, out)
+
+
+@register_norm("layernorm")
+class LayerNorm(Norm):
+    """out = (v - mean) / sqrt(mean((v - mean)^2) + eps) * weight + bias with v = x + delta, statistics in float32.  The
+    residual may hold several streams side by side: v is then what ``streams_norm`` is told to read of them (by default
+    their sum), and a delta comes as ``StreamDelta``."""
+
+    kernels = ("streams",)
+    graph_safe = True
+
+    def __init__(self, spec, build):
+        super().__init__(spec, build)
+        if spec.width > ops.STREAMS_MAX_WIDTH:
+            raise ValueError(f"layernorm: width={spec.width} must be at most {ops.STREAMS_MAX_WIDTH}")
+
+    def params(self) -> Dict[str, ParamSpec]:
+        return {"weight": ParamSpec((self.spec.width,), init="ones"), "bias": ParamSpec((self.spec.width,), init="around_zero")}
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.weight, self.bias = tensors["weight"], tensors["bias"]
+
+    def streams_norm(self, x, pending, read=None, rows=None, **convolution):
+        """Bring ``pending`` (None or a ``StreamDelta``) into the streams of x and norm sum_s read[s] x_s; the rest as
+        for ``ops.streams_norm``."""
+        update = dict(delta=pending.delta, mix=pending.mix, scale=pending.scale, mult=pending.mult) if pending is not None else {}
+        return ops.streams_norm(x, x.shape[1] // self.spec.width, self.weight, self.bias, self.spec.eps, self.build.dtype,
+                                read=read, rows=rows, **update, **convolution)
+
+    def add_norm(self, x, delta, ctx, rows=None):
+        if delta is not None and not isinstance(delta, StreamDelta):
+            delta = StreamDelta(delta.sum(0) if delta.dim() == 3 else delta, 1, None, None, 1.0)
+        return self.streams_norm(x, delta, rows=rows)

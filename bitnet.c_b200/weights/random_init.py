@@ -117,6 +117,8 @@ def random_parameters(spec, tensor_name, seed: int, dtype: torch.dtype, matrix_s
     from ..engine.model import parameter_table
     made: Dict[str, torch.Tensor] = {}  # parameters that share a tensor of the file get the same one
     for path, p in parameter_table(spec).items():
+        if p.init == "unused":
+            continue
         name = tensor_name(path)
         if name in made:
             yield path, name, made[name]
@@ -140,6 +142,9 @@ def _draw(path, name, p, seed, dtype, matrix_std, norm_std, device):
         z = standard_normal(seed, name, rows * p.high).reshape(rows, p.high)
         t = torch.from_numpy(np.argsort(z, axis=1, kind="stable")[:, :cols].astype(np.int32))
         yield path, name, t if device is None else t.to(device)
+    elif p.init == "identity":  # a matrix near the identity
+        yield path, name, (random_tensor(seed, name, p.shape, 0.0, norm_std, torch.float32, device)
+                           + torch.eye(p.shape[0], device=device)).to(dtype)
     elif p.init == "zeros":
         yield path, name, torch.zeros(p.shape, dtype=torch.int32 if p.integer else dtype, device=device)
     else:
