@@ -554,6 +554,38 @@ NETANEX_SIZES = {
 }
 
 
+def rudolix_sizes(width, heads, kv_heads, dim, m_heads, m_vdim, state, d_heads, d_kv_heads, d_dim, d_vdim, taps, ff, experts, top,
+                  streams, vocab):
+    """A Rudolix configuration of four layers on several residual streams (Mamba-2 with the dense unit, delta rule with
+    experts, attention with the dense unit, Mamba-2 with experts; a token's experts together as wide as the dense
+    unit), the Llama configuration of the same width, heads, layers, vocabulary and feed-forward width, and a Lotilix
+    configuration of that size, whose delta rule is the nearest relative of the recurrences."""
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff // top, "limit": 7.0}}
+    mamba = {"heads": m_heads, "groups": 1, "state": state, "vdim": m_vdim, "conv": taps, "norm_groups": 1}
+    delta = {"heads": d_heads, "kv_heads": d_kv_heads, "dim": d_dim, "vdim": d_vdim, "conv": taps}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": {"base": 5e5, "dims": dim}}
+    layers = [{"type": "mamba2", "mixer": mamba, "mlp": dense}, {"type": "delta", "mixer": delta, "mlp": moe},
+              {"type": "attention", "mixer": att, "mlp": dense}, {"type": "mamba2", "mixer": dict(mamba), "mlp": moe}]
+    rud = {"architecture": "Rudolix", "vocab": vocab, "width": width, "streams": streams, "residual_mult": 0.5, "norm": {"eps": 1e-6},
+           "canon": {"taps": 4}, "embedding": {"scale": 1.0}, "layers": layers, "max_positions": 8192}
+    llama = {"architectures": ["LlamaForCausalLM"], "model_type": "llama", "hidden_size": width, "intermediate_size": ff,
+             "num_hidden_layers": len(layers), "num_attention_heads": heads, "num_key_value_heads": kv_heads, "head_dim": dim,
+             "vocab_size": vocab, "max_position_embeddings": 8192, "rope_theta": 500000.0, "rms_norm_eps": 1e-5,
+             "tie_word_embeddings": True, "hidden_act": "silu"}
+    return rud, llama, {"lotilix": lotilix_sizes(**LOTILIX_SIZES[f"w{width}"])[0]}
+
+
+RUDOLIX_SIZES = {
+    "w1024": dict(width=1024, heads=8, kv_heads=2, dim=128, m_heads=32, m_vdim=64, state=128, d_heads=8, d_kv_heads=8, d_dim=128,
+                  d_vdim=128, taps=4, ff=4096, experts=8, top=2, streams=2, vocab=32000),
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, m_heads=64, m_vdim=64, state=128, d_heads=16, d_kv_heads=16, d_dim=128,
+                  d_vdim=128, taps=4, ff=8192, experts=8, top=2, streams=2, vocab=32000),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, m_heads=128, m_vdim=64, state=128, d_heads=32, d_kv_heads=32, d_dim=128,
+                  d_vdim=128, taps=4, ff=14336, experts=8, top=2, streams=2, vocab=32000),
+}
+
+
 def kernel_classes(model, vocab, tokens, batch, prompt_len):
     """Device time by entry point (ms) of one step of ``tokens`` prompt tokens and of one decode step of
     ``batch`` sequences behind prompts of ``prompt_len``, each kernel between two events (no graph, so the
@@ -594,7 +626,7 @@ def kernel_classes(model, vocab, tokens, batch, prompt_len):
 
 
 def run_design(args):
-    """``--design fesorax | lotilix | mekevik | netanex``: prefill and decode throughput of that design at layer sizes of real
+    """``--design fesorax | lotilix | mekevik | netanex | rudolix``: prefill and decode throughput of that design at layer sizes of real
     models (random weights, bfloat16), beside the Llama decoder of equal width, heads, layers, vocabulary and
     feed-forward work per token, with each step's device time by kernel entry point."""
     import torch
@@ -604,14 +636,14 @@ def run_design(args):
            "dtype": "bf16", "data": "synthetic", "n_gpus": 1, "peaks": pk, "prefill_tokens": PREFILL_TOKENS,
            "decode_batch": args.batch, "decode_prompt": PROMPT_LEN, "sizes": {}}
     sizes, maker = {"lotilix": (LOTILIX_SIZES, lotilix_sizes), "mekevik": (MEKEVIK_SIZES, mekevik_sizes),
-                    "netanex": (NETANEX_SIZES, netanex_sizes),
+                    "netanex": (NETANEX_SIZES, netanex_sizes), "rudolix": (RUDOLIX_SIZES, rudolix_sizes),
                     "fesorax": (DESIGN_SIZES, fesorax_sizes)}[args.design]
     rec["metric"] = rec["metric"].replace("Fesorax", args.design.capitalize())
     names = [n for n in sizes if not args.sizes or n in args.sizes.split(",")]
     for name in names:
-        fes, llama = maker(**sizes[name])
+        fes, llama, *others = maker(**sizes[name])
         row = {}
-        for label, cfg in ((args.design, fes), ("llama", llama)):
+        for label, cfg in ((args.design, fes), ("llama", llama), *(others[0].items() if others else ())):
             model = Model.from_random(cfg, seed=0, dtype="bfloat16", device="cuda:0", norm_std=0.0)
             shim = {"vocab_size": sizes[name]["vocab"], "max_position_embeddings": 4096}
             pre_ms = run_prefill(model, shim)
@@ -645,7 +677,7 @@ def main():
                          "(comparisons, profiling)")
     ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16",
                     help="compute type of the main decode run (float32: profiling of the 32-bit path, with --skip-points)")
-    ap.add_argument("--design", choices=["fesorax", "lotilix", "mekevik", "netanex"],
+    ap.add_argument("--design", choices=["fesorax", "lotilix", "mekevik", "netanex", "rudolix"],
                     help="measure another design of the library beside Llama at equal size instead (prefill, decode, "
                          "time by kernel); the default workload and its record stay as they are")
     ap.add_argument("--sizes", default="", help="with --design: which size sets, with commas (default: all)")

@@ -270,6 +270,406 @@ __global__ void __launch_bounds__(GS_THREADS) gated_state_kernel(const GatedStat
   gs_keep_inputs<T>(a, s, h, tile * 32, min(32, vdim - tile * 32), tile == 0 && h % per_group == 0);
 }
 
+// ---- runs of many tokens: the recurrence chunk by chunk ------------------------------------------------
+// Within a chunk of 64 tokens the recurrence is unrolled into sums.  With c_t the sum of the log decays from the chunk's
+// first token to t and S0 the state before the chunk,
+//
+//   o_t = e^{c_t} S0^T q_t + sum_{s <= t} e^{c_t - c_s} (q_t . k_s) u_s,      S_end = e^{c_end} S0 + sum_s e^{c_end - c_s} k_s u_s^T
+//
+// where u_s = b_s v_s for the state-space update.  In the delta rule u solves a unit lower triangular system,
+// (I + A) U = diag(b) (V - diag(e^c) K S0) with A_ts = b_t e^{c_t - c_s} (k_t . k_s) for s < t: its inverse depends on the
+// chunk alone.  (I + A)^-1 diag(b) of every chunk and head, and q_t . k_s of every chunk and group, come from a first
+// kernel, all chunks at once; a second one carries the state through the chunks with small float32 products.  Every
+// exponent is at most zero.  The sums run in another order than token by token: the forms agree to rounding.
+#define GC_L 64
+#define GC_THREADS 256
+#define GC_PLD 68  // padded rows of the chunk's 64 x 64 matrices
+
+__device__ __forceinline__ void gc_copy16(float* smem, const float* gmem, bool valid) {
+  const unsigned dst = (unsigned)__cvta_generic_to_shared(smem);
+  const int n = valid ? 16 : 0;  // zeros where there is nothing to read
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(gmem), "r"(n) : "memory");
+}
+__device__ __forceinline__ void gc_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void gc_wait() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
+// rows [row0, row0 + 64) of the matrix at src (row stride src_ld, `cols` numbers, a multiple of four), zeros past n_valid rows
+__device__ __forceinline__ void gc_load_rows(float* dst, int dst_ld, const float* src, size_t src_ld, int cols, int n_valid) {
+  const int per_row = cols >> 2;
+  for (int i = threadIdx.x; i < GC_L * per_row; i += GC_THREADS) {
+    const int r = i / per_row, c = (i - r * per_row) * 4;
+    gc_copy16(dst + r * dst_ld + c, src + (size_t)(r < n_valid ? r : 0) * src_ld + c, r < n_valid);
+  }
+}
+
+// Sums of the log decays over a chunk's tokens, by one warp: lane holds tokens 2 lane and 2 lane + 1.
+__device__ __forceinline__ float2 gc_cumulate(float l0, float l1, int lane) {
+  float both = l0 + l1;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float up = __shfl_up_sync(0xffffffffu, both, o);
+    if (lane >= o) both += up;
+  }
+  return make_float2(both - l1, both);
+}
+
+// One block per (chunk, head) in the delta rule, per (chunk, group) otherwise.  qk [T, groups, 64]: q_t . k_s for the
+// tokens s of t's chunk; winv [T, heads, 64]: the rows of (I + A)^-1 diag(b).
+template <bool DELTA>
+__global__ void __launch_bounds__(GC_THREADS) gated_state_local_kernel(const GatedStateArgs a, const float* __restrict__ qn,
+                                                                       const float* __restrict__ kn, const float* __restrict__ lb,
+                                                                       const int* __restrict__ tile_seq, const int* __restrict__ tile_row0,
+                                                                       float* __restrict__ qk, float* __restrict__ winv) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float sm[];
+  const int dim = a.dim, ld = dim + 4;
+  float* sK = sm;
+  float* sQ = sK + GC_L * ld;
+  float* sA = sQ + GC_L * ld;  // [64][GC_PLD]
+  __shared__ float sc[GC_L], sb[GC_L];
+  const int h = DELTA ? blockIdx.y : 0, per_group = a.heads / a.groups, g = DELTA ? h / per_group : blockIdx.y;
+  const int s = tile_seq[blockIdx.x], row0 = tile_row0[blockIdx.x];
+  const int first = a.seq_start[s] + row0, n_tok = min(GC_L, a.seq_start[s + 1] - first);
+  const int n_qk = a.n_qk(), tid = threadIdx.x, lane = tid & 31;
+  gc_load_rows(sK, ld, kn + (size_t)first * n_qk + g * dim, n_qk, dim, n_tok);
+  const bool with_qk = !DELTA || h % per_group == 0;
+  if (with_qk) gc_load_rows(sQ, ld, qn + (size_t)first * n_qk + g * dim, n_qk, dim, n_tok);
+  gc_commit();
+  if (DELTA && tid < 32) {
+    float l[2], b[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = 2 * lane + e;
+      const float* p = lb + ((size_t)(first + t) * a.heads + h) * 2;
+      l[e] = t < n_tok ? p[0] : 0.f;
+      b[e] = t < n_tok ? p[1] : 0.f;
+    }
+    const float2 c = gc_cumulate(l[0], l[1], lane);
+    sc[2 * lane] = c.x; sc[2 * lane + 1] = c.y;
+    sb[2 * lane] = b[0]; sb[2 * lane + 1] = b[1];
+  }
+  gc_wait();
+  __syncthreads();
+  const int rg = tid >> 4, cg = tid & 15;  // rows rg + 16 i, columns cg + 16 j
+  for (int which = DELTA ? 0 : 1; which < 2; ++which) {  // 0: k . k, 1: q . k
+    if (which == 1 && !with_qk) break;
+    const float* X = which ? sQ : sK;
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    for (int d = 0; d < dim; d += 4) {
+      float4 x[4], y[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x[i] = *reinterpret_cast<const float4*>(X + (rg + 16 * i) * ld + d);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) y[j] = *reinterpret_cast<const float4*>(sK + (cg + 16 * j) * ld + d);
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (j <= i) {  // column block j beyond row block i lies above the diagonal
+            acc[i][j] = fmaf(x[i].x, y[j].x, acc[i][j]); acc[i][j] = fmaf(x[i].y, y[j].y, acc[i][j]);
+            acc[i][j] = fmaf(x[i].z, y[j].z, acc[i][j]); acc[i][j] = fmaf(x[i].w, y[j].w, acc[i][j]);
+          }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int t = rg + 16 * i, u = cg + 16 * j;
+        if (which == 0) sA[t * GC_PLD + u] = u < t ? sb[t] * expf(sc[t] - sc[u]) * acc[i][j] : 0.f;
+        else if (t < n_tok) qk[((size_t)(first + t) * a.groups + g) * GC_L + u] = u <= t ? acc[i][j] : 0.f;
+      }
+  }
+  if (!DELTA) return;
+  __syncthreads();
+  if (tid < GC_L) {  // a thread per column of the inverse, by forward substitution in registers
+    float x[GC_L];
+#pragma unroll
+    for (int t = 0; t < GC_L; ++t) {
+      float p0 = t == tid ? 1.0f : 0.f, p1 = 0.f, p2 = 0.f, p3 = 0.f;
+#pragma unroll
+      for (int u = 0; u + 3 < t; u += 4) {
+        const float4 r = *reinterpret_cast<const float4*>(sA + t * GC_PLD + u);
+        p0 = fmaf(-r.x, x[u], p0); p1 = fmaf(-r.y, x[u + 1], p1); p2 = fmaf(-r.z, x[u + 2], p2); p3 = fmaf(-r.w, x[u + 3], p3);
+      }
+#pragma unroll
+      for (int u = t / 4 * 4; u < t; ++u) p0 = fmaf(-sA[t * GC_PLD + u], x[u], p0);
+      x[t] = (p0 + p1) + (p2 + p3);
+    }
+    const float b = sb[tid];
+#pragma unroll
+    for (int t = 0; t < GC_L; ++t)
+      if (t < n_tok) winv[((size_t)(first + t) * a.heads + h) * GC_L + tid] = x[t] * b;
+  }
+}
+
+template <int N>
+__device__ __forceinline__ void gc_read(const float* p, float* o);
+template <>
+__device__ __forceinline__ void gc_read<4>(const float* p, float* o) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  o[0] = a.x; o[1] = a.y; o[2] = a.z; o[3] = a.w;
+}
+template <>
+__device__ __forceinline__ void gc_read<2>(const float* p, float* o) {
+  const float2 a = *reinterpret_cast<const float2*>(p);
+  o[0] = a.x; o[1] = a.y;
+}
+template <int N>
+__device__ __forceinline__ void gc_write(float* p, const float* o);
+template <>
+__device__ __forceinline__ void gc_write<4>(float* p, const float* o) { *reinterpret_cast<float4*>(p) = make_float4(o[0], o[1], o[2], o[3]); }
+template <>
+__device__ __forceinline__ void gc_write<2>(float* p, const float* o) { *reinterpret_cast<float2*>(p) = make_float2(o[0], o[1]); }
+
+// acc[i][:] += M[row rg + 32 i][0 .. end) . U for the thread's TC columns; M's rows GC_PLD apart, end a multiple of four
+template <int NR, int TC>
+__device__ __forceinline__ void gc_product(float (*acc)[TC], const float* M, const float* U, int ct, int rg, int cg, int end) {
+  for (int s = 0; s < end; s += 4) {
+    float4 m[NR];
+#pragma unroll
+    for (int i = 0; i < NR; ++i) m[i] = *reinterpret_cast<const float4*>(M + (rg + 32 * i) * GC_PLD + s);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float u[TC];
+      gc_read<TC>(U + (s + e) * ct + cg * TC, u);
+#pragma unroll
+      for (int i = 0; i < NR; ++i) {
+        const float f = e == 0 ? m[i].x : e == 1 ? m[i].y : e == 2 ? m[i].z : m[i].w;
+#pragma unroll
+        for (int c = 0; c < TC; ++c) acc[i][c] = fmaf(f, u[c], acc[i][c]);
+      }
+    }
+  }
+}
+
+static size_t gc_smem_floats(int dim, int ct, int stages) {
+  return (size_t)stages * 2 * GC_L * (dim + 4) + (size_t)dim * ct + 3 * GC_L * ct + (size_t)stages * GC_L * GC_PLD + GC_L * GC_PLD + 4 * GC_L;
+}
+
+// The chain: one block per (sequence, head, CT value columns).  Thread = (tokens rg and rg + 32, TC columns); in the
+// state's update (four rows of the state, TC columns).  With two stages the next chunk's rows arrive while this one's are
+// worked on.
+template <typename T, bool DELTA, int CT>
+__global__ void __launch_bounds__(GC_THREADS) gated_state_chunk_kernel(const GatedStateArgs a, const float* __restrict__ qn,
+                                                                       const float* __restrict__ kn, const float* __restrict__ vc,
+                                                                       const float* __restrict__ lb, const float* __restrict__ qk,
+                                                                       const float* __restrict__ winv, int col_tiles, int stages,
+                                                                       float* __restrict__ out) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int TC = CT / 8;
+  constexpr int NR = DELTA ? 4 : 2;  // rows of [K; Q] S0 per thread: K rows rg, rg + 32 (delta), then Q rows
+  extern __shared__ __align__(16) float sm[];
+  const int heads = a.heads, dim = a.dim, vdim = a.vdim, ld = dim + 4, n_qk = a.n_qk();
+  float* sKQ = sm;                                        // [stages][K 64 rows | Q 64 rows][ld]
+  float* sS = sKQ + (size_t)stages * 2 * GC_L * ld;       // [dim][CT]
+  float* sR = sS + (size_t)dim * CT;                      // [64][CT] right-hand sides
+  float* sU = sR + GC_L * CT;                             // [64][CT] u
+  float* sD = sU + GC_L * CT;                             // [64][CT] u times its weight in the state after the chunk
+  float* sP = sD + GC_L * CT;                             // [stages][64][GC_PLD]
+  float* sW = sP + (size_t)stages * GC_L * GC_PLD;        // [64][GC_PLD]
+  float* sc = sW + GC_L * GC_PLD;                         // [64] c, then b, e^c, e^(c_end - c)
+  float *sb = sc + GC_L, *se = sb + GC_L, *sd = se + GC_L;
+  const int tile = blockIdx.x % col_tiles, h = (blockIdx.x / col_tiles) % heads, s = blockIdx.x / (col_tiles * heads);
+  const int per_group = heads / a.groups, g = h / per_group;
+  const int tid = threadIdx.x, lane = tid & 31, rg = tid >> 3, cg = tid & 7;
+  const int col0 = tile * CT, col = col0 + cg * TC;
+  const int start = a.seq_start[s], n = a.seq_start[s + 1] - start;
+  float* S_g = a.state + (size_t)a.slots[s] * a.state_stride + (size_t)h * dim * vdim;
+  for (int i = tid; i < dim * CT; i += GC_THREADS) {
+    const int d = i / CT, c = col0 + i - d * CT;
+    sS[i] = c < vdim ? S_g[(size_t)d * vdim + c] : 0.f;
+  }
+  const float skip = a.d ? a.d[h] : 0.f;
+  auto load_kq = [&](int base, int stage) {
+    float* dst = sKQ + (size_t)stage * 2 * GC_L * ld;
+    const int left = min(GC_L, n - base);
+    gc_load_rows(dst, ld, kn + (size_t)(start + base) * n_qk + g * dim, n_qk, dim, left);
+    gc_load_rows(dst + GC_L * ld, ld, qn + (size_t)(start + base) * n_qk + g * dim, n_qk, dim, left);
+    gc_load_rows(sP + (size_t)stage * GC_L * GC_PLD, GC_PLD, qk + ((size_t)(start + base) * a.groups + g) * GC_L, (size_t)a.groups * GC_L,
+                 GC_L, left);
+  };
+  auto load_w = [&](int base) {
+    gc_load_rows(sW, GC_PLD, winv + ((size_t)(start + base) * heads + h) * GC_L, (size_t)heads * GC_L, GC_L, min(GC_L, n - base));
+  };
+  float v_next[2][TC], l_next[2] = {0.f, 0.f}, b_next[2] = {0.f, 0.f};
+  auto load_v = [&](int base) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int t = base + rg + 32 * i;
+#pragma unroll
+      for (int c = 0; c < TC; ++c)
+        v_next[i][c] = t < n && col + c < vdim ? vc[(size_t)(start + t) * heads * vdim + (size_t)h * vdim + col + c] : 0.f;
+    }
+    if (tid < 32) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int t = base + 2 * lane + e;
+        const float* p = lb + ((size_t)(start + t) * heads + h) * 2;
+        l_next[e] = t < n ? p[0] : 0.f;
+        b_next[e] = t < n ? p[1] : 0.f;
+      }
+    }
+  };
+  if (stages == 2) load_kq(0, 0);
+  if (DELTA) load_w(0);
+  gc_commit();
+  load_v(0);
+  for (int base = 0, stage = 0; base < n; base += GC_L, stage ^= stages - 1) {
+    __syncthreads();  // the chunk before is done with everything in shared memory
+    if (stages == 1) {
+      load_kq(base, 0);
+      gc_commit();
+    }
+    if (tid < 32) {
+      const float2 c = gc_cumulate(l_next[0], l_next[1], lane);
+      const float end = __shfl_sync(0xffffffffu, c.y, 31);  // tokens past the end have log decay 0
+      sc[2 * lane] = c.x; sc[2 * lane + 1] = c.y;
+      sb[2 * lane] = b_next[0]; sb[2 * lane + 1] = b_next[1];
+      se[2 * lane] = expf(c.x); se[2 * lane + 1] = expf(c.y);
+      sd[2 * lane] = expf(end - c.x); sd[2 * lane + 1] = expf(end - c.y);
+    }
+    float v[2][TC];
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int c = 0; c < TC; ++c) v[i][c] = v_next[i][c];
+    gc_wait();
+    __syncthreads();
+    const bool more = base + GC_L < n;
+    if (more) {
+      if (stages == 2) {
+        load_kq(base + GC_L, stage ^ 1);
+        gc_commit();
+      }
+      load_v(base + GC_L);
+    }
+    const float* K = sKQ + (size_t)stage * 2 * GC_L * ld;
+    float* P = sP + (size_t)stage * GC_L * GC_PLD;
+    // the decays onto q . k (above the diagonal the first kernel left zeros)
+    for (int i = tid; i < GC_L * GC_L; i += GC_THREADS) {
+      const int t = i >> 6, u = i & 63;
+      if (u <= t) P[t * GC_PLD + u] *= expf(sc[t] - sc[u]);
+    }
+    float acc[NR][TC];
+#pragma unroll
+    for (int i = 0; i < NR; ++i)
+#pragma unroll
+      for (int c = 0; c < TC; ++c) acc[i][c] = 0.f;
+    const float* X = DELTA ? K : K + GC_L * ld;
+    for (int d = 0; d < dim; d += 4) {
+      float4 x[NR];
+#pragma unroll
+      for (int i = 0; i < NR; ++i) x[i] = *reinterpret_cast<const float4*>(X + (rg + 32 * i) * ld + d);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        float sv[TC];
+        gc_read<TC>(sS + (d + e) * CT + cg * TC, sv);
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+          const float f = e == 0 ? x[i].x : e == 1 ? x[i].y : e == 2 ? x[i].z : x[i].w;
+#pragma unroll
+          for (int c = 0; c < TC; ++c) acc[i][c] = fmaf(f, sv[c], acc[i][c]);
+        }
+      }
+    }
+    float o[2][TC];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int t = rg + 32 * i;
+      float r[TC];
+#pragma unroll
+      for (int c = 0; c < TC; ++c) {
+        o[i][c] = acc[NR - 2 + i][c] * se[t];
+        r[c] = DELTA ? v[i][c] - acc[i][c] * se[t] : v[i][c] * sb[t];
+      }
+      if (DELTA) {
+        gc_write<TC>(sR + t * CT + cg * TC, r);
+      } else {
+        gc_write<TC>(sU + t * CT + cg * TC, r);
+#pragma unroll
+        for (int c = 0; c < TC; ++c) r[c] *= sd[t];
+        gc_write<TC>(sD + t * CT + cg * TC, r);
+      }
+    }
+    __syncthreads();
+    // a warp's tokens are 4 w .. 4 w + 3 and those + 32: sums over the chunk's earlier tokens end behind the later ones
+    const int last = (tid >> 5) * 4 + 36;
+    if (DELTA) {
+      float u[2][TC];
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int c = 0; c < TC; ++c) u[i][c] = 0.f;
+      gc_product<2, TC>(u, sW, sR, CT, rg, cg, last);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int t = rg + 32 * i;
+        gc_write<TC>(sU + t * CT + cg * TC, u[i]);
+#pragma unroll
+        for (int c = 0; c < TC; ++c) u[i][c] *= sd[t];
+        gc_write<TC>(sD + t * CT + cg * TC, u[i]);
+      }
+      __syncthreads();
+      if (more) {
+        load_w(base + GC_L);
+        gc_commit();
+      }
+    }
+    gc_product<2, TC>(o, P, sU, CT, rg, cg, last);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int t = base + rg + 32 * i;
+      if (t < n) {
+        float* dst = out + (size_t)(start + t) * heads * vdim + (size_t)h * vdim + col;
+#pragma unroll
+        for (int c = 0; c < TC; ++c)
+          if (col + c < vdim) dst[c] = fmaf(skip, v[i][c], o[i][c]);
+      }
+    }
+    const float carry = se[GC_L - 1];
+    for (int d = rg * 4; d < dim; d += 128) {
+      float n4[4][TC];
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+#pragma unroll
+        for (int c = 0; c < TC; ++c) n4[e][c] = 0.f;
+#pragma unroll 4
+      for (int t = 0; t < GC_L; ++t) {
+        const float4 k = *reinterpret_cast<const float4*>(K + t * ld + d);
+        float u[TC];
+        gc_read<TC>(sD + t * CT + cg * TC, u);
+#pragma unroll
+        for (int c = 0; c < TC; ++c) {
+          n4[0][c] = fmaf(k.x, u[c], n4[0][c]);
+          n4[1][c] = fmaf(k.y, u[c], n4[1][c]);
+          n4[2][c] = fmaf(k.z, u[c], n4[2][c]);
+          n4[3][c] = fmaf(k.w, u[c], n4[3][c]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        float old[TC];
+        gc_read<TC>(sS + (d + e) * CT + cg * TC, old);
+#pragma unroll
+        for (int c = 0; c < TC; ++c) old[c] = fmaf(carry, old[c], n4[e][c]);
+        gc_write<TC>(sS + (d + e) * CT + cg * TC, old);
+      }
+    }
+  }
+  __syncthreads();
+  for (int i = tid; i < dim * CT; i += GC_THREADS) {
+    const int d = i / CT, c = col0 + i - d * CT;
+    if (c < vdim) S_g[(size_t)d * vdim + c] = sS[i];
+  }
+  gs_keep_inputs<T>(a, s, h, col0, min(CT, vdim - col0), tile == 0 && h % per_group == 0);
+}
+
 // Steps of one token per sequence: convolution, gates, unit norms, one step of the recurrence and the ring in one
 // launch.  Blocks as above; each of them convolves its group's q and k channels itself.
 template <typename T, int RW, bool DELTA>
@@ -456,6 +856,61 @@ extern "C" int bn_gated_state_run(GS_PARAMS, const float* qn, const float* kn, c
   else if (dtype == BN_BF16) GS_BY_SIZE(GS_RUN, __nv_bfloat16);
   else return BN_ERR_BAD_ARG;
 #undef GS_RUN
+  return BN_OK;
+}
+
+// As bn_gated_state_run, by chunks of 64 tokens (for steps that bring runs of many tokens; dim a multiple of four).
+// tile_seq / tile_row0: the sequence and first row of every run of 64 new tokens.  qk [T, groups, 64] and, for the delta
+// rule, winv [T, heads, 64] are working space.
+extern "C" int bn_gated_state_chunks(GS_PARAMS, const float* qn, const float* kn, const float* vc, const float* lb, const int* tile_seq,
+                                     const int* tile_row0, int n_tiles, float* qk, float* winv, float* out, cudaStream_t stream) {
+  if (n_tokens <= 0 || n_seqs <= 0) return BN_OK;
+  const GatedStateArgs a = gs_args(GS_PASS);
+  const bool delta = b_off >= 0;
+  if (!gs_fits(a) || !qn || !kn || !vc || !lb || !out || !tile_seq || !tile_row0 || n_tiles <= 0 || !qk || (delta && !winv) || dim % 4 ||
+      heads > 65535 || (((uintptr_t)qn | (uintptr_t)kn | (uintptr_t)qk | (uintptr_t)winv) & 15))
+    return BN_ERR_BAD_ARG;
+  const size_t local = ((size_t)(2 * GC_L) * (dim + 4) + (delta ? GC_L * GC_PLD : 0)) * sizeof(float);
+  if (local > 200 * 1024) return BN_ERR_BAD_ARG;
+  static size_t granted_local[2] = {0, 0};
+  if (local > 48 * 1024 && local > granted_local[delta]) {
+    cudaError_t e = delta ? cudaFuncSetAttribute(gated_state_local_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)local)
+                          : cudaFuncSetAttribute(gated_state_local_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)local);
+    if (e != cudaSuccess) return BN_ERR_LAUNCH + (int)e;
+    granted_local[delta] = local;
+  }
+  if (delta)
+    BN_LAUNCH(gated_state_local_kernel<true>, dim3(n_tiles, heads), GC_THREADS, local, stream, a, qn, kn, lb, tile_seq, tile_row0, qk, winv);
+  else
+    BN_LAUNCH(gated_state_local_kernel<false>, dim3(n_tiles, groups), GC_THREADS, local, stream, a, qn, kn, lb, tile_seq, tile_row0, qk, winv);
+  // 32 columns per block, or 16 where that leaves most of the SMs without one
+  const int ct = (long long)n_seqs * heads * ((vdim + 31) / 32) >= 100 || vdim <= 8 ? 32 : 16;
+  const int col_tiles = (vdim + ct - 1) / ct;
+  const int stages = gc_smem_floats(dim, ct, 2) * sizeof(float) <= 227 * 1024 ? 2 : 1;
+  const size_t smem = gc_smem_floats(dim, ct, stages) * sizeof(float);
+  const long long blocks = (long long)n_seqs * heads * col_tiles;
+  if (smem > 227 * 1024 || blocks > 2147483647LL) return BN_ERR_BAD_ARG;
+#define GC_RUN(TT, DD, CC)                                                                                                               \
+  do {                                                                                                                                   \
+    static size_t granted = 0;                                                                                                           \
+    if (smem > granted) {                                                                                                                \
+      cudaError_t e = cudaFuncSetAttribute(gated_state_chunk_kernel<TT, DD, CC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      if (e != cudaSuccess) return BN_ERR_LAUNCH + (int)e;                                                                               \
+      granted = smem;                                                                                                                    \
+    }                                                                                                                                    \
+    BN_LAUNCH((gated_state_chunk_kernel<TT, DD, CC>), (unsigned)blocks, GC_THREADS, smem, stream, a, qn, kn, vc, lb, qk, winv, col_tiles, \
+              stages, out);                                                                                                              \
+  } while (0)
+#define GC_RUN_T(TT)                                                                       \
+  do {                                                                                     \
+    if (delta) { if (ct == 32) GC_RUN(TT, true, 32); else GC_RUN(TT, true, 16); }          \
+    else { if (ct == 32) GC_RUN(TT, false, 32); else GC_RUN(TT, false, 16); }              \
+  } while (0)
+  if (dtype == BN_F32) GC_RUN_T(float);
+  else if (dtype == BN_BF16) GC_RUN_T(__nv_bfloat16);
+  else return BN_ERR_BAD_ARG;
+#undef GC_RUN_T
+#undef GC_RUN
   return BN_OK;
 }
 

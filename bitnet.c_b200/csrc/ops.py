@@ -1615,6 +1615,7 @@ def delta_output(o: torch.Tensor, gain: torch.Tensor, gate: torch.Tensor, heads:
 # ---- matrix states under one decay per head ------------------------------------------------------
 GATED_STATE_MAX_DIM = 256
 GATED_STATE_MAX_TAPS = 16
+GATED_STATE_CHUNK = 64  # tokens per chunk; must equal GC_L in gated_state.cu and the step's runs of new tokens
 
 
 def gated_state_floats(heads: int, groups: int, dim: int, vdim: int, taps: int) -> int:
@@ -1627,7 +1628,7 @@ def gated_state(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: t
                 conv_w: torch.Tensor, conv_b: Optional[torch.Tensor], dt_bias: torch.Tensor, a_log: torch.Tensor,
                 skip: Optional[torch.Tensor], state: torch.Tensor, tok_seq: torch.Tensor, seq_start: torch.Tensor,
                 seq_pos0: torch.Tensor, slots: torch.Tensor, n_seqs: int, heads: int, groups: int, dim: int, vdim: int,
-                one_token: bool) -> torch.Tensor:
+                one_token: bool, tile_seq: Optional[torch.Tensor] = None, tile_row0: Optional[torch.Tensor] = None) -> torch.Tensor:
     """A matrix state per head over the new tokens of every sequence, from and into ``state`` ``[slots,
     gated_state_floats]`` (float32), under one decay per head and token.  ``proj`` ``[T, n]``: rows with the channels of
     q and k (``groups * dim`` each) and v (``heads * vdim``) at their offsets; each channel passes a causal convolution
@@ -1637,7 +1638,9 @@ def gated_state(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: t
     softplus(a + ``dt_bias``), b = sigmoid(.); S <- e^l S; u = b (v - S^T k); S <- S + k u^T; o = S^T q.
     ``b_off`` < 0, the state-space update: b = softplus(a + ``dt_bias``), l = -exp(``a_log``) b;
     S <- e^l S + b k v^T; o = S^T q + ``skip`` v.
-    ``one_token``: every sequence brings one token (one launch does it all).  Returns o, float32 ``[T, heads * vdim]``."""
+    ``one_token``: every sequence brings one token (one launch does it all).  ``tile_seq`` / ``tile_row0``: the runs of 64
+    new tokens (sequence, first row); with them the recurrence goes chunk by chunk instead of token by token (``dim`` a
+    multiple of four).  Returns o, float32 ``[T, heads * vdim]``."""
     _need(proj, "proj", dims=2)
     _need(conv_w, "conv_w", torch.float32, 2)
     _need(state, "state", torch.float32, 2)
@@ -1674,6 +1677,16 @@ def gated_state(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: t
     lb = torch.empty((T, heads, 2), dtype=torch.float32, device=dev)
     between = (_ptr(qn), _ptr(kn), _ptr(vc), _ptr(lb))
     _check(_fn("gated_state", "bn_gated_state_prepare")(*args, *between, _stream()), "gated_state_prepare")
+    if tile_seq is not None and dim % 4 == 0:
+        _need(tile_seq, "tile_seq", torch.int32, 1)
+        _need(tile_row0, "tile_row0", torch.int32, 1)
+        qk = torch.empty((T, groups, GATED_STATE_CHUNK), dtype=torch.float32, device=dev)
+        winv = torch.empty((T, heads, GATED_STATE_CHUNK), dtype=torch.float32, device=dev) if b_off >= 0 else None
+        global LAUNCHES
+        LAUNCHES += 1  # what each chunk needs of itself, then the chain through the chunks
+        _check(_fn("gated_state", "bn_gated_state_chunks")(*args, *between, _ptr(tile_seq), _ptr(tile_row0), int(tile_seq.shape[0]),
+                                                           _ptr(qk), _ptr(winv), _ptr(out), _stream()), "gated_state_chunks")
+        return out
     _check(_fn("gated_state", "bn_gated_state_run")(*args, *between, _ptr(out), _stream()), "gated_state_run")
     return out
 

@@ -20,6 +20,7 @@ class GatedStateMixer(Mixer):
 
     kernels = ("linear", "linear_mma", "linear_tc", "gemm_tc", "gated_state")
     graph_safe = True
+    CHUNKED_MIN_TOKENS = 16  # steps with a run of so many new tokens take the recurrence chunk by chunk
     n_heads = n_groups = dim = vdim = taps = 0  # set by the mixers
 
     def _check_sizes(self) -> None:
@@ -51,9 +52,11 @@ class GatedStateMixer(Mixer):
                 ops.linear(h, self.w_in[self.main:], out_dtype=torch.float32))
 
     def _recur(self, proj, gates, ctx, state):
+        chunked = not ctx.decode and ctx.max_new >= self.CHUNKED_MIN_TOKENS and ctx.tile_seq is not None
+        tiles = dict(tile_seq=ctx.tile_seq, tile_row0=ctx.tile_row0) if chunked else {}
         o = ops.gated_state(proj, self.q_off, self.k_off, self.v_off, gates, self.a_off, self.b_off, self.conv_w, self.conv_b,
                             self.dt_bias, self.a_log, self.skip, state, ctx.tok_seq, ctx.seq_start, ctx.seq_pos0, ctx.slots,
-                            ctx.n_seqs, self.n_heads, self.n_groups, self.dim, self.vdim, one_token=ctx.decode)
+                            ctx.n_seqs, self.n_heads, self.n_groups, self.dim, self.vdim, one_token=ctx.decode, **tiles)
         ctx.tap("state_raw", o)
         return o
 
