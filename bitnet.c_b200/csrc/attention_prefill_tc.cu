@@ -22,6 +22,9 @@
 // the tensor pipe runs its instructions in order, so S_{j+2}, issued after P_j V_j, cannot
 // overwrite P_j before it has been used.  V is that product's B operand with the head dimension
 // contiguous (MN-major); K and Q are K-major.
+// With PRECISE the weights enter the second product as two bfloat16 terms, P = P_hi + P_lo (16 bits of mantissa): P_lo
+// takes the second half of the columns S_j came from, and O += P_lo V_j follows O += P_hi V_j.  Value rows may have a
+// width of their own (VD), and a sink, a score per head without a key or a value, may enlarge the rows' sums at the end.
 // The new tokens' own keys and values must already be in the cache, so the same kernel serves
 // whole prompts, pieces of prompts and ragged batches (a table gives each block its sequence and
 // first row).  Head sizes in steps of 16 up to 128 run on the instantiation for 64 or 128: columns
@@ -48,7 +51,8 @@
 struct PtArgs {
   __nv_bfloat16* out;
   int out_stride;
-  int n_heads, n_kv_heads, head_dim;
+  int n_heads, n_kv_heads, head_dim, v_dim;
+  const float* sink;  // [n_heads] or null
   float scale_log2e;
   int window;
   const int* tile_seq;
@@ -78,29 +82,30 @@ __device__ __forceinline__ bool pt_wait(unsigned bar, unsigned parity, volatile 
   }
 }
 
-template <int HD, int KS, int VS>
+template <int HD, int VD, int KS, int VS, bool PRECISE>
 __global__ void __launch_bounds__(PT_THREADS)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, PtArgs a) {
   pdl_launch_dependents();  // the next kernel in the stream may begin its prologue
   extern __shared__ __align__(1024) unsigned char smem_raw[];
-  constexpr int BOXES = HD / 64;
+  constexpr int BOXES = HD / 64, V_BOXES = VD / 64;
   constexpr int Q_BOX = PT_ROWS * 128;             // 16 KB: 128 rows x 64 dimensions
   constexpr int KV_BOX = PT_KEYS * 128;            // 8 KB: 64 keys x 64 dimensions
   constexpr int Q_BYTES = BOXES * Q_BOX;
-  constexpr int PAGE_BYTES = BOXES * KV_BOX;       // one page of keys (or values) of one head
+  constexpr int PAGE_BYTES = BOXES * KV_BOX;       // one page of keys of one head
+  constexpr int V_BYTES = V_BOXES * KV_BOX;        // and of values
   constexpr unsigned TMEM_COLS = 256;              // S0 at 0, S1 at 64, O at 128
   constexpr unsigned O_COL = 128;
-  // D float32, A and B bfloat16, M = 128; scores: N = 64, both operands K-major; output: N = HD, B MN-major
+  // D float32, A and B bfloat16, M = 128; scores: N = 64, both operands K-major; output: N = VD, B MN-major
   constexpr unsigned IDESC_S = (1u << 4) | (1u << 7) | (1u << 10) | ((unsigned)(PT_KEYS >> 3) << 17) | ((PT_ROWS >> 4) << 24);
-  constexpr unsigned IDESC_O = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((unsigned)(HD >> 3) << 17) | ((PT_ROWS >> 4) << 24);
+  constexpr unsigned IDESC_O = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((unsigned)(VD >> 3) << 17) | ((PT_ROWS >> 4) << 24);
 
   // The block has no static shared memory, so the dynamic part starts at the (1024-byte aligned)
   // base of the block's window: the swizzle is a function of the address.
   unsigned char* q_smem = smem_raw;
   unsigned char* k_smem = q_smem + Q_BYTES;                   // KS pages of keys
   unsigned char* v_smem = k_smem + KS * PAGE_BYTES;           // VS pages of values
-  unsigned long long* bars = (unsigned long long*)(v_smem + VS * PAGE_BYTES);
+  unsigned long long* bars = (unsigned long long*)(v_smem + VS * V_BYTES);
   // barriers: q_full, k_full[KS], k_empty[KS], v_full[VS], v_empty[VS], s_full[2], p_full[2], pv_done
   const unsigned bar0 = smem_u32(bars);
   const unsigned q_full = bar0, k_full0 = bar0 + 8, k_empty0 = k_full0 + 8 * KS, v_full0 = k_empty0 + 8 * KS,
@@ -177,11 +182,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const unsigned empty = (values ? v_empty0 : k_empty0) + 8 * s, bar = (values ? v_full0 : k_full0) + 8 * s;
         const int page = __ldg(pt + tile_lo + j);  // asked for before the wait, needed after it
         if (round > 0 && !pt_wait(empty, (unsigned)(round - 1) & 1u, failed, a.status)) return false;
-        const unsigned dst = smem_u32((values ? v_smem : k_smem) + s * PAGE_BYTES);
-        mbar_expect_tx(bar, PAGE_BYTES);
+        const unsigned dst = smem_u32(values ? v_smem + s * V_BYTES : k_smem + s * PAGE_BYTES);
+        mbar_expect_tx(bar, values ? V_BYTES : PAGE_BYTES);
 #pragma unroll
-        for (int bx = 0; bx < BOXES; ++bx)
-          tma_load_3d(dst + bx * KV_BOX, values ? &map_v : &map_k, bar, bx * 64, kvh * BN_PAGE, page);
+        for (int bx = 0; bx < (BOXES > V_BOXES ? BOXES : V_BOXES); ++bx)
+          if (bx < (values ? V_BOXES : BOXES)) tma_load_3d(dst + bx * KV_BOX, values ? &map_v : &map_k, bar, bx * 64, kvh * BN_PAGE, page);
         return true;
       };
       bool ok = true;
@@ -233,12 +238,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         BN_TRACE_ONLY(const bool tr = tracing && i < PT_TRACE_TILES;)
         BN_TRACE_ONLY(if (tr) a.trace[i * 12 + 7] = global_timer();)
-        const unsigned sv = smem_u32(v_smem + s * PAGE_BYTES);
+        const unsigned sv = smem_u32(v_smem + s * V_BYTES);
         if (issuer) {
 #pragma unroll
           for (int kk = 0; kk < PT_KEYS / 16; ++kk)
             umma_mma_ts(tbase + O_COL, tbase + b * PT_KEYS + kk * 8, umma_desc_mn(sv + kk * 2048, KV_BOX), IDESC_O,
                       (i | kk) ? 1u : 0u);
+          if (PRECISE) {
+#pragma unroll
+            for (int kk = 0; kk < PT_KEYS / 16; ++kk)
+              umma_mma_ts(tbase + O_COL, tbase + b * PT_KEYS + PT_KEYS / 2 + kk * 8, umma_desc_mn(sv + kk * 2048, KV_BOX), IDESC_O, 1u);
+          }
           umma_commit(v_empty0 + 8 * s);    // the value stage may be refilled
           umma_commit(pv_done);             // O holds the pages up to i
           BN_TRACE_ONLY(if (tr) a.trace[i * 12 + 8] = global_timer();)
@@ -289,7 +299,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const float alpha = need ? exp2f(m_ref - m_tile) : 1.0f;
         if (need) { m_ref = m_tile; l_run *= alpha; }
 #pragma unroll
-        for (int c = 0; c < HD; c += 32) {
+        for (int c = 0; c < VD; c += 32) {
           float o[32];
           tmem_ld32(lane_addr + O_COL + c, o);
 #pragma unroll
@@ -314,17 +324,29 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       {
         float pk[32];
 #pragma unroll
-        for (int c = 0; c < 32; ++c) pk[c] = __uint_as_float(pack_bf16x2(s[2 * c], s[2 * c + 1]));
+        for (int c = 0; c < 32; ++c) {
+          const unsigned both = pack_bf16x2(s[2 * c], s[2 * c + 1]);
+          pk[c] = __uint_as_float(both);
+          if (PRECISE) {  // what the rounding left over
+            s[2 * c] -= __uint_as_float(both << 16);
+            s[2 * c + 1] -= __uint_as_float(both & 0xffff0000u);
+          }
+        }
         tmem_st32(lane_addr + b * PT_KEYS, pk);
+        if (PRECISE) {
+#pragma unroll
+          for (int c = 0; c < 32; ++c) pk[c] = __uint_as_float(pack_bf16x2(s[2 * c], s[2 * c + 1]));
+          tmem_st32(lane_addr + b * PT_KEYS + PT_KEYS / 2, pk);
+        }
         asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
       }
       if (tile * PT_KEYS + PT_KEYS - 1 > seq_last) {
         // the page holds rows behind the sequence's last position: their weights are zero, but zero
         // times anything must be zero, so clear those value rows (warp w takes every fourth row)
-        unsigned char* sv = v_smem + (j % VS) * PAGE_BYTES;
+        unsigned char* sv = v_smem + (j % VS) * V_BYTES;
         const int first = max(0, seq_last + 1 - tile * PT_KEYS);
-        for (int e = (warp - 2) * 32 + lane; e < (PT_KEYS - first) * (HD / 8); e += 128) {
-          int row = first + e / (HD / 8), c = e % (HD / 8);
+        for (int e = (warp - 2) * 32 + lane; e < (PT_KEYS - first) * (VD / 8); e += 128) {
+          int row = first + e / (VD / 8), c = e % (VD / 8);
           *reinterpret_cast<uint4*>(sv + (c >> 3) * KV_BOX + row * 128 + (((c & 7) ^ (row & 7)) << 4)) = make_uint4(0u, 0u, 0u, 0u);
         }
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // before the MMA reads the cleared rows
@@ -337,16 +359,20 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     // ---- epilogue: O / sum -> out
     if (ok && pt_wait(pv_done, (unsigned)(n_tiles - 1) & 1u, failed, a.status)) {
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const float inv = 1.0f / l_run;
-      __nv_bfloat16* orow = a.out + (size_t)(start + row0 + r) * a.out_stride + (size_t)h * head_dim;
+      float inv = 1.0f / l_run;
+      if (a.sink) {  // 1 / (sum + 2^(sink - m)), also when the sink exceeds every score
+        const float sk = a.sink[h] * 1.4426950408889634f, top = fmaxf(m_ref, sk), down = exp2f(m_ref - top);
+        inv = down / (l_run * down + exp2f(sk - top));
+      }
+      __nv_bfloat16* orow = a.out + (size_t)(start + row0 + r) * a.out_stride + (size_t)h * a.v_dim;
 #pragma unroll
-      for (int c = 0; c < HD; c += 32) {
+      for (int c = 0; c < VD; c += 32) {
         float o[32];
         tmem_ld32(lane_addr + O_COL + c, o);
         if (r < rows_here) {
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
-            if (c + g * 8 < head_dim) {  // head sizes are multiples of 16: groups of 8 are whole
+            if (c + g * 8 < a.v_dim) {  // head sizes are multiples of 16: groups of 8 are whole
               uint4 w = make_uint4(pack_bf16x2(o[g * 8] * inv, o[g * 8 + 1] * inv), pack_bf16x2(o[g * 8 + 2] * inv, o[g * 8 + 3] * inv),
                                    pack_bf16x2(o[g * 8 + 4] * inv, o[g * 8 + 5] * inv), pack_bf16x2(o[g * 8 + 6] * inv, o[g * 8 + 7] * inv));
               *reinterpret_cast<uint4*>(orow + c + g * 8) = w;
@@ -391,20 +417,20 @@ extern "C" int bn_attention_prefill_tc_trace_read(unsigned long long* host) {
 }
 #endif
 
-template <int HD, int KS, int VS>
+template <int HD, int VD, int KS, int VS, bool PRECISE>
 static int launch_pt(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const PtArgs& a, int n_tiles,
                      cudaStream_t stream) {
-  size_t smem = (size_t)PT_ROWS * HD * 2 + (size_t)(KS + VS) * PT_KEYS * HD * 2 + (2 * KS + 2 * VS + 6) * 8 + 16;
+  size_t smem = (size_t)PT_ROWS * HD * 2 + (size_t)(KS * HD + VS * VD) * PT_KEYS * 2 + (2 * KS + 2 * VS + 6) * 8 + 16;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, KS, VS>,
+    cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, VD, KS, VS, PRECISE>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return BN_ERR_LAUNCH + (int)e;
     configured = true;
   }
   if (n_tiles > 65535) return BN_ERR_BAD_ARG;
   dim3 grid(a.n_heads, n_tiles);
-  BN_LAUNCH((attention_prefill_tc_kernel<HD, KS, VS>), grid, PT_THREADS, smem, stream, mq, mk, mv, a);
+  BN_LAUNCH((attention_prefill_tc_kernel<HD, VD, KS, VS, PRECISE>), grid, PT_THREADS, smem, stream, mq, mk, mv, a);
   return BN_OK;
 }
 
@@ -416,14 +442,16 @@ static int launch_pt(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
 // already hold the new tokens.  head_dim: a multiple of 16 up to 128.  status: one int on the
 // device, left as it is unless a wait inside the kernel gave up (then 5; nothing is stored by
 // that block).
-extern "C" int bn_attention_prefill_tc(const void* q, int q_stride, int n_tokens, void* out, int out_stride, int n_tiles,
-                                       int n_heads, int n_kv_heads, int head_dim, float scale, int window,
-                                       const int* tile_seq, const int* tile_row0, const int* seq_start,
-                                       const int* seq_pos0, const int* slots, const int* page_table, int pt_stride,
-                                       const void* k_cache, const void* v_cache, int n_cache_pages, int* status,
-                                       cudaStream_t stream) {
+// The values' cache is [n_cache_pages, n_kv_heads, 64, v_dim] with v_dim a multiple of 16 up to 128.  precise: the weights
+// enter the value product with 16 bits of mantissa.  sink: [n_heads] float32 scores that stand in the sums only, or null.
+extern "C" int bn_attention_prefill_tc_ex(const void* q, int q_stride, int n_tokens, void* out, int out_stride, int n_tiles,
+                                          int n_heads, int n_kv_heads, int head_dim, int v_dim, float scale, int window, int precise,
+                                          const float* sink, const int* tile_seq, const int* tile_row0, const int* seq_start,
+                                          const int* seq_pos0, const int* slots, const int* page_table, int pt_stride,
+                                          const void* k_cache, const void* v_cache, int n_cache_pages, int* status,
+                                          cudaStream_t stream) {
   if (n_tiles <= 0) return BN_OK;
-  if (head_dim <= 0 || head_dim % 16 || head_dim > 128 || n_kv_heads <= 0 || n_heads % n_kv_heads || window < 0 ||
+  if (head_dim <= 0 || head_dim % 16 || head_dim > 128 || v_dim <= 0 || v_dim % 16 || v_dim > 128 || !(scale > 0.f) || n_kv_heads <= 0 || n_heads % n_kv_heads || window < 0 ||
       n_heads > 65535 || (q_stride % 8) || (out_stride % 8) || n_tokens <= 0 || n_cache_pages <= 0 || !status ||
       (((uintptr_t)q | (uintptr_t)out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15))
     return BN_ERR_BAD_ARG;
@@ -431,11 +459,11 @@ extern "C" int bn_attention_prefill_tc(const void* q, int q_stride, int n_tokens
   if (!tma_map_bf16_strided(&mq, q, (unsigned long long)n_tokens, (unsigned long long)n_heads * head_dim,
                             (unsigned long long)q_stride, PT_ROWS) ||
       !tma_map_bf16_pages(&mk, k_cache, n_cache_pages, (unsigned long long)n_kv_heads * BN_PAGE, head_dim, BN_PAGE) ||
-      !tma_map_bf16_pages(&mv, v_cache, n_cache_pages, (unsigned long long)n_kv_heads * BN_PAGE, head_dim, BN_PAGE))
+      !tma_map_bf16_pages(&mv, v_cache, n_cache_pages, (unsigned long long)n_kv_heads * BN_PAGE, v_dim, BN_PAGE))
     return BN_ERR_BAD_ARG;
   PtArgs a = {};
   a.out = (__nv_bfloat16*)out; a.out_stride = out_stride; a.n_heads = n_heads; a.n_kv_heads = n_kv_heads;
-  a.head_dim = head_dim; a.scale_log2e = scale * 1.4426950408889634f; a.window = window; a.tile_seq = tile_seq;
+  a.head_dim = head_dim; a.v_dim = v_dim; a.sink = sink; a.scale_log2e = scale * 1.4426950408889634f; a.window = window; a.tile_seq = tile_seq;
   a.tile_row0 = tile_row0; a.seq_start = seq_start; a.seq_pos0 = seq_pos0; a.slots = slots; a.page_table = page_table;
   a.pt_stride = pt_stride; a.status = status;
   BN_TRACE_ONLY(a.trace = nullptr;)
@@ -443,6 +471,22 @@ extern "C" int bn_attention_prefill_tc(const void* q, int q_stride, int n_tokens
   // shared memory per block: 64 KB and 96 KB, so that two blocks share an SM (tensor memory
   // allows no more: 256 columns each) and one block's softmax overlaps the other's products
   // (a third key stage at head size 128 was measured and changes nothing: the softmax is the pace)
-  if (head_dim <= 64) return launch_pt<64, 3, 3>(mq, mk, mv, a, n_tiles, stream);
-  return launch_pt<128, 2, 2>(mq, mk, mv, a, n_tiles, stream);
+#define PT_RUN(HD, VD, KS, VS) \
+  return precise ? launch_pt<HD, VD, KS, VS, true>(mq, mk, mv, a, n_tiles, stream) : launch_pt<HD, VD, KS, VS, false>(mq, mk, mv, a, n_tiles, stream)
+  if (head_dim <= 64 && v_dim <= 64) PT_RUN(64, 64, 3, 3);
+  if (head_dim <= 64) PT_RUN(64, 128, 3, 2);
+  if (v_dim <= 64) PT_RUN(128, 64, 2, 3);
+  PT_RUN(128, 128, 2, 2);
+#undef PT_RUN
+}
+
+extern "C" int bn_attention_prefill_tc(const void* q, int q_stride, int n_tokens, void* out, int out_stride, int n_tiles,
+                                       int n_heads, int n_kv_heads, int head_dim, float scale, int window,
+                                       const int* tile_seq, const int* tile_row0, const int* seq_start,
+                                       const int* seq_pos0, const int* slots, const int* page_table, int pt_stride,
+                                       const void* k_cache, const void* v_cache, int n_cache_pages, int* status,
+                                       cudaStream_t stream) {
+  return bn_attention_prefill_tc_ex(q, q_stride, n_tokens, out, out_stride, n_tiles, n_heads, n_kv_heads, head_dim, head_dim, scale,
+                                    window, 0, nullptr, tile_seq, tile_row0, seq_start, seq_pos0, slots, page_table, pt_stride,
+                                    k_cache, v_cache, n_cache_pages, status, stream);
 }

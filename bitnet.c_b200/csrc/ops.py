@@ -742,10 +742,12 @@ USE_TCGEN05_ATTENTION = True  # prefill attention with head sizes up to 128 runs
 def attention_prefill_tc(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int,
                          scale: float, window: int, tile_seq: torch.Tensor, tile_row0: torch.Tensor,
                          seq_start: torch.Tensor, seq_pos0: torch.Tensor, slots: torch.Tensor, page_table: torch.Tensor,
-                         k_cache: torch.Tensor, v_cache: torch.Tensor) -> torch.Tensor:
+                         k_cache: torch.Tensor, v_cache: torch.Tensor, *, precise: bool = False,
+                         sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """bfloat16 causal attention of runs of new tokens on tcgen05 tensor cores with TMA-fed operands;
     block i handles up to 128 new tokens of sequence tile_seq[i] from its row tile_row0[i] on.
-    Head sizes up to 128."""
+    Key and value widths up to 128 (a value head has the width of ``v_cache``'s rows).  ``precise``: the softmax weights
+    enter the value product with 16 bits of mantissa instead of 8; ``sink`` as for ``attention_general``."""
     if not q.is_cuda or q.dim() != 2 or q.stride(-1) != 1 or q.stride(0) != q_stride or q.dtype != torch.bfloat16:
         raise KernelError("attention_prefill_tc: q must be a bfloat16 CUDA matrix with unit inner stride")
     _need(out, "out", torch.bfloat16, 2)
@@ -755,12 +757,25 @@ def attention_prefill_tc(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_he
     _need(page_table, "page_table", torch.int32, 2)
     _need(k_cache, "k_cache", torch.bfloat16, 4)
     _need(v_cache, "v_cache", torch.bfloat16, 4)
-    if tuple(k_cache.shape[1:]) != (n_kv_heads, PAGE, head_dim) or k_cache.shape != v_cache.shape:
-        raise KernelError(f"attention_prefill_tc: cache {tuple(k_cache.shape)} is not [pages, {n_kv_heads}, {PAGE}, {head_dim}]")
-    if head_dim % 16 or head_dim > 128 or n_heads % n_kv_heads:
-        raise KernelError(f"attention_prefill_tc: head_dim={head_dim}, heads {n_heads}/{n_kv_heads} not supported")
-    if out.shape[1] != n_heads * head_dim or q_stride % 8 or n_heads * head_dim > q_stride or out.shape[0] < q.shape[0]:
+    v_dim = v_cache.shape[3]
+    if tuple(k_cache.shape[1:]) != (n_kv_heads, PAGE, head_dim) or k_cache.shape[:3] != v_cache.shape[:3]:
+        raise KernelError(f"attention_prefill_tc: cache {tuple(k_cache.shape)} / {tuple(v_cache.shape)} is not "
+                          f"[pages, {n_kv_heads}, {PAGE}, {head_dim} / value width]")
+    if head_dim % 16 or head_dim > 128 or v_dim % 16 or v_dim > 128 or n_heads % n_kv_heads:
+        raise KernelError(f"attention_prefill_tc: head_dim={head_dim}, value width {v_dim}, heads {n_heads}/{n_kv_heads} not supported")
+    if sink is not None:
+        _need(sink, "sink", torch.float32, 1)
+        if sink.shape[0] != n_heads:
+            raise KernelError(f"attention_prefill_tc: {sink.shape[0]} sink scores for {n_heads} heads")
+    if out.shape[1] != n_heads * v_dim or q_stride % 8 or n_heads * head_dim > q_stride or out.shape[0] < q.shape[0]:
         raise KernelError("attention_prefill_tc: out or q_stride does not fit")
+    if precise or sink is not None or v_dim != head_dim:
+        _check(_fn("attention_prefill_tc", "bn_attention_prefill_tc_ex")(
+            _ptr(q), int(q_stride), int(q.shape[0]), _ptr(out), int(out.shape[1]), int(tile_seq.shape[0]), int(n_heads),
+            int(n_kv_heads), int(head_dim), int(v_dim), c_float(scale), int(window), int(bool(precise)), _ptr(sink), _ptr(tile_seq),
+            _ptr(tile_row0), _ptr(seq_start), _ptr(seq_pos0), _ptr(slots), _ptr(page_table), int(page_table.shape[1]), _ptr(k_cache),
+            _ptr(v_cache), int(k_cache.shape[0]), _ptr(tc_status(q.device)), _stream()), "attention_prefill_tc")
+        return out
     _check(_fn("attention_prefill_tc", "bn_attention_prefill_tc")(
         _ptr(q), int(q_stride), int(q.shape[0]), _ptr(out), int(out.shape[1]), int(tile_seq.shape[0]),
         int(n_heads), int(n_kv_heads), int(head_dim), c_float(scale), int(window), _ptr(tile_seq), _ptr(tile_row0),

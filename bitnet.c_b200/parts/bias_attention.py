@@ -36,7 +36,7 @@ class BiasAttention(Mixer):
     keys as projected, before the encoding (``values_are_keys``); a learned score per head that only enlarges the softmax's
     denominator (``sink``)."""
 
-    kernels = ("linear", "linear_mma", "linear_tc", "gemm_tc", "attention", "attention_prefill", "unit_norm", "rotary_pairs")
+    kernels = ("linear", "linear_mma", "linear_tc", "gemm_tc", "attention", "attention_prefill", "attention_prefill_tc", "unit_norm", "rotary_pairs")
     TILED_MIN_TOKENS = 16  # runs of new tokens from this many on take the tensor-core kernel (bfloat16)
     graph_safe = True
 
@@ -53,6 +53,10 @@ class BiasAttention(Mixer):
         self.position = build_part("position", spec.position, build) if spec.position is not None else None
         if self.position is not None and (spec.unit_norm or not hasattr(self.position, "apply")):
             raise ValueError("this mixer takes a position encoding that offers ``apply`` (rotary_pairs), and no unit norm with it")
+        # what the tcgen05 kernel for runs of tokens has no place for takes the mma.sync one
+        self.on_tcgen05 = (build.dtype == torch.bfloat16 and ops.USE_TCGEN05_ATTENTION and not spec.bias_buckets and not spec.head_gate
+                           and not spec.keep_first and not spec.chunk and spec.scale > 0
+                           and max(spec.head_dim, spec.v_head_dim) <= 128 and spec.head_dim % 16 == 0 and spec.v_head_dim % 16 == 0)
         self.w_in: Optional[torch.Tensor] = None
         self.w_o: Optional[torch.Tensor] = None
         self.rel: Optional[torch.Tensor] = None
@@ -153,10 +157,15 @@ class BiasAttention(Mixer):
         out = torch.empty((n, s.n_heads * s.v_head_dim), dtype=self.build.dtype, device=h.device)
         gate = proj[:, self.g_off:] if s.head_gate else None
         keep = s.keep_first if s.window > 0 else 0
-        if (self.build.dtype == torch.bfloat16 and not ctx.decode and ctx.tile_seq is not None and ctx.max_new >= self.TILED_MIN_TOKENS
+        if self.on_tcgen05 and not ctx.decode and ctx.wide_tile_seq is not None and ctx.max_new >= self.TILED_MIN_TOKENS:
+            # runs of new tokens on tcgen05: 128 tokens of a sequence and a head per block, the softmax weights with 16
+            # bits of mantissa
+            ops.attention_prefill_tc(proj, self.row, out, s.n_heads, s.n_kv_heads, s.head_dim, s.scale, s.window, ctx.wide_tile_seq,
+                                     ctx.wide_tile_row0, ctx.seq_start, ctx.seq_pos0, ctx.slots, kv.page_table, kv.k, kv.v,
+                                     precise=True, sink=self.sink)
+        elif (self.build.dtype == torch.bfloat16 and not ctx.decode and ctx.tile_seq is not None and ctx.max_new >= self.TILED_MIN_TOKENS
                 and s.v_head_dim % 16 == 0 and s.head_dim % 16 == 0):
-            # runs of new tokens: 64 tokens of a sequence and a head per block on the tensor cores, the
-            # softmax weights with 16 bits of mantissa
+            # the same on mma.sync, 64 tokens per block: with a bias, a gate, kept first tokens, chunks or wide heads
             ops.attention_prefill(proj, self.row, out, s.n_heads, s.n_kv_heads, s.head_dim, s.scale, s.window, ctx.tile_seq,
                                   ctx.tile_row0, ctx.seq_start, ctx.seq_pos0, ctx.slots, kv.page_table, kv.k, kv.v,
                                   keep_first=keep, rel=self.rel, gate=gate, gate_stride=self.row, precise=True, chunk=s.chunk,

@@ -359,6 +359,65 @@ def test_the_attention_mixer_finds_one_key_far_away(cuda_device, dtype, dims, he
                 cache.close(s)
 
 
+@pytest.mark.parametrize("H,G,d,dv,window", [(4, 2, 32, 16, 0), (8, 1, 128, 128, 0), (3, 3, 48, 80, 0), (16, 4, 64, 64, 70), (2, 1, 112, 32, 129), (6, 2, 16, 128, 1)])
+def test_runs_of_tokens_on_tcgen05_with_precise_weights_and_a_sink(cuda_device, H, G, d, dv, window):
+    """Whole prompts and pieces behind cached tokens in scattered pages: keys planted just inside and outside a window or at
+    the start, values that dwarf the rest, sinks that hold a good part of the weight or exceed every score by far; the
+    weights carry 16 bits of mantissa (with weights of 8 bits the result is visibly rougher)."""
+    from bitnet_c_b200.csrc import ops
+    rng = np.random.default_rng(H * d + window)
+    lens = [300, 70, 17]
+    T, scale, per = sum(lens), 1.0 / np.sqrt(d), H // G
+    q, k, v = (bf(rng.standard_normal((T, n, w))) for n, w in ((H, d), (G, d), (G, dv)))
+    last = lens[0] - 1
+    far = last - window + 1 if window else 0
+    k[far] = bf(q[last].reshape(G, per, d)[:, 0] * 2.0)
+    v[far] = bf(8.0 + 0.03 * rng.standard_normal((G, dv)))
+    if window:
+        k[far - 1], v[far - 1] = bf(q[last].reshape(G, per, d)[:, 0] * 4.0), 500.0  # must not be seen
+    starts = np.concatenate([[0], np.cumsum(lens)])
+    pages = [(n + 63) // 64 for n in lens]
+    order = rng.permutation(sum(pages) + 2)
+    table = np.zeros((4, max(pages)), dtype=np.int32)
+    kc = torch.full((sum(pages) + 2, G, 64, d), float("nan"), dtype=torch.bfloat16, device="cuda")
+    vc = torch.full((sum(pages) + 2, G, 64, dv), float("inf"), dtype=torch.bfloat16, device="cuda")
+    at = 0
+    for s, n in enumerate(lens):
+        table[s + 1, :pages[s]] = order[at:at + pages[s]]
+        at += pages[s]
+        for p in range(n):
+            kc[int(table[s + 1, p // 64]), :, p % 64] = dev(k[starts[s] + p], torch.bfloat16)
+            vc[int(table[s + 1, p // 64]), :, p % 64] = dev(v[starts[s] + p], torch.bfloat16)
+    table = torch.from_numpy(table).cuda()
+    for sink in (None, f32(rng.standard_normal(H) + 3), np.full(H, 200.0)):
+        want = np.zeros((T, H, dv))
+        for s, n in enumerate(lens):
+            i, j = np.arange(n)[:, None], np.arange(n)[None, :]
+            seen = (j <= i) & ((i - j < window) if window else True)
+            for h in range(H):
+                a = slice(starts[s], starts[s] + n)
+                sc = np.where(seen, q[a, h] @ k[a, h // per].T * scale, -np.inf)
+                want[a, h] = pr.softmax_with_sink(sc, -1e30 if sink is None else float(sink[h])) @ v[a, h // per]
+        want = want.reshape(T, H * dv)
+        for new in (lens, [150, 33, 16], [129, 2, 1]):
+            rows = np.concatenate([np.arange(starts[s] + lens[s] - c, starts[s] + lens[s]) for s, c in enumerate(new)])
+            tiles = [(s, r) for s, c in enumerate(new) for r in range(0, c, 128)]
+            qd = dev(q.reshape(T, -1)[rows], torch.bfloat16)
+            err = {}
+            for precise in (True, False):
+                out = torch.full((len(rows), H * dv), float("nan"), dtype=torch.bfloat16, device="cuda")
+                ops.attention_prefill_tc(qd, H * d, out, H, G, d, scale, window, ints(s for s, _ in tiles), ints(r for _, r in tiles),
+                                         ints(np.concatenate([[0], np.cumsum(new)])), ints(n - c for n, c in zip(lens, new)), ints([1, 2, 3]),
+                                         table, kc, vc, precise=precise, sink=dev(sink) if sink is not None else None)
+                got = out.float().cpu().numpy()
+                assert np.isfinite(got).all()
+                err[precise] = np.abs(got - want[rows])
+            # what is left is the rounding of the result itself
+            assert (err[True] <= 2.0 ** -8 * np.abs(want[rows]) + 2e-5 * (1 + np.abs(v).max(where=np.abs(v) < 100, initial=0))).all(), (sink, new)
+            assert err[True].sum() < err[False].sum() or window == 1 or (sink is not None and sink[0] == 200.0)
+    ops.check_tc_status(torch.device("cuda:0"))
+
+
 # ---- whole models --------------------------------------------------------------------------------------
 @pytest.fixture(scope="module")
 def folders(tmp_path_factory):
