@@ -283,6 +283,7 @@ __global__ void __launch_bounds__(GS_THREADS) gated_state_kernel(const GatedStat
 // exponent is at most zero.  The sums run in another order than token by token: the forms agree to rounding.
 #define GC_L 64
 #define GC_THREADS 256
+#define GC_CHAIN_THREADS 512
 #define GC_PLD 68  // padded rows of the chunk's 64 x 64 matrices
 
 __device__ __forceinline__ void gc_copy16(float* smem, const float* gmem, bool valid) {
@@ -293,12 +294,28 @@ __device__ __forceinline__ void gc_copy16(float* smem, const float* gmem, bool v
 __device__ __forceinline__ void gc_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void gc_wait() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
 
-// rows [row0, row0 + 64) of the matrix at src (row stride src_ld, `cols` numbers, a multiple of four), zeros past n_valid rows
-__device__ __forceinline__ void gc_load_rows(float* dst, int dst_ld, const float* src, size_t src_ld, int cols, int n_valid) {
-  const int per_row = cols >> 2;
-  for (int i = threadIdx.x; i < GC_L * per_row; i += GC_THREADS) {
-    const int r = i / per_row, c = (i - r * per_row) * 4;
-    gc_copy16(dst + r * dst_ld + c, src + (size_t)(r < n_valid ? r : 0) * src_ld + c, r < n_valid);
+// Which 16-byte pieces of 64 rows of `cols` numbers (a multiple of four) a thread copies: from (row, col) on, always
+// (d_row, d_col) further.
+struct CopyPlan {
+  int row, col, d_row, d_col, per_row;
+  __device__ __forceinline__ explicit CopyPlan(int cols) {
+    per_row = cols >> 2;
+    row = threadIdx.x / per_row;
+    col = threadIdx.x - row * per_row;
+    d_row = blockDim.x / per_row;
+    d_col = blockDim.x - d_row * per_row;
+  }
+};
+// 64 rows of the matrix at src (src_ld apart) to dst (dst_ld apart), zeros past n_valid rows
+__device__ __forceinline__ void gc_load_rows(const CopyPlan& p, float* dst, int dst_ld, const float* src, size_t src_ld, int n_valid) {
+  for (int r = p.row, c = p.col; r < GC_L;) {
+    gc_copy16(dst + r * dst_ld + c * 4, src + (size_t)(r < n_valid ? r : 0) * src_ld + c * 4, r < n_valid);
+    r += p.d_row;
+    c += p.d_col;
+    if (c >= p.per_row) {
+      c -= p.per_row;
+      ++r;
+    }
   }
 }
 
@@ -332,9 +349,10 @@ __global__ void __launch_bounds__(GC_THREADS) gated_state_local_kernel(const Gat
   const int s = tile_seq[blockIdx.x], row0 = tile_row0[blockIdx.x];
   const int first = a.seq_start[s] + row0, n_tok = min(GC_L, a.seq_start[s + 1] - first);
   const int n_qk = a.n_qk(), tid = threadIdx.x, lane = tid & 31;
-  gc_load_rows(sK, ld, kn + (size_t)first * n_qk + g * dim, n_qk, dim, n_tok);
+  const CopyPlan rows_dim(dim);
+  gc_load_rows(rows_dim, sK, ld, kn + (size_t)first * n_qk + g * dim, n_qk, n_tok);
   const bool with_qk = !DELTA || h % per_group == 0;
-  if (with_qk) gc_load_rows(sQ, ld, qn + (size_t)first * n_qk + g * dim, n_qk, dim, n_tok);
+  if (with_qk) gc_load_rows(rows_dim, sQ, ld, qn + (size_t)first * n_qk + g * dim, n_qk, n_tok);
   gc_commit();
   if (DELTA && tid < 32) {
     float l[2], b[2];
@@ -426,85 +444,261 @@ __device__ __forceinline__ void gc_write<4>(float* p, const float* o) { *reinter
 template <>
 __device__ __forceinline__ void gc_write<2>(float* p, const float* o) { *reinterpret_cast<float2*>(p) = make_float2(o[0], o[1]); }
 
-// acc[i][:] += M[row rg + 32 i][0 .. end) . U for the thread's TC columns; M's rows GC_PLD apart, end a multiple of four
-template <int NR, int TC>
-__device__ __forceinline__ void gc_product(float (*acc)[TC], const float* M, const float* U, int ct, int rg, int cg, int end) {
+// acc += row[0 .. end) . U, TC columns; U's rows u_ld apart, end a multiple of four
+template <int TC>
+__device__ __forceinline__ void gc_row_product(float* acc, const float* row, const float* U, int u_ld, int end) {
   for (int s = 0; s < end; s += 4) {
-    float4 m[NR];
-#pragma unroll
-    for (int i = 0; i < NR; ++i) m[i] = *reinterpret_cast<const float4*>(M + (rg + 32 * i) * GC_PLD + s);
+    const float4 m = *reinterpret_cast<const float4*>(row + s);
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       float u[TC];
-      gc_read<TC>(U + (s + e) * ct + cg * TC, u);
+      gc_read<TC>(U + (s + e) * u_ld, u);
+      const float f = e == 0 ? m.x : e == 1 ? m.y : e == 2 ? m.z : m.w;
 #pragma unroll
-      for (int i = 0; i < NR; ++i) {
-        const float f = e == 0 ? m[i].x : e == 1 ? m[i].y : e == 2 ? m[i].z : m[i].w;
+      for (int c = 0; c < TC; ++c) acc[c] = fmaf(f, u[c], acc[c]);
+    }
+  }
+}
+
+// Floats of shared memory of the chain's block; the operands that lie token by token (or state row by state row) have rows
+// of CT + 8 numbers, which keeps the tensor cores' fragment reads free of bank conflicts.
+static size_t gc_smem_floats(bool delta, int dim, int ct, int stages) {
+  const int sld = ct + 8;
+  return (size_t)stages * 2 * GC_L * (dim + 4) + (size_t)dim * sld + 2 * GC_L * sld + (size_t)stages * GC_L * GC_PLD +
+         (delta ? GC_L * GC_PLD : dim * sld) + 4 * GC_L;
+}
+
+__device__ __forceinline__ void gc_named_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+__device__ __forceinline__ void gc_named_arrive(int id, int threads) { asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+
+// Single-precision products on the tensor cores: every operand as the sum of two TF32 numbers (22 bits together), three
+// products, float32 sums.  The warp's tile is 16 rows x 8 NT columns; lane = 4 g + q holds the rows g and g + 8.
+__device__ __forceinline__ void gc_split(float x, unsigned& hi, unsigned& lo) {
+  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(hi) : "f"(x));
+  lo = __float_as_uint(x - __uint_as_float(hi));
+}
+__device__ __forceinline__ void gc_mma(float* c, const unsigned* a, const unsigned* b) {
+  asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+}
+// acc += A B over k < k_end (a multiple of eight): A's element (row, k) at A[row * a_row + k * a_k], B's (k, column) at
+// B[k * b_row + column]; both pointers already at the tile's first row and column.
+template <int NT>
+__device__ __forceinline__ void gc_tile_product(float* acc, const float* A, int a_row, int a_k, const float* B, int b_row, int k_end, int lane) {
+  const int g = lane >> 2, q = lane & 3;
+#pragma unroll 2
+  for (int k = 0; k < k_end; k += 8) {
+    unsigned ah[4], al[4];
+    const float* p = A + (size_t)g * a_row + (size_t)(k + q) * a_k;
+    gc_split(p[0], ah[0], al[0]);
+    gc_split(p[8 * a_row], ah[1], al[1]);
+    gc_split(p[4 * a_k], ah[2], al[2]);
+    gc_split(p[8 * a_row + 4 * a_k], ah[3], al[3]);
 #pragma unroll
-        for (int c = 0; c < TC; ++c) acc[i][c] = fmaf(f, u[c], acc[i][c]);
+    for (int j = 0; j < NT; ++j) {
+      unsigned bh[2], bl[2];
+      const float* r = B + (size_t)(k + q) * b_row + 8 * j + g;
+      gc_split(r[0], bh[0], bl[0]);
+      gc_split(r[4 * b_row], bh[1], bl[1]);
+      gc_mma(acc + 4 * j, al, bh);
+      gc_mma(acc + 4 * j, ah, bl);
+      gc_mma(acc + 4 * j, ah, bh);
+    }
+  }
+}
+
+// Where element e of a thread's CT / 4 results lies in the chunk's [64][CT] matrices (e and e + 1, e even, are neighbours).
+template <int CT, bool MMA>
+__device__ __forceinline__ int2 gc_place(int t256, int e) {
+  if (MMA) {
+    const int warp = t256 >> 5, lane = t256 & 31;
+    return make_int2((warp >> 1) * 16 + (lane >> 2) + (e & 2 ? 8 : 0), (warp & 1) * (CT / 2) + (e >> 2) * 8 + (lane & 3) * 2 + (e & 1));
+  }
+  return make_int2((t256 >> 3) + 32 * (e / (CT / 8)), (t256 & 7) * (CT / 8) + e % (CT / 8));
+}
+
+// o = X S for the thread's elements: X [64][ld], S [dim][sld]
+template <int CT, bool MMA>
+__device__ __forceinline__ void gc_state_product(float* o, const float* X, int ld, const float* S, int dim, int t256) {
+  constexpr int SLD = CT + 8, TC = CT / 8;
+#pragma unroll
+  for (int e = 0; e < CT / 4; ++e) o[e] = 0.f;
+  if (MMA) {
+    const int warp = t256 >> 5;
+    gc_tile_product<CT / 16>(o, X + (size_t)(warp >> 1) * 16 * ld, ld, 1, S + (warp & 1) * (CT / 2), SLD, dim, t256 & 31);
+    return;
+  }
+  const int rg = t256 >> 3, cg = t256 & 7;
+#pragma unroll 2
+  for (int d = 0; d < dim; d += 4) {
+    float4 x[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) x[i] = *reinterpret_cast<const float4*>(X + (rg + 32 * i) * ld + d);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float sv[TC];
+      gc_read<TC>(S + (d + e) * SLD + cg * TC, sv);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const float f = e == 0 ? x[i].x : e == 1 ? x[i].y : e == 2 ? x[i].z : x[i].w;
+#pragma unroll
+        for (int c = 0; c < TC; ++c) o[i * TC + c] = fmaf(f, sv[c], o[i * TC + c]);
       }
     }
   }
 }
 
-static size_t gc_smem_floats(int dim, int ct, int stages) {
-  return (size_t)stages * 2 * GC_L * (dim + 4) + (size_t)dim * ct + 3 * GC_L * ct + (size_t)stages * GC_L * GC_PLD + GC_L * GC_PLD + 4 * GC_L;
+// o += M U for the thread's elements: M [64][GC_PLD] lower triangular, U [64][sld]
+template <int CT, bool MMA>
+__device__ __forceinline__ void gc_chunk_product(float* o, const float* M, const float* U, int t256) {
+  constexpr int SLD = CT + 8, TC = CT / 8;
+  const int warp = t256 >> 5;
+  if (MMA) {
+    gc_tile_product<CT / 16>(o, M + (warp >> 1) * 16 * GC_PLD, GC_PLD, 1, U + (warp & 1) * (CT / 2), SLD, (warp >> 1) * 16 + 16, t256 & 31);
+    return;
+  }
+  const int rg = t256 >> 3, cg = t256 & 7;
+  const int end = warp * 4 + 36;  // the warp's rows are 4 w .. 4 w + 3 and those + 32
+  for (int s = 0; s < end; s += 4) {
+    float4 m[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) m[i] = *reinterpret_cast<const float4*>(M + (rg + 32 * i) * GC_PLD + s);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float u[TC];
+      gc_read<TC>(U + (s + e) * SLD + cg * TC, u);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const float f = e == 0 ? m[i].x : e == 1 ? m[i].y : e == 2 ? m[i].z : m[i].w;
+#pragma unroll
+        for (int c = 0; c < TC; ++c) o[i * TC + c] = fmaf(f, u[c], o[i * TC + c]);
+      }
+    }
+  }
 }
 
-// The chain: one block per (sequence, head, CT value columns).  Thread = (tokens rg and rg + 32, TC columns); in the
-// state's update (four rows of the state, TC columns).  With two stages the next chunk's rows arrive while this one's are
-// worked on.
-template <typename T, bool DELTA, int CT>
-__global__ void __launch_bounds__(GC_THREADS) gated_state_chunk_kernel(const GatedStateArgs a, const float* __restrict__ qn,
-                                                                       const float* __restrict__ kn, const float* __restrict__ vc,
-                                                                       const float* __restrict__ lb, const float* __restrict__ qk,
-                                                                       const float* __restrict__ winv, int col_tiles, int stages,
-                                                                       float* __restrict__ out) {
+// to = carry * from + K^T D by eight warps: K [64][ld], D [64][sld], to and from [dim][sld] (they may be one)
+template <int CT, bool MMA>
+__device__ __forceinline__ void gc_advance_state(float* to, const float* from, float carry, const float* K, int ld, const float* D, int dim,
+                                                 int t256) {
+  constexpr int SLD = CT + 8, TC = CT / 8;
+  if (MMA) {
+    const int lane = t256 & 31, g = lane >> 2, q = lane & 3;
+    for (int d0 = (t256 >> 5) * 16; d0 < dim; d0 += 128) {
+      float acc[CT / 2];
+#pragma unroll
+      for (int e = 0; e < CT / 2; ++e) acc[e] = 0.f;
+      gc_tile_product<CT / 8>(acc, K + d0, 1, ld, D, SLD, GC_L, lane);
+#pragma unroll
+      for (int e = 0; e < CT / 2; e += 2) {
+        const int d = d0 + g + (e & 2 ? 8 : 0), at = d * SLD + (e >> 2) * 8 + 2 * q;
+        if (d < dim) {
+          float old[2];
+          gc_read<2>(from + at, old);
+          old[0] = fmaf(carry, old[0], acc[e]);
+          old[1] = fmaf(carry, old[1], acc[e + 1]);
+          gc_write<2>(to + at, old);
+        }
+      }
+    }
+    return;
+  }
+  const int rg = t256 >> 3, cg = t256 & 7;
+  for (int d = rg * 4; d < dim; d += 128) {
+    float acc[4][TC];
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+#pragma unroll
+      for (int c = 0; c < TC; ++c) acc[e][c] = 0.f;
+#pragma unroll 4
+    for (int t = 0; t < GC_L; ++t) {
+      const float4 k = *reinterpret_cast<const float4*>(K + t * ld + d);
+      float u[TC];
+      gc_read<TC>(D + t * SLD + cg * TC, u);
+#pragma unroll
+      for (int c = 0; c < TC; ++c) {
+        acc[0][c] = fmaf(k.x, u[c], acc[0][c]);
+        acc[1][c] = fmaf(k.y, u[c], acc[1][c]);
+        acc[2][c] = fmaf(k.z, u[c], acc[2][c]);
+        acc[3][c] = fmaf(k.w, u[c], acc[3][c]);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float old[TC];
+      gc_read<TC>(from + (d + e) * SLD + cg * TC, old);
+#pragma unroll
+      for (int c = 0; c < TC; ++c) old[c] = fmaf(carry, old[c], acc[e][c]);
+      gc_write<TC>(to + (d + e) * SLD + cg * TC, old);
+    }
+  }
+}
+
+// The chain: one block per (sequence, head, CT value columns), two halves of eight warps.  A thread of either half has CT / 4
+// elements of the chunk's [64][CT] matrices (gc_place).  The second half makes the outputs, Q S0 and P U; the first
+// advances the state, in the delta rule after it has made the right-hand sides V - e^c K S0 and both halves have
+// multiplied them into U.  Without a delta rule the halves meet once per chunk: the state goes into a buffer of its own while
+// the other half still reads the old one.  With two stages the next chunk's rows arrive while this one's are worked on.
+// MMA: the products on the tensor cores (dim a multiple of eight), else on the CUDA cores.
+template <typename T, bool DELTA, int CT, bool MMA>
+__global__ void __launch_bounds__(GC_CHAIN_THREADS) gated_state_chunk_kernel(const GatedStateArgs a, const float* __restrict__ qn,
+                                                                             const float* __restrict__ kn, const float* __restrict__ vc,
+                                                                             const float* __restrict__ lb, const float* __restrict__ qk,
+                                                                             const float* __restrict__ winv, int col_tiles, int stages,
+                                                                             float* __restrict__ out) {
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int TC = CT / 8;
-  constexpr int NR = DELTA ? 4 : 2;  // rows of [K; Q] S0 per thread: K rows rg, rg + 32 (delta), then Q rows
+  constexpr int TC = CT / 8, NE = CT / 4, SLD = CT + 8;
   extern __shared__ __align__(16) float sm[];
   const int heads = a.heads, dim = a.dim, vdim = a.vdim, ld = dim + 4, n_qk = a.n_qk();
   float* sKQ = sm;                                        // [stages][K 64 rows | Q 64 rows][ld]
-  float* sS = sKQ + (size_t)stages * 2 * GC_L * ld;       // [dim][CT]
-  float* sR = sS + (size_t)dim * CT;                      // [64][CT] right-hand sides
-  float* sU = sR + GC_L * CT;                             // [64][CT] u
-  float* sD = sU + GC_L * CT;                             // [64][CT] u times its weight in the state after the chunk
-  float* sP = sD + GC_L * CT;                             // [stages][64][GC_PLD]
-  float* sW = sP + (size_t)stages * GC_L * GC_PLD;        // [64][GC_PLD]
-  float* sc = sW + GC_L * GC_PLD;                         // [64] c, then b, e^c, e^(c_end - c)
+  float* sS = sKQ + (size_t)stages * 2 * GC_L * ld;       // [dim][SLD]
+  float* sU = sS + (size_t)dim * SLD;                     // [64][SLD] u
+  float* sD = sU + GC_L * SLD;                            // [64][SLD] right-hand sides; u times its weight in the state after the chunk
+  float* sP = sD + GC_L * SLD;                            // [stages][64][GC_PLD]
+  float* sW = sP + (size_t)stages * GC_L * GC_PLD;        // delta: [64][GC_PLD]
+  float* sS2 = sW;                                        // otherwise: [dim][SLD], the state after the chunk
+  float* sc = sW + (DELTA ? GC_L * GC_PLD : dim * SLD);   // [64] c, then b, e^c, e^(c_end - c)
   float *sb = sc + GC_L, *se = sb + GC_L, *sd = se + GC_L;
   const int tile = blockIdx.x % col_tiles, h = (blockIdx.x / col_tiles) % heads, s = blockIdx.x / (col_tiles * heads);
   const int per_group = heads / a.groups, g = h / per_group;
-  const int tid = threadIdx.x, lane = tid & 31, rg = tid >> 3, cg = tid & 7;
-  const int col0 = tile * CT, col = col0 + cg * TC;
+  const int tid = threadIdx.x, t256 = tid & 255, lane = tid & 31;
+  const bool outputs = tid >= 256;  // the second half
+  const int col0 = tile * CT;
   const int start = a.seq_start[s], n = a.seq_start[s + 1] - start;
   float* S_g = a.state + (size_t)a.slots[s] * a.state_stride + (size_t)h * dim * vdim;
-  for (int i = tid; i < dim * CT; i += GC_THREADS) {
-    const int d = i / CT, c = col0 + i - d * CT;
-    sS[i] = c < vdim ? S_g[(size_t)d * vdim + c] : 0.f;
+  for (int i = tid; i < dim * CT; i += GC_CHAIN_THREADS) {
+    const int d = i / CT, c = i - d * CT;
+    sS[d * SLD + c] = col0 + c < vdim ? S_g[(size_t)d * vdim + col0 + c] : 0.f;
   }
   const float skip = a.d ? a.d[h] : 0.f;
+  const CopyPlan rows_dim(dim), rows_64(GC_L);
   auto load_kq = [&](int base, int stage) {
     float* dst = sKQ + (size_t)stage * 2 * GC_L * ld;
     const int left = min(GC_L, n - base);
-    gc_load_rows(dst, ld, kn + (size_t)(start + base) * n_qk + g * dim, n_qk, dim, left);
-    gc_load_rows(dst + GC_L * ld, ld, qn + (size_t)(start + base) * n_qk + g * dim, n_qk, dim, left);
-    gc_load_rows(sP + (size_t)stage * GC_L * GC_PLD, GC_PLD, qk + ((size_t)(start + base) * a.groups + g) * GC_L, (size_t)a.groups * GC_L,
-                 GC_L, left);
+    gc_load_rows(rows_dim, dst, ld, kn + (size_t)(start + base) * n_qk + g * dim, n_qk, left);
+    gc_load_rows(rows_dim, dst + GC_L * ld, ld, qn + (size_t)(start + base) * n_qk + g * dim, n_qk, left);
+    gc_load_rows(rows_64, sP + (size_t)stage * GC_L * GC_PLD, GC_PLD, qk + ((size_t)(start + base) * a.groups + g) * GC_L,
+                 (size_t)a.groups * GC_L, left);
   };
   auto load_w = [&](int base) {
-    gc_load_rows(sW, GC_PLD, winv + ((size_t)(start + base) * heads + h) * GC_L, (size_t)heads * GC_L, GC_L, min(GC_L, n - base));
+    gc_load_rows(rows_64, sW, GC_PLD, winv + ((size_t)(start + base) * heads + h) * GC_L, (size_t)heads * GC_L, min(GC_L, n - base));
   };
-  float v_next[2][TC], l_next[2] = {0.f, 0.f}, b_next[2] = {0.f, 0.f};
+  const bool pairs = vdim % 2 == 0 && (((uintptr_t)vc | (uintptr_t)out) & 7) == 0;
+  float v_next[NE], l_next[2] = {0.f, 0.f}, b_next[2] = {0.f, 0.f};
   auto load_v = [&](int base) {
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int t = base + rg + 32 * i;
-#pragma unroll
-      for (int c = 0; c < TC; ++c)
-        v_next[i][c] = t < n && col + c < vdim ? vc[(size_t)(start + t) * heads * vdim + (size_t)h * vdim + col + c] : 0.f;
+    for (int e = 0; e < NE; e += 2) {
+      const int2 at = gc_place<CT, MMA>(t256, e);
+      const int t = base + at.x, col = col0 + at.y;
+      const float* p = vc + (size_t)(start + t) * heads * vdim + (size_t)h * vdim + col;
+      if (pairs && t < n && col < vdim) {
+        gc_read<2>(p, v_next + e);
+      } else {
+        v_next[e] = t < n && col < vdim ? p[0] : 0.f;
+        v_next[e + 1] = t < n && col + 1 < vdim ? p[1] : 0.f;
+      }
     }
     if (tid < 32) {
 #pragma unroll
@@ -534,11 +728,9 @@ __global__ void __launch_bounds__(GC_THREADS) gated_state_chunk_kernel(const Gat
       se[2 * lane] = expf(c.x); se[2 * lane + 1] = expf(c.y);
       sd[2 * lane] = expf(end - c.x); sd[2 * lane + 1] = expf(end - c.y);
     }
-    float v[2][TC];
+    float v[NE];
 #pragma unroll
-    for (int i = 0; i < 2; ++i)
-#pragma unroll
-      for (int c = 0; c < TC; ++c) v[i][c] = v_next[i][c];
+    for (int e = 0; e < NE; ++e) v[e] = v_next[e];
     gc_wait();
     __syncthreads();
     const bool more = base + GC_L < n;
@@ -551,121 +743,99 @@ __global__ void __launch_bounds__(GC_THREADS) gated_state_chunk_kernel(const Gat
     }
     const float* K = sKQ + (size_t)stage * 2 * GC_L * ld;
     float* P = sP + (size_t)stage * GC_L * GC_PLD;
-    // the decays onto q . k (above the diagonal the first kernel left zeros)
-    for (int i = tid; i < GC_L * GC_L; i += GC_THREADS) {
-      const int t = i >> 6, u = i & 63;
-      if (u <= t) P[t * GC_PLD + u] *= expf(sc[t] - sc[u]);
-    }
-    float acc[NR][TC];
-#pragma unroll
-    for (int i = 0; i < NR; ++i)
-#pragma unroll
-      for (int c = 0; c < TC; ++c) acc[i][c] = 0.f;
-    const float* X = DELTA ? K : K + GC_L * ld;
-    for (int d = 0; d < dim; d += 4) {
-      float4 x[NR];
-#pragma unroll
-      for (int i = 0; i < NR; ++i) x[i] = *reinterpret_cast<const float4*>(X + (rg + 32 * i) * ld + d);
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        float sv[TC];
-        gc_read<TC>(sS + (d + e) * CT + cg * TC, sv);
-#pragma unroll
-        for (int i = 0; i < NR; ++i) {
-          const float f = e == 0 ? x[i].x : e == 1 ? x[i].y : e == 2 ? x[i].z : x[i].w;
-#pragma unroll
-          for (int c = 0; c < TC; ++c) acc[i][c] = fmaf(f, sv[c], acc[i][c]);
-        }
+    float o[NE];
+    if (outputs) {
+      // the decays onto q . k (above the diagonal the first kernel left zeros), then Q S0
+      for (int i = t256; i < GC_L * GC_L; i += 256) {
+        const int t = i >> 6, u = i & 63;
+        if (u <= t) P[t * GC_PLD + u] *= expf(sc[t] - sc[u]);
       }
-    }
-    float o[2][TC];
+      gc_state_product<CT, MMA>(o, K + GC_L * ld, ld, sS, dim, t256);
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int t = rg + 32 * i;
-      float r[TC];
+      for (int e = 0; e < NE; ++e) o[e] *= se[gc_place<CT, MMA>(t256, e).x];
+    } else if (DELTA) {
+      gc_state_product<CT, MMA>(o, K, ld, sS, dim, t256);
 #pragma unroll
-      for (int c = 0; c < TC; ++c) {
-        o[i][c] = acc[NR - 2 + i][c] * se[t];
-        r[c] = DELTA ? v[i][c] - acc[i][c] * se[t] : v[i][c] * sb[t];
+      for (int e = 0; e < NE; e += 2) {
+        const int2 at = gc_place<CT, MMA>(t256, e);
+        const float r[2] = {v[e] - o[e] * se[at.x], v[e + 1] - o[e + 1] * se[at.x]};
+        gc_write<2>(sD + at.x * SLD + at.y, r);
       }
-      if (DELTA) {
-        gc_write<TC>(sR + t * CT + cg * TC, r);
-      } else {
-        gc_write<TC>(sU + t * CT + cg * TC, r);
+    } else {
 #pragma unroll
-        for (int c = 0; c < TC; ++c) r[c] *= sd[t];
-        gc_write<TC>(sD + t * CT + cg * TC, r);
+      for (int e = 0; e < NE; e += 2) {
+        const int2 at = gc_place<CT, MMA>(t256, e);
+        const float u[2] = {v[e] * sb[at.x], v[e + 1] * sb[at.x]}, w[2] = {u[0] * sd[at.x], u[1] * sd[at.x]};
+        gc_write<2>(sU + at.x * SLD + at.y, u);
+        gc_write<2>(sD + at.x * SLD + at.y, w);
       }
+      gc_named_arrive(2, GC_CHAIN_THREADS);  // the other half may read u
+      gc_named_sync(1, 256);
+      gc_advance_state<CT, MMA>(sS2, sS, se[GC_L - 1], K, ld, sD, dim, t256);
     }
-    __syncthreads();
-    // a warp's tokens are 4 w .. 4 w + 3 and those + 32: sums over the chunk's earlier tokens end behind the later ones
-    const int last = (tid >> 5) * 4 + 36;
     if (DELTA) {
-      float u[2][TC];
+      __syncthreads();
+      // U = W R over both halves: a tile of 16 x 8 per warp, or a token and TC columns per thread
+      constexpr int UE = MMA ? 4 : TC;
+      const int warp = tid >> 5;
+      const bool has_u = !MMA || (warp & 3) * 8 < CT;
+      float u[UE];
 #pragma unroll
-      for (int i = 0; i < 2; ++i)
+      for (int e = 0; e < UE; ++e) u[e] = 0.f;
+      if (MMA) {
+        if (has_u)
+          gc_tile_product<1>(u, sW + (warp >> 2) * 16 * GC_PLD, GC_PLD, 1, sD + (warp & 3) * 8, SLD, (warp >> 2) * 16 + 16, lane);
+      } else {
+        gc_row_product<TC>(u, sW + (tid >> 3) * GC_PLD, sD + (tid & 7) * TC, SLD, (warp + 1) * 4);
+      }
+      __syncthreads();  // the right-hand sides have been read
+      if (has_u) {
 #pragma unroll
-        for (int c = 0; c < TC; ++c) u[i][c] = 0.f;
-      gc_product<2, TC>(u, sW, sR, CT, rg, cg, last);
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = rg + 32 * i;
-        gc_write<TC>(sU + t * CT + cg * TC, u[i]);
-#pragma unroll
-        for (int c = 0; c < TC; ++c) u[i][c] *= sd[t];
-        gc_write<TC>(sD + t * CT + cg * TC, u[i]);
+        for (int e = 0; e < UE; e += 2) {
+          const int t = MMA ? (warp >> 2) * 16 + (lane >> 2) + (e & 2 ? 8 : 0) : tid >> 3;
+          const int at = t * SLD + (MMA ? (warp & 3) * 8 + (lane & 3) * 2 : (tid & 7) * TC + e);
+          const float w[2] = {u[e] * sd[t], u[e + 1] * sd[t]};
+          gc_write<2>(sU + at, u + e);
+          gc_write<2>(sD + at, w);
+        }
       }
       __syncthreads();
       if (more) {
         load_w(base + GC_L);
         gc_commit();
       }
+      if (!outputs) gc_advance_state<CT, MMA>(sS, sS, se[GC_L - 1], K, ld, sD, dim, t256);
+    } else if (outputs) {
+      gc_named_sync(2, GC_CHAIN_THREADS);  // u, and this half's decays
     }
-    gc_product<2, TC>(o, P, sU, CT, rg, cg, last);
+    if (outputs) {
+      gc_chunk_product<CT, MMA>(o, P, sU, t256);
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int t = base + rg + 32 * i;
-      if (t < n) {
-        float* dst = out + (size_t)(start + t) * heads * vdim + (size_t)h * vdim + col;
-#pragma unroll
-        for (int c = 0; c < TC; ++c)
-          if (col + c < vdim) dst[c] = fmaf(skip, v[i][c], o[i][c]);
-      }
-    }
-    const float carry = se[GC_L - 1];
-    for (int d = rg * 4; d < dim; d += 128) {
-      float n4[4][TC];
-#pragma unroll
-      for (int e = 0; e < 4; ++e)
-#pragma unroll
-        for (int c = 0; c < TC; ++c) n4[e][c] = 0.f;
-#pragma unroll 4
-      for (int t = 0; t < GC_L; ++t) {
-        const float4 k = *reinterpret_cast<const float4*>(K + t * ld + d);
-        float u[TC];
-        gc_read<TC>(sD + t * CT + cg * TC, u);
-#pragma unroll
-        for (int c = 0; c < TC; ++c) {
-          n4[0][c] = fmaf(k.x, u[c], n4[0][c]);
-          n4[1][c] = fmaf(k.y, u[c], n4[1][c]);
-          n4[2][c] = fmaf(k.z, u[c], n4[2][c]);
-          n4[3][c] = fmaf(k.w, u[c], n4[3][c]);
+      for (int e = 0; e < NE; e += 2) {
+        const int2 at = gc_place<CT, MMA>(t256, e);
+        const int t = base + at.x, col = col0 + at.y;
+        if (t < n && col < vdim) {
+          float* dst = out + (size_t)(start + t) * heads * vdim + (size_t)h * vdim + col;
+          const float y[2] = {fmaf(skip, v[e], o[e]), fmaf(skip, v[e + 1], o[e + 1])};
+          if (pairs) {
+            gc_write<2>(dst, y);
+          } else {
+            dst[0] = y[0];
+            if (col + 1 < vdim) dst[1] = y[1];
+          }
         }
       }
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        float old[TC];
-        gc_read<TC>(sS + (d + e) * CT + cg * TC, old);
-#pragma unroll
-        for (int c = 0; c < TC; ++c) old[c] = fmaf(carry, old[c], n4[e][c]);
-        gc_write<TC>(sS + (d + e) * CT + cg * TC, old);
-      }
+    }
+    if (!DELTA) {
+      float* swap = sS;
+      sS = sS2;
+      sS2 = swap;
     }
   }
   __syncthreads();
-  for (int i = tid; i < dim * CT; i += GC_THREADS) {
-    const int d = i / CT, c = col0 + i - d * CT;
-    if (c < vdim) S_g[(size_t)d * vdim + c] = sS[i];
+  for (int i = tid; i < dim * CT; i += GC_CHAIN_THREADS) {
+    const int d = i / CT, c = i - d * CT;
+    if (col0 + c < vdim) S_g[(size_t)d * vdim + col0 + c] = sS[d * SLD + c];
   }
   gs_keep_inputs<T>(a, s, h, col0, min(CT, vdim - col0), tile == 0 && h % per_group == 0);
 }
@@ -883,31 +1053,35 @@ extern "C" int bn_gated_state_chunks(GS_PARAMS, const float* qn, const float* kn
     BN_LAUNCH(gated_state_local_kernel<true>, dim3(n_tiles, heads), GC_THREADS, local, stream, a, qn, kn, lb, tile_seq, tile_row0, qk, winv);
   else
     BN_LAUNCH(gated_state_local_kernel<false>, dim3(n_tiles, groups), GC_THREADS, local, stream, a, qn, kn, lb, tile_seq, tile_row0, qk, winv);
-  // 32 columns per block, or 16 where that leaves most of the SMs without one
-  const int ct = (long long)n_seqs * heads * ((vdim + 31) / 32) >= 100 || vdim <= 8 ? 32 : 16;
+  // 32 columns per block, or 16 where that leaves most of the SMs without one (or a block's memory too small)
+  const size_t most = 227 * 1024;  // shared memory of a block
+  const bool fits32 = gc_smem_floats(delta, dim, 32, 1) * sizeof(float) <= most;
+  const int ct = fits32 && (long long)n_seqs * heads * ((vdim + 31) / 32) >= 60 ? 32 : 16;
   const int col_tiles = (vdim + ct - 1) / ct;
-  const int stages = gc_smem_floats(dim, ct, 2) * sizeof(float) <= 227 * 1024 ? 2 : 1;
-  const size_t smem = gc_smem_floats(dim, ct, stages) * sizeof(float);
+  const int stages = gc_smem_floats(delta, dim, ct, 2) * sizeof(float) <= most ? 2 : 1;
+  const size_t smem = gc_smem_floats(delta, dim, ct, stages) * sizeof(float);
   const long long blocks = (long long)n_seqs * heads * col_tiles;
-  if (smem > 227 * 1024 || blocks > 2147483647LL) return BN_ERR_BAD_ARG;
-#define GC_RUN(TT, DD, CC)                                                                                                               \
+  if (smem > most || blocks > 2147483647LL) return BN_ERR_BAD_ARG;
+#define GC_RUN(TT, DD, CC, MM)                                                                                                           \
   do {                                                                                                                                   \
     static size_t granted = 0;                                                                                                           \
     if (smem > granted) {                                                                                                                \
-      cudaError_t e = cudaFuncSetAttribute(gated_state_chunk_kernel<TT, DD, CC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      cudaError_t e = cudaFuncSetAttribute(gated_state_chunk_kernel<TT, DD, CC, MM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
       if (e != cudaSuccess) return BN_ERR_LAUNCH + (int)e;                                                                               \
       granted = smem;                                                                                                                    \
     }                                                                                                                                    \
-    BN_LAUNCH((gated_state_chunk_kernel<TT, DD, CC>), (unsigned)blocks, GC_THREADS, smem, stream, a, qn, kn, vc, lb, qk, winv, col_tiles, \
-              stages, out);                                                                                                              \
+    BN_LAUNCH((gated_state_chunk_kernel<TT, DD, CC, MM>), (unsigned)blocks, GC_CHAIN_THREADS, smem, stream, a, qn, kn, vc, lb, qk, winv, \
+              col_tiles, stages, out);                                                                                                   \
   } while (0)
-#define GC_RUN_T(TT)                                                                       \
-  do {                                                                                     \
-    if (delta) { if (ct == 32) GC_RUN(TT, true, 32); else GC_RUN(TT, true, 16); }          \
-    else { if (ct == 32) GC_RUN(TT, false, 32); else GC_RUN(TT, false, 16); }              \
+#define GC_RUN_T(TT, MM)                                                                           \
+  do {                                                                                             \
+    if (delta) { if (ct == 32) GC_RUN(TT, true, 32, MM); else GC_RUN(TT, true, 16, MM); }          \
+    else { if (ct == 32) GC_RUN(TT, false, 32, MM); else GC_RUN(TT, false, 16, MM); }              \
   } while (0)
-  if (dtype == BN_F32) GC_RUN_T(float);
-  else if (dtype == BN_BF16) GC_RUN_T(__nv_bfloat16);
+  // the float32 path keeps to the CUDA cores
+  if (dtype == BN_F32) GC_RUN_T(float, false);
+  else if (dtype == BN_BF16 && dim % 8 == 0) GC_RUN_T(__nv_bfloat16, true);
+  else if (dtype == BN_BF16) GC_RUN_T(__nv_bfloat16, false);
   else return BN_ERR_BAD_ARG;
 #undef GC_RUN_T
 #undef GC_RUN

@@ -267,49 +267,90 @@ extern "C" int bn_streams_norm(float* x, int n_rows, int width, int streams, con
 }
 
 // Runs of tokens: out[t] = h[t] + sum_j taps[j] h[t - n_taps + 1 + j] over the rows of each sequence, inputs before the
-// step from its slot's history, which then receives the last n_taps - 1 inputs.  A thread takes V columns of one row;
-// the thread of a sequence's first row also takes the n_taps - 2 rows behind it, which read the history too, and
-// replaces the history: nobody else touches those columns of it.
+// step from its slot's history, which then receives the last n_taps - 1 inputs.  The first n_taps - 1 rows of a sequence
+// read the history: the thread that owns a column group of the first row takes all of these rows, one after another, and
+// then replaces the history, so nobody else touches those columns of it.
 template <typename T, int V>
-__global__ void input_convolution_kernel(const T* __restrict__ h, T* __restrict__ out, int width, int n_tokens,
-                                         const float* __restrict__ taps, int n_taps, T* hist, size_t hist_stride,
-                                         const int* __restrict__ tok_seq, const int* __restrict__ seq_start,
-                                         const int* __restrict__ slots) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int dtype = sizeof(T) == 4 ? BN_F32 : BN_BF16;
-  const int per_row = width / V;
-  const size_t item = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-  const int t = (int)(item / per_row);
-  if (t >= n_tokens) return;
-  const int c = (int)(item - (size_t)t * per_row) * V;
-  const int s = tok_seq[t], start = seq_start[s], r = t - start;
-  const int back = n_taps - 1;
-  if (r > 0 && r < back) return;  // the first row's thread does these
-  T* hs = hist ? hist + (size_t)slots[s] * hist_stride + c : nullptr;
-  const int n = seq_start[s + 1] - start;
-  const int todo = r == 0 ? max(1, min(n, back)) : 1;
-  for (int i = 0; i < todo; ++i) {
+__device__ __forceinline__ void convolve_first_rows(const T* h, T* out, int width, const float* taps, int n_taps, T* hs, int start, int n,
+                                                    int c) {
+  const int dtype = sizeof(T) == 4 ? BN_F32 : BN_BF16, back = n_taps - 1;
+  for (int i = 0; i < min(n, back); ++i) {
     float acc[V], v[V], w[V];
-    load_v<V>(h, dtype, (size_t)(t + i) * width + c, acc);
+    load_v<V>(h, dtype, (size_t)(start + i) * width + c, acc);
     for (int j = 0; j <= back; ++j) {
-      const int src = r + i - back + j;  // place among the sequence's new rows
+      const int src = i - back + j;  // place among the sequence's new rows
       if (src >= 0) load_v<V>(h, dtype, (size_t)(start + src) * width + c, v);
       else load_v<V>(hs, dtype, (size_t)(back + src) * width, v);
       load_v<V>(taps, BN_F32, (size_t)j * width + c, w);
 #pragma unroll
       for (int e = 0; e < V; ++e) acc[e] = fmaf(w[e], v[e], acc[e]);
     }
-    store_v<V>(out, dtype, (size_t)(t + i) * width + c, acc);
+    store_v<V>(out, dtype, (size_t)(start + i) * width + c, acc);
   }
-  if (r == 0) {
-    for (int j = 0; j < back; ++j) {  // rising j: what is still needed lies ahead of what is overwritten
-      float v[V];
-      const int src = j + n;
-      if (src < back) load_v<V>(hs, dtype, (size_t)src * width, v);
-      else load_v<V>(h, dtype, (size_t)(start + src - back) * width + c, v);
-      store_v<V>(hs, dtype, (size_t)j * width, v);
+  for (int j = 0; j < back; ++j) {  // rising j: what is still needed lies ahead of what is overwritten
+    float v[V];
+    const int src = j + n;
+    if (src < back) load_v<V>(hs, dtype, (size_t)src * width, v);
+    else load_v<V>(h, dtype, (size_t)(start + src - back) * width + c, v);
+    store_v<V>(hs, dtype, (size_t)j * width, v);
+  }
+}
+
+// A thread takes V columns of R neighbouring packed rows; with N taps fixed the rows it looks at are read once and wait
+// in registers (N 0: any number of taps, every input is read where it is needed).  Grid (column groups, row groups).
+template <typename T, int V, int N, int R>
+__global__ void __launch_bounds__(128) input_convolution_kernel(const T* __restrict__ h, T* __restrict__ out, int width, int n_tokens,
+                                                                const float* __restrict__ taps, int n_taps, T* hist, size_t hist_stride,
+                                                                const int* __restrict__ tok_seq, const int* __restrict__ seq_start,
+                                                                const int* __restrict__ slots) {
+  pdl_launch_dependents();
+  const int dtype = sizeof(T) == 4 ? BN_F32 : BN_BF16;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V, t0 = blockIdx.y * R;
+  if (c >= width) return;
+  const int back = (N ? N : n_taps) - 1;
+  float w[N ? N : 1][V];
+  if (N) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) load_v<V>(taps, BN_F32, (size_t)j * width + c, w[j]);
+  }
+  pdl_wait();
+  float x[N ? R + N - 1 : 1][V];
+  if (N) {
+#pragma unroll
+    for (int i = 0; i < R + N - 1; ++i) {
+      const int t = t0 + i - (N - 1);
+      if (t >= 0 && t < n_tokens) load_v<V>(h, dtype, (size_t)t * width + c, x[i]);
     }
+  }
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int t = t0 + i;
+    if (t >= n_tokens) return;
+    const int s = tok_seq[t], start = seq_start[s], r = t - start;
+    if (r < back) {
+      if (r == 0)
+        convolve_first_rows<T, V>(h, out, width, taps, back + 1, hist + (size_t)slots[s] * hist_stride + c, start, seq_start[s + 1] - start, c);
+      continue;
+    }
+    float acc[V];
+    if (N) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] = x[i + N - 1][e];
+#pragma unroll
+      for (int j = 0; j < N; ++j)
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc[e] = fmaf(w[j][e], x[i + j][e], acc[e]);
+    } else {
+      load_v<V>(h, dtype, (size_t)t * width + c, acc);
+      for (int j = 0; j <= back; ++j) {
+        float v[V], tw[V];
+        load_v<V>(h, dtype, (size_t)(t - back + j) * width + c, v);
+        load_v<V>(taps, BN_F32, (size_t)j * width + c, tw);
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc[e] = fmaf(tw[e], v[e], acc[e]);
+      }
+    }
+    store_v<V>(out, dtype, (size_t)t * width + c, acc);
   }
 }
 
@@ -320,20 +361,25 @@ extern "C" int bn_input_convolution(const void* h, void* out, int dtype, int n_t
   if (!h || !out || h == out || !taps || width <= 0 || n_taps < 1 || n_taps > ST_MAX_TAPS || !tok_seq || !seq_start || !slots ||
       (n_taps > 1 && !hist))
     return BN_ERR_BAD_ARG;
-  if (n_taps == 1) hist = nullptr;
   const bool vec = width % 8 == 0 && hist_stride % 8 == 0 && !(((uintptr_t)h | (uintptr_t)out | (uintptr_t)taps | (uintptr_t)hist) & 15);
-  const size_t items = (size_t)n_tokens * (vec ? width / 4 : width);
-  const unsigned blocks = (unsigned)((items + 255) / 256);
-#define ST_CONV(TT, VV)                                                                                                        \
-  BN_LAUNCH((input_convolution_kernel<TT, VV>), blocks, 256, 0, stream, (const TT*)h, (TT*)out, width, n_tokens, taps, n_taps, \
-            (TT*)hist, (size_t)hist_stride, tok_seq, seq_start, slots)
-  if (dtype == BN_F32) {
-    if (vec) ST_CONV(float, 4); else ST_CONV(float, 1);
-  } else if (dtype == BN_BF16) {
-    if (vec) ST_CONV(__nv_bfloat16, 4); else ST_CONV(__nv_bfloat16, 1);
-  } else {
-    return BN_ERR_BAD_ARG;
-  }
+#define ST_CONV(TT, VV, NN, RR)                                                                                                  \
+  do {                                                                                                                           \
+    if ((n_tokens + RR - 1) / RR > 65535) return BN_ERR_BAD_ARG;                                                                 \
+    BN_LAUNCH((input_convolution_kernel<TT, VV, NN, RR>), dim3((width / VV + 127) / 128, (n_tokens + RR - 1) / RR), 128, 0, stream, \
+              (const TT*)h, (TT*)out, width, n_tokens, taps, n_taps, (TT*)hist, (size_t)hist_stride, tok_seq, seq_start, slots); \
+  } while (0)
+#define ST_CONV_T(TT)                                   \
+  do {                                                  \
+    if (!vec) ST_CONV(TT, 1, 0, 4);                     \
+    else if (n_taps == 2) ST_CONV(TT, 4, 2, 4);         \
+    else if (n_taps == 3) ST_CONV(TT, 4, 3, 4);         \
+    else if (n_taps == 4) ST_CONV(TT, 4, 4, 4);         \
+    else ST_CONV(TT, 4, 0, 4);                          \
+  } while (0)
+  if (dtype == BN_F32) ST_CONV_T(float);
+  else if (dtype == BN_BF16) ST_CONV_T(__nv_bfloat16);
+  else return BN_ERR_BAD_ARG;
+#undef ST_CONV_T
 #undef ST_CONV
   return BN_OK;
 }
