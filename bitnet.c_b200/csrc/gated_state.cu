@@ -471,10 +471,11 @@ static size_t gc_smem_floats(bool delta, int dim, int ct, int stages) {
 __device__ __forceinline__ void gc_named_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 __device__ __forceinline__ void gc_named_arrive(int id, int threads) { asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 
-// Single-precision products on the tensor cores: every operand as the sum of two TF32 numbers (22 bits together), three
-// products, float32 sums.  The warp's tile is 16 rows x 8 NT columns; lane = 4 g + q holds the rows g and g + 8.
+// Single-precision products on the tensor cores: every operand as the sum of two TF32 numbers (its first 11 bits and the
+// next 11), three products, float32 sums.  The warp's tile is 16 rows x 8 NT columns; lane = 4 g + q holds the rows g and
+// g + 8.
 __device__ __forceinline__ void gc_split(float x, unsigned& hi, unsigned& lo) {
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(hi) : "f"(x));
+  hi = __float_as_uint(x) & 0xffffe000u;
   lo = __float_as_uint(x - __uint_as_float(hi));
 }
 __device__ __forceinline__ void gc_mma(float* c, const unsigned* a, const unsigned* b) {
@@ -482,30 +483,40 @@ __device__ __forceinline__ void gc_mma(float* c, const unsigned* a, const unsign
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
 }
-// acc += A B over k < k_end (a multiple of eight): A's element (row, k) at A[row * a_row + k * a_k], B's (k, column) at
-// B[k * b_row + column]; both pointers already at the tile's first row and column.
-template <int NT>
-__device__ __forceinline__ void gc_tile_product(float* acc, const float* A, int a_row, int a_k, const float* B, int b_row, int k_end, int lane) {
+// acc += A B over k < k_end (a multiple of eight), pointers at the tile's first row and column: A's element (row, k) at
+// A[row * a_ld + k], with A_BY_K at A[k * a_ld + row]; B's (k, column) at B[k * SLD + column].
+template <int NT, int SLD, bool A_BY_K>
+__device__ __forceinline__ void gc_tile_product(float* acc, const float* A, int a_ld, const float* B, int k_end, int lane) {
   const int g = lane >> 2, q = lane & 3;
+  const float* p0 = A + (A_BY_K ? q * a_ld + g : g * a_ld + q);
+  const float* p1 = p0 + (A_BY_K ? 4 * a_ld : 8 * a_ld);
+  const float* r = B + q * SLD + g;
+  const int step = A_BY_K ? 8 * a_ld : 8;
 #pragma unroll 2
   for (int k = 0; k < k_end; k += 8) {
     unsigned ah[4], al[4];
-    const float* p = A + (size_t)g * a_row + (size_t)(k + q) * a_k;
-    gc_split(p[0], ah[0], al[0]);
-    gc_split(p[8 * a_row], ah[1], al[1]);
-    gc_split(p[4 * a_k], ah[2], al[2]);
-    gc_split(p[8 * a_row + 4 * a_k], ah[3], al[3]);
+    gc_split(p0[0], ah[0], al[0]);
+    gc_split(A_BY_K ? p0[8] : p1[0], ah[1], al[1]);
+    gc_split(A_BY_K ? p1[0] : p0[4], ah[2], al[2]);
+    gc_split(A_BY_K ? p1[8] : p1[4], ah[3], al[3]);
+    p0 += step;
+    p1 += step;
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
       unsigned bh[2], bl[2];
-      const float* r = B + (size_t)(k + q) * b_row + 8 * j + g;
-      gc_split(r[0], bh[0], bl[0]);
-      gc_split(r[4 * b_row], bh[1], bl[1]);
+      gc_split(r[8 * j], bh[0], bl[0]);
+      gc_split(r[8 * j + 4 * SLD], bh[1], bl[1]);
       gc_mma(acc + 4 * j, al, bh);
       gc_mma(acc + 4 * j, ah, bl);
       gc_mma(acc + 4 * j, ah, bh);
     }
+    r += 8 * SLD;
   }
+}
+__device__ __forceinline__ float gc_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 
 // Where element e of a thread's CT / 4 results lies in the chunk's [64][CT] matrices (e and e + 1, e even, are neighbours).
@@ -526,7 +537,7 @@ __device__ __forceinline__ void gc_state_product(float* o, const float* X, int l
   for (int e = 0; e < CT / 4; ++e) o[e] = 0.f;
   if (MMA) {
     const int warp = t256 >> 5;
-    gc_tile_product<CT / 16>(o, X + (size_t)(warp >> 1) * 16 * ld, ld, 1, S + (warp & 1) * (CT / 2), SLD, dim, t256 & 31);
+    gc_tile_product<CT / 16, SLD, false>(o, X + (warp >> 1) * 16 * ld, ld, S + (warp & 1) * (CT / 2), dim, t256 & 31);
     return;
   }
   const int rg = t256 >> 3, cg = t256 & 7;
@@ -555,7 +566,7 @@ __device__ __forceinline__ void gc_chunk_product(float* o, const float* M, const
   constexpr int SLD = CT + 8, TC = CT / 8;
   const int warp = t256 >> 5;
   if (MMA) {
-    gc_tile_product<CT / 16>(o, M + (warp >> 1) * 16 * GC_PLD, GC_PLD, 1, U + (warp & 1) * (CT / 2), SLD, (warp >> 1) * 16 + 16, t256 & 31);
+    gc_tile_product<CT / 16, SLD, false>(o, M + (warp >> 1) * 16 * GC_PLD, GC_PLD, U + (warp & 1) * (CT / 2), (warp >> 1) * 16 + 16, t256 & 31);
     return;
   }
   const int rg = t256 >> 3, cg = t256 & 7;
@@ -589,7 +600,7 @@ __device__ __forceinline__ void gc_advance_state(float* to, const float* from, f
       float acc[CT / 2];
 #pragma unroll
       for (int e = 0; e < CT / 2; ++e) acc[e] = 0.f;
-      gc_tile_product<CT / 8>(acc, K + d0, 1, ld, D, SLD, GC_L, lane);
+      gc_tile_product<CT / 8, SLD, true>(acc, K + d0, ld, D, GC_L, lane);
 #pragma unroll
       for (int e = 0; e < CT / 2; e += 2) {
         const int d = d0 + g + (e & 2 ? 8 : 0), at = d * SLD + (e >> 2) * 8 + 2 * q;
@@ -746,9 +757,20 @@ __global__ void __launch_bounds__(GC_CHAIN_THREADS) gated_state_chunk_kernel(con
     float o[NE];
     if (outputs) {
       // the decays onto q . k (above the diagonal the first kernel left zeros), then Q S0
-      for (int i = t256; i < GC_L * GC_L; i += 256) {
-        const int t = i >> 6, u = i & 63;
-        if (u <= t) P[t * GC_PLD + u] *= expf(sc[t] - sc[u]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int t = (t256 >> 4) + 16 * j, u = (t256 & 15) * 4;
+        if (u <= t) {
+          float p[4], c[4];
+          gc_read<4>(P + t * GC_PLD + u, p);
+          gc_read<4>(sc + u, c);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float x = fminf(sc[t] - c[e], 0.f);  // above the diagonal p is zero
+            p[e] *= MMA ? gc_ex2(x * 1.4426950408889634f) : expf(x);
+          }
+          gc_write<4>(P + t * GC_PLD + u, p);
+        }
       }
       gc_state_product<CT, MMA>(o, K + GC_L * ld, ld, sS, dim, t256);
 #pragma unroll
@@ -784,7 +806,7 @@ __global__ void __launch_bounds__(GC_CHAIN_THREADS) gated_state_chunk_kernel(con
       for (int e = 0; e < UE; ++e) u[e] = 0.f;
       if (MMA) {
         if (has_u)
-          gc_tile_product<1>(u, sW + (warp >> 2) * 16 * GC_PLD, GC_PLD, 1, sD + (warp & 3) * 8, SLD, (warp >> 2) * 16 + 16, lane);
+          gc_tile_product<1, SLD, false>(u, sW + (warp >> 2) * 16 * GC_PLD, GC_PLD, sD + (warp & 3) * 8, (warp >> 2) * 16 + 16, lane);
       } else {
         gc_row_product<TC>(u, sW + (tid >> 3) * GC_PLD, sD + (tid & 7) * TC, SLD, (warp + 1) * 4);
       }
