@@ -357,6 +357,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       BN_TRACE_ONLY(if (tr) a.trace[j * 12 + 5] = global_timer();)
     }
     // ---- epilogue: O / sum -> out
+    // A warp may be here while the others still owe their share of P for the page before the last: the last scores were
+    // issued ahead of that page's product.  pv_done is asked for both pages in turn, since its parity alone would not tell
+    // the last page from the one two before it.
+    if (ok && n_tiles > 1) ok = pt_wait(pv_done, (unsigned)n_tiles & 1u, failed, a.status);
     if (ok && pt_wait(pv_done, (unsigned)(n_tiles - 1) & 1u, failed, a.status)) {
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       float inv = 1.0f / l_run;

@@ -418,6 +418,32 @@ def test_runs_of_tokens_on_tcgen05_with_precise_weights_and_a_sink(cuda_device, 
     ops.check_tc_status(torch.device("cuda:0"))
 
 
+@pytest.mark.parametrize("d", [64, 128])
+def test_every_row_of_long_runs_holds_its_last_page(cuda_device, d):
+    """A thousand tokens and some, several heads, scores of every temper (warps of a block then run through their rows at
+    unequal speeds): the tcgen05 kernel against the general one, row by row."""
+    from bitnet_c_b200.csrc import ops
+    for seed, n in enumerate((1122, 439, 640, 65, 129, 1000, 770, 1500)):
+        H, G = 8, 4
+        g = torch.Generator(device="cuda").manual_seed(seed)
+        q = (torch.randn((n, H * d), device="cuda", generator=g) * (1 + 3 * (seed % 3))).bfloat16()
+        pages = (n + 63) // 64
+        k = torch.randn((pages, G, 64, d), device="cuda", generator=g).bfloat16()
+        v = torch.randn((pages, G, 64, d), device="cuda", generator=g).bfloat16()
+        table = torch.randperm(pages, device="cuda", generator=g).int().view(1, pages)
+        sink = torch.randn(H, device="cuda", generator=g) * 2 + 3
+        out, ref = (torch.full((n, H * d), float("nan"), dtype=torch.bfloat16, device="cuda") for _ in range(2))
+        zero, pos = ints([0]), torch.arange(n, dtype=torch.int32, device="cuda")
+        ops.attention_general(q, H * d, ref, n, H, G, d, d ** -0.5, 0, torch.zeros_like(pos), pos, zero, table, k, v, sink=sink)
+        tiles = list(range(0, n, 128))
+        for precise in (True, False):
+            for _ in range(4):
+                ops.attention_prefill_tc(q, H * d, out, H, G, d, d ** -0.5, 0, ints([0] * len(tiles)), ints(tiles), ints([0, n]), zero, zero, table,
+                                         k, v, precise=precise, sink=sink)
+                err = (out.float() - ref.float()).abs().amax(1)
+                assert float(err.max()) < 0.05 * float(ref.float().abs().max()), f"{n} tokens, precise {precise}: row {int(err.argmax())}"
+
+
 # ---- whole models --------------------------------------------------------------------------------------
 @pytest.fixture(scope="module")
 def folders(tmp_path_factory):
