@@ -1078,7 +1078,7 @@ extern "C" int bn_gated_state_chunks(GS_PARAMS, const float* qn, const float* kn
   // 32 columns per block, or 16 where that leaves most of the SMs without one (or a block's memory too small)
   const size_t most = 227 * 1024;  // shared memory of a block
   const bool fits32 = gc_smem_floats(delta, dim, 32, 1) * sizeof(float) <= most;
-  const int ct = fits32 && (long long)n_seqs * heads * ((vdim + 31) / 32) >= 60 ? 32 : 16;
+  const int ct = fits32 && (long long)n_seqs * heads * ((vdim + 31) / 32) >= 100 ? 32 : 16;
   const int col_tiles = (vdim + ct - 1) / ct;
   const int stages = gc_smem_floats(delta, dim, ct, 2) * sizeof(float) <= most ? 2 : 1;
   const size_t smem = gc_smem_floats(delta, dim, ct, stages) * sizeof(float);
