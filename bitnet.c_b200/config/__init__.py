@@ -4,6 +4,7 @@ from .spec import (DeltaRuleSpec, LatentAttentionSpec, ParallelBlockSpec, Rotary
 from .spec import (LimitedMlpSpec, SigmoidAttentionSpec)  # noqa: F401
 from .spec import (NormedAttentionSpec, RotaryBlendSpec, SandwichBlockSpec)  # noqa: F401
 from .spec import (HeadDeltaSpec, LayerNormSpec, Mamba2Spec, PolyMlpSpec, StreamsBlockSpec)  # noqa: F401
+from .spec import (GatedLinearSpec, LightningSpec, PairSpec)  # noqa: F401
 from .spec import (AttentionSpec, BlockSpec, ConfigError, GatedMlpSpec, LinearHeadSpec, ModelSpec, NoPositionSpec,
                    RmsNormSpec, RotarySpec, ScheduleEntry)
 from .registry import (Architecture, architecture, architecture_of, known_architectures,
@@ -83,7 +84,20 @@ register_architecture(Architecture(
     config_to_dict=RudolixConfig.to_dict,
 ))
 
+from . import lakadra as _lakadra
+from .lakadra import LakadraConfig
+
+register_architecture(Architecture(
+    name=_lakadra.ARCHITECTURE,
+    read_config=LakadraConfig.from_dict,
+    to_spec=LakadraConfig.to_spec,
+    tensor_name=_lakadra.tensor_name,
+    cap_positions=LakadraConfig.with_max_positions,
+    config_to_dict=LakadraConfig.to_dict,
+))
+
 __all__ = [
+    "LakadraConfig", "GatedLinearSpec", "LightningSpec", "PairSpec",
     "RudolixConfig", "HeadDeltaSpec", "LayerNormSpec", "Mamba2Spec", "PolyMlpSpec", "StreamsBlockSpec",
     "NetanexConfig", "NormedAttentionSpec", "RotaryBlendSpec", "SandwichBlockSpec",
     "AttentionSpec", "BlockSpec", "ConfigError", "GatedMlpSpec", "LinearHeadSpec", "ModelSpec", "NoPositionSpec",

@@ -82,6 +82,7 @@ class RotaryBlendSpec:
     slow: float = 1.0
     magnitude_slope: float = 0.1
     pairing: str = "halves"
+    slowdown: float = 1.0  # every frequency is divided by this (linear scaling), with or without the ramp
     kind: str = "rotary_blend"
 
 
@@ -143,6 +144,9 @@ class BiasAttentionSpec:
     position: Any = None  # a position spec whose encoding q and k get (after the unit norm, if any); None: none
     values_are_keys: bool = False  # no value projection: the values are the keys as projected, before any encoding
     sink: bool = False  # a learned score per head in the softmax's denominator, without a key or a value
+    zero_sink: bool = False  # the same with a score of 0 for every head: one is added to the denominator
+    proj_bias: bool = False  # biases on the query, key and value projections
+    out_bias: bool = False  # a bias on the output projection
     kind: str = "bias_attention"
 
 
@@ -215,7 +219,8 @@ class LatentAttentionSpec:
     (``v_head_dim``) come, and one rotated key part of ``rot_dim`` numbers that all heads share.  Only the latent
     and the rotated part are cached.  ``window``: the last so many keys (0: all); a logistic gate per head
     (``head_gate``) or per output number (``element_gate``); ``sink``: a learned score per head in the softmax's
-    denominator, without a key or a value."""
+    denominator, without a key or a value.  A run without a latent of its own (``own_kv`` False) reads another run's rows
+    with its own queries, keys and values made from them, and output."""
 
     width: int
     n_heads: int
@@ -231,6 +236,7 @@ class LatentAttentionSpec:
     head_gate: bool = True
     element_gate: bool = False
     sink: bool = False
+    own_kv: bool = True  # False: no latent of its own; the run reads the rows another run cached
     kind: str = "latent_attention"
 
 
@@ -287,6 +293,43 @@ class Mamba2Spec:
 
 
 @dataclass(frozen=True)
+class LightningSpec:
+    """Linear attention with one fixed decay per head: SiLU on queries, keys and values, S <- ``decay`` S + k v^T, o = S^T q;
+    the heads' outputs RMS-normed together with a gain, times the logistic function of a projection of the mixer's input."""
+
+    width: int
+    n_heads: int
+    head_dim: int
+    v_head_dim: int
+    decay: Tuple[float, ...]
+    norm_eps: float
+    kind: str = "lightning"
+
+
+@dataclass(frozen=True)
+class GatedLinearSpec:
+    """A real-gated linear recurrence per channel behind a short convolution, beside a GELU branch: ``inner`` channels, the
+    gates' matrices block-diagonal in ``parts`` equal parts."""
+
+    width: int
+    inner: int
+    parts: int
+    conv_taps: int
+    kind: str = "gated_linear"
+
+
+@dataclass(frozen=True)
+class PairSpec:
+    """Two mixers side by side on the same input: ``left_scale`` left(h) + ``right_scale`` right(h)."""
+
+    left: Any
+    right: Any
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+    kind: str = "pair"
+
+
+@dataclass(frozen=True)
 class MlstmSpec:
     """mLSTM: a matrix memory per head with exponential gating, a soft cap on the gates' pre-activations,
     a unit norm per head, a gain over all heads and a logistic output gate."""
@@ -320,8 +363,15 @@ class MoeSpec:
     table_rows: int = 0
     weight_scale: float = 1.0  # factor on the (renormalised) weights
     renormalise_eps: float = 0.0  # added to the sum the weights are divided by
-    activation: str = "limited"  # "limited": the clamped unit above; "silu" / "gelu_tanh": act(g) * u, no clamps
+    # "limited": the clamped unit above; "silu" / "gelu_tanh": act(g) * u, no clamps; "relu2": no gate, max(u, 0)^2
+    activation: str = "limited"
     router_bias: bool = False  # a learned number per expert added to the router's logits before the choice
+    # the choice goes by score + a learned correction per expert; the weights are the scores without it
+    correction: bool = False
+    groups: int = 1  # with a correction: the experts form so many equal groups of neighbours ...
+    keep_groups: int = 1  # ... and are chosen among those of the so many groups whose best choice score is largest
+    identity: int = 0  # the router's last so many outputs are experts whose output is the input itself
+    shared_gate: bool = False  # the shared expert's output times the logistic function of one number per token
     kind: str = "moe"
 
 

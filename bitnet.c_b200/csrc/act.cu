@@ -357,3 +357,34 @@ extern "C" int bn_poly_norm(const void* z, int z_dtype, const float* coef, float
 #undef BN_POLY
   return BN_ERR_BAD_ARG;
 }
+
+// The unit without a gate: the square of relu, number by number (x and out may be one).  16-byte pieces, then what is left.
+template <typename T>
+__global__ void relu_squared_kernel(const T* x, T* out, size_t n) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int V = 16 / (int)sizeof(T);
+  const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (i + V <= n) {
+    uint4 raw = *reinterpret_cast<const uint4*>(x + i);
+    T* v = reinterpret_cast<T*>(&raw);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = from_f32<T>(relu_squared(to_f32<T>(v[e])));
+    *reinterpret_cast<uint4*>(out + i) = raw;
+  } else {
+    for (size_t j = i; j < n; ++j) out[j] = from_f32<T>(relu_squared(to_f32<T>(x[j])));
+  }
+}
+
+// x, out: n numbers of one type, 16-byte aligned.
+extern "C" int bn_relu_squared(const void* x, void* out, int dtype, long long n, cudaStream_t stream) {
+  if (n <= 0) return BN_OK;
+  if (!x || !out || (((uintptr_t)x | (uintptr_t)out) & 15)) return BN_ERR_BAD_ARG;
+  const int v = dtype == BN_F32 ? 4 : 8;
+  const unsigned blocks = (unsigned)(((size_t)n + 256 * v - 1) / (256 * v));
+  if (dtype == BN_F32) BN_LAUNCH(relu_squared_kernel<float>, blocks, 256, 0, stream, (const float*)x, (float*)out, (size_t)n);
+  else if (dtype == BN_BF16)
+    BN_LAUNCH(relu_squared_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (const __nv_bfloat16*)x, (__nv_bfloat16*)out, (size_t)n);
+  else return BN_ERR_BAD_ARG;
+  return BN_OK;
+}

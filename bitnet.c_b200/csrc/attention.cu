@@ -59,6 +59,7 @@ __device__ __forceinline__ void store_result(T* out, int out_wide, size_t at, fl
 //   rel, n_rel   additive bias by distance, rel[min(pos - p, n_rel - 1) * n_heads + h] (float32; the
 //                scale does not multiply it)
 //   gate         per token and head a number whose logistic function multiplies the head's output
+//   out_scale    a factor on all of the output (1: none)
 //   chunk        positions are cut into chunks of this many and a token sees the earlier keys of its own
 //                chunk only (takes the place of the window)
 //   v_row        width of a row of the value plane when it is more than v_dim: the values are the first
@@ -77,7 +78,7 @@ __global__ void attention_general_kernel(const T* __restrict__ q, int q_stride, 
                                          const int* __restrict__ tok_pos, const int* __restrict__ slots,
                                          const int* __restrict__ page_table, int pt_stride,
                                          const T* __restrict__ k_cache, const T* __restrict__ v_cache,
-                                         float* __restrict__ part, int n_splits, const float* __restrict__ sink, int v_share, int out_wide) {
+                                         float* __restrict__ part, int n_splits, const float* __restrict__ sink, int v_share, int out_wide, float out_scale) {
   pdl_launch_dependents();  // the next kernel in the stream may begin its prologue
   pdl_wait();               // the kernels before this one have completed and their writes are visible
   extern __shared__ __align__(16) float sm[];
@@ -184,6 +185,7 @@ __global__ void attention_general_kernel(const T* __restrict__ q, int q_stride, 
   }
   float inv = sink && !part ? sink_inverse(m_run, l_run, sink[h]) : 1.0f / l_run;
   if (gate) inv *= 1.0f / (1.0f + expf(-to_f32<T>(gate[(size_t)t * gate_stride + h])));
+  inv *= out_scale;
   const size_t orow = (size_t)t * out_stride + (size_t)h * v_dim;
   float* prow = part ? part + (((size_t)t * n_heads + h) * n_splits + blockIdx.z) * (v_dim + 2) : nullptr;
   if (prow && threadIdx.x == 0) { prow[0] = m_run; prow[1] = l_run; }
@@ -245,7 +247,7 @@ attention_grouped_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
                          const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, const int* __restrict__ slots,
                          const int* __restrict__ page_table, int pt_stride, const T* __restrict__ k_cache,
                          const T* __restrict__ v_cache, float* __restrict__ part, int n_splits,
-                         const float* __restrict__ sink, int v_share, int out_wide) {
+                         const float* __restrict__ sink, int v_share, int out_wide, float out_scale) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
@@ -371,6 +373,7 @@ attention_grouped_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
     const int h = h0 + r;
     float inv = sink && !part ? sink_inverse(m_run[r], l_run[r], sink[h]) : 1.0f / l_run[r];
     if (gate) inv *= 1.0f / (1.0f + expf(-to_f32<T>(gate[(size_t)t * gate_stride + h])));
+    inv *= out_scale;
     const size_t orow = (size_t)t * out_stride + (size_t)h * v_dim;
     float* prow = part ? part + (((size_t)t * n_heads + h) * n_splits + blockIdx.z) * (v_dim + 2) : nullptr;
     if (prow && threadIdx.x == 0) { prow[0] = m_run[r]; prow[1] = l_run[r]; }
@@ -387,7 +390,7 @@ attention_grouped_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
 template <typename T>
 __global__ void attention_merge_kernel(const float* __restrict__ part, int n_splits, int n_heads, int v_dim,
                                        const T* __restrict__ gate, int gate_stride, T* __restrict__ out, int out_stride,
-                                       const float* __restrict__ sink, int out_wide) {
+                                       const float* __restrict__ sink, int out_wide, float out_scale) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y;
@@ -401,6 +404,7 @@ __global__ void attention_merge_kernel(const float* __restrict__ part, int n_spl
   }
   float inv = sink ? sink_inverse(M, L, sink[h]) : 1.0f / L;
   if (gate) inv *= 1.0f / (1.0f + expf(-to_f32<T>(gate[(size_t)t * gate_stride + h])));
+  inv *= out_scale;
   for (int d = threadIdx.x; d < v_dim; d += blockDim.x) {
     float a = 0.f;
     for (int z = 0; z < n_splits; ++z) {
@@ -419,7 +423,7 @@ extern "C" int bn_attention_general_ex(const void* q, int q_stride, void* out, i
                                        const void* gate, int gate_stride, const int* tok_seq, const int* tok_pos, const int* slots,
                                        const int* page_table, int pt_stride,
                                        const void* k_cache, const void* v_cache, float* part, int n_splits,
-                                       const float* sink, int v_share, int out_wide, cudaStream_t stream) {
+                                       const float* sink, int v_share, int out_wide, float out_scale, cudaStream_t stream) {
   if (n_tokens <= 0) return BN_OK;
   if (v_share < 1 || n_kv_heads % v_share || (v_share > 1 && v_row > 0)) return BN_ERR_BAD_ARG;
   if (n_splits < 1 || n_splits > 64 || (n_splits > 1 && !part)) return BN_ERR_BAD_ARG;
@@ -452,7 +456,7 @@ extern "C" int bn_attention_general_ex(const void* q, int q_stride, void* out, i
     BN_LAUNCH((attention_grouped_kernel<TT, RR>), ggrid, ATT_THREADS, gsmem, stream, (const TT*)q, q_stride, (TT*)out,       \
               out_stride, n_heads, n_kv_heads, head_dim, v_dim, scale, window, keep_first, chunk, v_row, rel, n_rel,        \
               (const TT*)gate, gate_stride, tok_seq, tok_pos, slots, page_table, pt_stride, (const TT*)k_cache,              \
-              (const TT*)v_cache, part, n_splits, sink, v_share, out_wide);                                                           \
+              (const TT*)v_cache, part, n_splits, sink, v_share, out_wide, out_scale);                                                           \
   } while (0)
     if (gsmem <= 160 * 1024 && (dtype == BN_F32 || dtype == BN_BF16)) {
       if (dtype == BN_F32) { if (R == 4) BN_GROUPED(float, 4); else BN_GROUPED(float, 2); }
@@ -462,10 +466,10 @@ extern "C" int bn_attention_general_ex(const void* q, int q_stride, void* out, i
         dim3 mgrid(n_tokens, n_heads);
         if (dtype == BN_F32)
           BN_LAUNCH((attention_merge_kernel<float>), mgrid, 128, 0, stream, (const float*)part, n_splits, n_heads, v_dim,
-                    (const float*)gate, gate_stride, (float*)out, out_stride, sink, out_wide);
+                    (const float*)gate, gate_stride, (float*)out, out_stride, sink, out_wide, out_scale);
         else
           BN_LAUNCH((attention_merge_kernel<__nv_bfloat16>), mgrid, 128, 0, stream, (const float*)part, n_splits, n_heads, v_dim,
-                    (const __nv_bfloat16*)gate, gate_stride, (__nv_bfloat16*)out, out_stride, sink, out_wide);
+                    (const __nv_bfloat16*)gate, gate_stride, (__nv_bfloat16*)out, out_stride, sink, out_wide, out_scale);
       }
       BN_CHECK_LAUNCH();
       return BN_OK;
@@ -477,23 +481,23 @@ extern "C" int bn_attention_general_ex(const void* q, int q_stride, void* out, i
     BN_LAUNCH((attention_general_kernel<float>), grid, ATT_THREADS, smem, stream, 
         (const float*)q, q_stride, (float*)out, out_stride, n_heads, n_kv_heads, head_dim, v_dim, scale, window,
         keep_first, chunk, v_row, rel, n_rel, (const float*)gate, gate_stride,
-        tok_seq, tok_pos, slots, page_table, pt_stride, (const float*)k_cache, (const float*)v_cache, part, n_splits, sink, v_share, out_wide);
+        tok_seq, tok_pos, slots, page_table, pt_stride, (const float*)k_cache, (const float*)v_cache, part, n_splits, sink, v_share, out_wide, out_scale);
   else if (dtype == BN_BF16)
     BN_LAUNCH((attention_general_kernel<__nv_bfloat16>), grid, ATT_THREADS, smem, stream, 
         (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, out_stride, n_heads, n_kv_heads, head_dim, v_dim,
         scale, window, keep_first, chunk, v_row, rel, n_rel, (const __nv_bfloat16*)gate, gate_stride,
         tok_seq, tok_pos, slots, page_table, pt_stride,
-        (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, part, n_splits, sink, v_share, out_wide);
+        (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, part, n_splits, sink, v_share, out_wide, out_scale);
   else
     return BN_ERR_BAD_ARG;
   if (part) {
     dim3 mgrid(n_tokens, n_heads);
     if (dtype == BN_F32)
       BN_LAUNCH((attention_merge_kernel<float>), mgrid, 128, 0, stream, (const float*)part, n_splits, n_heads, v_dim,
-                (const float*)gate, gate_stride, (float*)out, out_stride, sink, out_wide);
+                (const float*)gate, gate_stride, (float*)out, out_stride, sink, out_wide, out_scale);
     else
       BN_LAUNCH((attention_merge_kernel<__nv_bfloat16>), mgrid, 128, 0, stream, (const float*)part, n_splits, n_heads, v_dim,
-                (const __nv_bfloat16*)gate, gate_stride, (__nv_bfloat16*)out, out_stride, sink, out_wide);
+                (const __nv_bfloat16*)gate, gate_stride, (__nv_bfloat16*)out, out_stride, sink, out_wide, out_scale);
   }
   BN_CHECK_LAUNCH();
   return BN_OK;
@@ -506,5 +510,5 @@ extern "C" int bn_attention_general(const void* q, int q_stride, void* out, int 
                                     const void* k_cache, const void* v_cache, cudaStream_t stream) {
   return bn_attention_general_ex(q, q_stride, out, out_stride, dtype, n_tokens, n_heads, n_kv_heads, head_dim, head_dim,
                                  scale, window, 0, 0, 0, nullptr, 0, nullptr, 0, tok_seq, tok_pos, slots, page_table,
-                                 pt_stride, k_cache, v_cache, nullptr, 1, nullptr, 1, 0, stream);
+                                 pt_stride, k_cache, v_cache, nullptr, 1, nullptr, 1, 0, 1.0f, stream);
 }

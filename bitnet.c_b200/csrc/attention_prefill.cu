@@ -43,7 +43,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
                          const int* __restrict__ seq_start, const int* __restrict__ seq_pos0,
                          const int* __restrict__ slots, const int* __restrict__ page_table, int pt_stride,
                          const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
-                         const float* __restrict__ sink, int v_share, int out_wide) {
+                         const float* __restrict__ sink, int v_share, int out_wide, float out_scale) {
   pdl_launch_dependents();  // the next kernel in the stream may begin its prologue
   pdl_wait();               // the kernels before this one have completed and their writes are visible
   extern __shared__ __align__(128) unsigned char smem[];
@@ -256,6 +256,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
       inv = a / (l_run[e] * a + exp2f(s2 - top));
     }
     if (gate) inv *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)(start + row0 + r) * gate_stride + h])));
+    inv *= out_scale;
     const size_t oat = (size_t)(start + row0 + r) * out_stride + (size_t)h * v_dim;
 #pragma unroll
     for (int j = 0; j < NT_O; ++j) {
@@ -278,7 +279,7 @@ static int launch_prefill(const void* q, int q_stride, void* out, int out_stride
                           const float* rel, int n_rel, const void* gate, int gate_stride, const int* tile_seq,
                           const int* tile_row0, const int* seq_start, const int* seq_pos0, const int* slots,
                           const int* page_table, int pt_stride, const void* k_cache, const void* v_cache,
-                          const float* sink, int v_share, int out_wide, cudaStream_t stream) {
+                          const float* sink, int v_share, int out_wide, float out_scale, cudaStream_t stream) {
   size_t smem = (size_t)PF_M * HD * 2 + 2 * (size_t)PF_N * HD * 2 + 2 * (size_t)PF_N * VD * 2;
   static bool configured = false;
   if (!configured) {
@@ -292,7 +293,7 @@ static int launch_prefill(const void* q, int q_stride, void* out, int out_stride
   BN_LAUNCH((attention_prefill_kernel<HD, PRECISE, VD>), grid, PF_THREADS, smem, stream, 
       (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, out_stride, n_heads, n_kv_heads, head_dim, v_dim,
       scale * 1.4426950408889634f, window, keep_first, chunk, v_row, rel, n_rel, (const __nv_bfloat16*)gate, gate_stride, tile_seq, tile_row0, seq_start, seq_pos0, slots, page_table, pt_stride,
-      (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, sink, v_share, out_wide);
+      (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, sink, v_share, out_wide, out_scale);
   BN_CHECK_LAUNCH();
   return BN_OK;
 }
@@ -308,14 +309,14 @@ static int launch_prefill(const void* q, int q_stride, void* out, int out_stride
 // plane when the values are the first v_dim numbers of wider rows (0: v_dim); sink [n_heads] float32: a score
 // per head that stands in the softmax's denominator once, with no key and no value; v_share: so many
 // consecutive key heads read one value head (the value plane has n_kv_heads / v_share heads); out_wide: out is
-// a float32 array.
+// a float32 array; out_scale: a factor on all of the output.
 extern "C" int bn_attention_prefill_ex(const void* q, int q_stride, void* out, int out_stride, int n_tiles, int n_heads,
                                        int n_kv_heads, int head_dim, int v_dim, float scale, int window, int keep_first,
                                        int chunk, int v_row, const float* rel, int n_rel, const void* gate, int gate_stride, int precise,
                                        const int* tile_seq, const int* tile_row0, const int* seq_start,
                                        const int* seq_pos0, const int* slots, const int* page_table, int pt_stride,
                                        const void* k_cache, const void* v_cache, const float* sink, int v_share, int out_wide,
-                                       cudaStream_t stream) {
+                                       float out_scale, cudaStream_t stream) {
   if (n_tiles <= 0) return BN_OK;
   if (v_share < 1 || n_kv_heads % v_share || (v_share > 1 && v_row > 0)) return BN_ERR_BAD_ARG;
   if (v_row <= 0) v_row = v_dim;
@@ -326,7 +327,7 @@ extern "C" int bn_attention_prefill_ex(const void* q, int q_stride, void* out, i
     return BN_ERR_BAD_ARG;
 #define BN_PF_ARGS q, q_stride, out, out_stride, n_tiles, n_heads, n_kv_heads, head_dim, v_dim, scale, window, keep_first, chunk, v_row, rel, \
                    n_rel, gate, gate_stride, tile_seq, tile_row0, seq_start, seq_pos0, slots, page_table, pt_stride,      \
-                   k_cache, v_cache, sink, v_share, out_wide, stream
+                   k_cache, v_cache, sink, v_share, out_wide, out_scale, stream
   if (precise) {
     // key and value heads of their own widths: the instantiation for each
     const int hd = head_dim <= 64 ? 64 : head_dim <= 128 ? 128 : 256, vd = v_dim <= 64 ? 64 : v_dim <= 128 ? 128 : 256;
@@ -353,5 +354,5 @@ extern "C" int bn_attention_prefill(const void* q, int q_stride, void* out, int 
                                     const void* v_cache, cudaStream_t stream) {
   return bn_attention_prefill_ex(q, q_stride, out, out_stride, n_tiles, n_heads, n_kv_heads, head_dim, head_dim, scale, window, 0,
                                  0, 0, nullptr, 0, nullptr, 0, 0, tile_seq, tile_row0, seq_start, seq_pos0, slots, page_table,
-                                 pt_stride, k_cache, v_cache, nullptr, 1, 0, stream);
+                                 pt_stride, k_cache, v_cache, nullptr, 1, 0, 1.0f, stream);
 }

@@ -53,6 +53,9 @@ struct PtArgs {
   int out_stride;
   int n_heads, n_kv_heads, head_dim, v_dim;
   const float* sink;  // [n_heads] or null
+  const __nv_bfloat16* gate;  // [n_tokens, gate_stride]: a number per head whose logistic function multiplies its output, or null
+  int gate_stride;
+  float out_scale;
   float scale_log2e;
   int window;
   const int* tile_seq;
@@ -368,6 +371,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const float sk = a.sink[h] * 1.4426950408889634f, top = fmaxf(m_ref, sk), down = exp2f(m_ref - top);
         inv = down / (l_run * down + exp2f(sk - top));
       }
+      if (a.gate && r < rows_here) inv *= 1.0f / (1.0f + expf(-__bfloat162float(a.gate[(size_t)(start + row0 + r) * a.gate_stride + h])));
+      inv *= a.out_scale;
       __nv_bfloat16* orow = a.out + (size_t)(start + row0 + r) * a.out_stride + (size_t)h * a.v_dim;
 #pragma unroll
       for (int c = 0; c < VD; c += 32) {
@@ -448,9 +453,11 @@ static int launch_pt(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
 // that block).
 // The values' cache is [n_cache_pages, n_kv_heads, 64, v_dim] with v_dim a multiple of 16 up to 128.  precise: the weights
 // enter the value product with 16 bits of mantissa.  sink: [n_heads] float32 scores that stand in the sums only, or null.
+// gate [n_tokens, gate_stride]: a number per token and head whose logistic function multiplies the head's output, or null;
+// out_scale: a factor on all of the output.
 extern "C" int bn_attention_prefill_tc_ex(const void* q, int q_stride, int n_tokens, void* out, int out_stride, int n_tiles,
                                           int n_heads, int n_kv_heads, int head_dim, int v_dim, float scale, int window, int precise,
-                                          const float* sink, const int* tile_seq, const int* tile_row0, const int* seq_start,
+                                          const float* sink, const void* gate, int gate_stride, float out_scale, const int* tile_seq, const int* tile_row0, const int* seq_start,
                                           const int* seq_pos0, const int* slots, const int* page_table, int pt_stride,
                                           const void* k_cache, const void* v_cache, int n_cache_pages, int* status,
                                           cudaStream_t stream) {
@@ -467,7 +474,8 @@ extern "C" int bn_attention_prefill_tc_ex(const void* q, int q_stride, int n_tok
     return BN_ERR_BAD_ARG;
   PtArgs a = {};
   a.out = (__nv_bfloat16*)out; a.out_stride = out_stride; a.n_heads = n_heads; a.n_kv_heads = n_kv_heads;
-  a.head_dim = head_dim; a.v_dim = v_dim; a.sink = sink; a.scale_log2e = scale * 1.4426950408889634f; a.window = window; a.tile_seq = tile_seq;
+  a.head_dim = head_dim; a.v_dim = v_dim; a.sink = sink; a.gate = (const __nv_bfloat16*)gate;
+  a.gate_stride = gate_stride; a.out_scale = out_scale; a.scale_log2e = scale * 1.4426950408889634f; a.window = window; a.tile_seq = tile_seq;
   a.tile_row0 = tile_row0; a.seq_start = seq_start; a.seq_pos0 = seq_pos0; a.slots = slots; a.page_table = page_table;
   a.pt_stride = pt_stride; a.status = status;
   BN_TRACE_ONLY(a.trace = nullptr;)
@@ -491,6 +499,6 @@ extern "C" int bn_attention_prefill_tc(const void* q, int q_stride, int n_tokens
                                        const void* k_cache, const void* v_cache, int n_cache_pages, int* status,
                                        cudaStream_t stream) {
   return bn_attention_prefill_tc_ex(q, q_stride, n_tokens, out, out_stride, n_tiles, n_heads, n_kv_heads, head_dim, head_dim, scale,
-                                    window, 0, nullptr, tile_seq, tile_row0, seq_start, seq_pos0, slots, page_table, pt_stride,
+                                    window, 0, nullptr, nullptr, 0, 1.0f, tile_seq, tile_row0, seq_start, seq_pos0, slots, page_table, pt_stride,
                                     k_cache, v_cache, n_cache_pages, status, stream);
 }

@@ -51,6 +51,7 @@ SOURCES: Dict[str, str] = {
     "delta_rule": "delta_rule.cu",
     "streams": "streams.cu",
     "gated_state": "gated_state.cu",
+    "gated_linear": "gated_linear.cu",
     "sigmoid_attention": "sigmoid_attention.cu",
     "sigmoid_attention_prefill": "sigmoid_attention_prefill.cu",
 }

@@ -112,6 +112,12 @@ __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { retu
 // the bits above the low byte of their `mode` argument (mode 2 | BN_ACT_GELU_TANH << 8).
 #define BN_ACT_SILU 0
 #define BN_ACT_GELU_TANH 1
+// The activation of a feed-forward without a gate: the square of relu.
+#define BN_ACT_RELU2 2
+__device__ __forceinline__ float relu_squared(float z) {
+  const float p = fmaxf(z, 0.f);
+  return p * p;
+}
 __device__ __forceinline__ float glu_activation(float g, int act) {
   if (act == BN_ACT_GELU_TANH) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
   return g / (1.0f + expf(-g));

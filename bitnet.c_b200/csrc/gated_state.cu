@@ -1,5 +1,6 @@
-// Recurrences of a matrix state per head under one decay per head and token: the gated delta rule and the
-// state-space (Mamba-2) update, with the short convolutions in front of them and the gated norms behind.
+// Recurrences of a matrix state per head under one decay per head and token: the gated delta rule, the
+// state-space (Mamba-2) update and the update under a fixed decay per head (lightning attention), with the short
+// convolutions in front of them and the gated norms behind.
 //
 // Per head, with a state S [dim, vdim] (float32, zero at a sequence's start, kept per slot), a log decay l_t and a
 // factor b_t (both from per-head pre-activations):
@@ -8,6 +9,7 @@
 //                  q and k unit vectors per head, q times a scale                     l = -e^A softplus(. + bias)
 //   state space    S' = e^l S;  S = S' + b k v^T;    o = S^T q + D v                  b = softplus(. + bias), l = -e^A b
 //                  (k: the input matrix B, q: the read-out C, v: the inner input x)
+//   fixed decay    the state-space update with b = 1 and one log decay per head, the same for every token
 //
 // q and k belong to groups of heads (head h uses group h / (heads / groups)).  In front, every channel of q, k and v
 // goes through a short convolution along the sequence (optionally with a bias) and SiLU.  All of it float32.
@@ -30,7 +32,8 @@ __device__ __forceinline__ float gs_silu(float z) { return z / (1.0f + expf(-z))
 struct GatedStateArgs {
   const void* proj;
   const float* gate;          // [tokens, gate_stride]: log decays' (or step sizes') pre-activations at a_off, delta: b's at b_off
-  const float* conv_w;        // [taps][channels]
+  const float* log_decay;     // [heads]: fixed log decays (no gates are read then), or null
+  const float* conv_w;        // [taps][channels], or null: no convolution (taps = 1)
   const float* conv_b;        // [channels] or null
   const float* dt_bias;       // [heads]
   const float* a_log;         // [heads]
@@ -57,6 +60,7 @@ struct GatedStateArgs {
 // (log decay, factor) of a head at a token
 template <bool DELTA>
 __device__ __forceinline__ float2 gs_gates(const GatedStateArgs& a, int t, int h) {
+  if (!DELTA && a.log_decay) return make_float2(a.log_decay[h], 1.0f);
   const float* g = a.gate + (size_t)t * a.gate_stride;
   const float dt = gs_softplus(g[a.a_off + h] + a.dt_bias[h]);
   const float beta = DELTA ? 1.0f / (1.0f + expf(-g[a.b_off + h])) : dt;
@@ -105,7 +109,12 @@ __global__ void gated_state_prepare_kernel(const GatedStateArgs a, float* __rest
       const int back = a.taps - 1 - j;  // how many positions before this token the tap looks
       if (back > pos) continue;         // no such position
       float x[V], w[V];
-      gs_load<float, V>(a.conv_w + (size_t)j * n_ch + c, w);
+      if (a.conv_w) {
+        gs_load<float, V>(a.conv_w + (size_t)j * n_ch + c, w);
+      } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) w[e] = 1.0f;
+      }
       if (r - back >= 0) gs_load<T, V>(proj + (size_t)(t - back) * a.stride + col, x);
       else gs_load<float, V>(ring + (size_t)((pos - back) % a.taps) * n_ch + c, x);
 #pragma unroll
@@ -894,7 +903,7 @@ __global__ void __launch_bounds__(GS_THREADS) gated_state_token_kernel(const Gat
     if (which < 2 ? d < dim : d < cols) {
       const int c = which == 0 ? g * dim + d : (which == 1 ? n_qk + g * dim + d : 2 * n_qk + h * vdim + tile * 32 + d);
       const float x = to_f32<T>(row[a.column(c)]);
-      float acc = fmaf(a.conv_w[(size_t)(a.taps - 1) * n_ch + c], x, a.conv_b ? a.conv_b[c] : 0.f);
+      float acc = fmaf(a.conv_w ? a.conv_w[(size_t)(a.taps - 1) * n_ch + c] : 1.0f, x, a.conv_b ? a.conv_b[c] : 0.f);
       for (int j = 0; j < a.taps - 1; ++j) {
         const int p = pos - (a.taps - 1 - j);
         if (p >= 0) acc = fmaf(a.conv_w[(size_t)j * n_ch + c], ring[(size_t)(p % a.taps) * n_ch + c], acc);
@@ -949,21 +958,22 @@ __global__ void __launch_bounds__(GS_THREADS) gated_state_token_kernel(const Gat
 
 static bool gs_fits(const GatedStateArgs& a) {
   const int n_qk = a.groups * a.dim, n_v = a.heads * a.vdim;
-  return a.proj && a.gate && a.conv_w && a.dt_bias && a.a_log && a.state && a.tok_seq && a.seq_start && a.seq_pos0 && a.slots &&
+  const bool gates = a.log_decay || (a.gate && a.dt_bias && a.a_log && a.a_off >= 0 && a.a_off + a.heads <= a.gate_stride &&
+                                     a.b_off + a.heads <= a.gate_stride);
+  return a.proj && gates && (a.conv_w || a.taps == 1) && a.state && a.tok_seq && a.seq_start && a.seq_pos0 && a.slots &&
          a.groups > 0 && a.heads > 0 && a.heads % a.groups == 0 && a.dim > 0 && a.dim <= 256 && a.vdim > 0 && a.taps >= 1 &&
          a.taps <= GS_MAX_TAPS && a.q_off >= 0 && a.k_off >= 0 && a.v_off >= 0 && a.q_off + n_qk <= a.stride &&
-         a.k_off + n_qk <= a.stride && a.v_off + n_v <= a.stride && a.a_off >= 0 && a.a_off + a.heads <= a.gate_stride &&
-         a.b_off + a.heads <= a.gate_stride &&
+         a.k_off + n_qk <= a.stride && a.v_off + n_v <= a.stride &&
          a.state_stride >= (size_t)a.heads * a.dim * a.vdim + (a.taps > 1 ? (size_t)a.taps * (2 * n_qk + n_v) : 0);
 }
 
 static GatedStateArgs gs_args(const void* proj, int n_tokens, int stride, int q_off, int k_off, int v_off, const float* gate,
                               int gate_stride, int a_off, int b_off, int groups, int heads, int dim, int vdim, int taps,
                               const float* conv_w, const float* conv_b, const float* dt_bias, const float* a_log, const float* d,
-                              float q_scale, float* state, long long state_stride, const int* tok_seq, const int* seq_start,
+                              const float* log_decay, float q_scale, float* state, long long state_stride, const int* tok_seq, const int* seq_start,
                               const int* seq_pos0, const int* slots, int n_seqs) {
   GatedStateArgs a = {};
-  a.proj = proj; a.gate = gate; a.conv_w = conv_w; a.conv_b = conv_b; a.dt_bias = dt_bias; a.a_log = a_log; a.d = d;
+  a.proj = proj; a.gate = gate; a.conv_w = conv_w; a.conv_b = conv_b; a.dt_bias = dt_bias; a.a_log = a_log; a.d = d; a.log_decay = log_decay;
   a.state = state; a.tok_seq = tok_seq; a.seq_start = seq_start; a.seq_pos0 = seq_pos0; a.slots = slots;
   a.state_stride = (size_t)state_stride; a.q_scale = q_scale; a.stride = stride; a.gate_stride = gate_stride; a.q_off = q_off;
   a.k_off = k_off; a.v_off = v_off; a.a_off = a_off; a.b_off = b_off < 0 ? 0 : b_off; a.groups = groups; a.heads = heads; a.dim = dim;
@@ -971,15 +981,16 @@ static GatedStateArgs gs_args(const void* proj, int n_tokens, int stride, int q_
   return a;
 }
 
-// The arguments all entry points share (b_off < 0: the state-space update, else the delta rule).
+// The arguments all entry points share (b_off < 0: the state-space update, or with log_decay the one under fixed decays; else
+// the delta rule).
 #define GS_PARAMS                                                                                                              \
   const void *proj, int dtype, int n_tokens, int stride, int q_off, int k_off, int v_off, const float *gate, int gate_stride,  \
       int a_off, int b_off, int groups, int heads, int dim, int vdim, int taps, const float *conv_w, const float *conv_b,      \
-      const float *dt_bias, const float *a_log, const float *d, float q_scale, float *state, long long state_stride,           \
+      const float *dt_bias, const float *a_log, const float *d, const float *log_decay, float q_scale, float *state, long long state_stride,           \
       const int *tok_seq, const int *seq_start, const int *seq_pos0, const int *slots, int n_seqs
 #define GS_PASS                                                                                                                \
   proj, n_tokens, stride, q_off, k_off, v_off, gate, gate_stride, a_off, b_off, groups, heads, dim, vdim, taps, conv_w, conv_b, \
-      dt_bias, a_log, d, q_scale, state, state_stride, tok_seq, seq_start, seq_pos0, slots, n_seqs
+      dt_bias, a_log, d, log_decay, q_scale, state, state_stride, tok_seq, seq_start, seq_pos0, slots, n_seqs
 
 // q and k as they enter the recurrence, v, and (log decay, factor) per head, all float32.
 extern "C" int bn_gated_state_prepare(GS_PARAMS, float* qn, float* kn, float* vc, float* lb, cudaStream_t stream) {
@@ -1131,12 +1142,12 @@ extern "C" int bn_gated_state_token(GS_PARAMS, float* out, cudaStream_t stream) 
 // ---- behind the recurrence --------------------------------------------------------------------------
 // Every row of o [T, parts * len] in equal parts, with a gate z of the same width:
 //   gate first   y = o silu(z);            out = y / sqrt(mean over the part (y^2) + eps) * gain
-//   gate last    out = o / sqrt(mean over the part (o^2) + eps) * gain * silu(z)
+//   gate last    out = o / sqrt(mean over the part (o^2) + eps) * gain * silu(z), or * sigmoid(z)
 // gain holds one number per place of the row, or per place of a part (gain_len = len: shared by the parts).
 // THREADS 32: a warp per part, eight parts per block; else a block per part.  The part waits in shared memory.
 template <typename T, typename G, int THREADS, int V>
 __global__ void state_output_kernel(const float* __restrict__ o, const G* __restrict__ z, int z_stride, const float* __restrict__ gain,
-                                    int gain_len, int parts, int len, float eps, int gate_first, T* __restrict__ out, int n_items) {
+                                    int gain_len, int parts, int len, float eps, int gate_first, int logistic, T* __restrict__ out, int n_items) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float part[];
@@ -1175,7 +1186,7 @@ __global__ void state_output_kernel(const float* __restrict__ o, const G* __rest
 #pragma unroll
     for (int e = 0; e < V; ++e) {
       w[e] *= y[i + e] * scale;
-      if (!gate_first) w[e] *= gs_silu(g[e]);
+      if (!gate_first) w[e] *= logistic ? 1.0f / (1.0f + expf(-g[e])) : gs_silu(g[e]);
     }
     if (V == 4 && sizeof(T) == 2) {
       const __nv_bfloat162 a = __floats2bfloat162_rn(w[0], w[1 % V]), b = __floats2bfloat162_rn(w[2 % V], w[3 % V]);
@@ -1193,7 +1204,7 @@ __global__ void state_output_kernel(const float* __restrict__ o, const G* __rest
 
 template <typename T, typename G, int THREADS, int V>
 static int launch_state_output(const float* o, const void* z, int z_stride, const float* gain, int gain_len, int parts, int len,
-                               float eps, int gate_first, void* out, int n_items, cudaStream_t stream) {
+                               float eps, int gate_first, int logistic, void* out, int n_items, cudaStream_t stream) {
   const int padded = (len + 3) / 4 * 4;
   const size_t smem = (size_t)padded * sizeof(float) * (THREADS == 32 ? 8 : 1);
   if (smem > 200 * 1024) return BN_ERR_BAD_ARG;
@@ -1208,14 +1219,14 @@ static int launch_state_output(const float* o, const void* z, int z_stride, cons
   const unsigned blocks = THREADS == 32 ? (unsigned)((n_items + 7) / 8) : (unsigned)n_items;
   const int threads = THREADS == 32 ? 256 : (len >= 4096 ? 512 : 256);
   BN_LAUNCH((state_output_kernel<T, G, THREADS, V>), blocks, threads, smem, stream, o, (const G*)z, z_stride, gain, gain_len, parts, len,
-            eps, gate_first, (T*)out, n_items);
+            eps, gate_first, logistic, (T*)out, n_items);
   return BN_OK;
 }
 
 extern "C" int bn_state_output(const float* o, const void* z, int z_dtype, int z_stride, const float* gain, int gain_len, int dtype,
-                               int n_tokens, int parts, int len, float eps, int gate_first, void* out, cudaStream_t stream) {
+                               int n_tokens, int parts, int len, float eps, int gate_first, int logistic, void* out, cudaStream_t stream) {
   if (n_tokens <= 0) return BN_OK;
-  if (!o || !z || !gain || !out || parts <= 0 || len <= 0 || z_stride < parts * len || !(eps > 0.f) ||
+  if (!o || !z || !gain || !out || parts <= 0 || len <= 0 || z_stride < parts * len || !(eps > 0.f) || (gate_first && logistic) ||
       (gain_len != len && gain_len != parts * len))
     return BN_ERR_BAD_ARG;
   const int items = n_tokens * parts;
@@ -1223,10 +1234,10 @@ extern "C" int bn_state_output(const float* o, const void* z, int z_dtype, int z
 #define GS_OUT(TT, GG)                                                                                                               \
   do {                                                                                                                               \
     if (len <= 512)                                                                                                                  \
-      return vec ? launch_state_output<TT, GG, 32, 4>(o, z, z_stride, gain, gain_len, parts, len, eps, gate_first, out, items, stream) \
-                 : launch_state_output<TT, GG, 32, 1>(o, z, z_stride, gain, gain_len, parts, len, eps, gate_first, out, items, stream); \
-    return vec ? launch_state_output<TT, GG, 256, 4>(o, z, z_stride, gain, gain_len, parts, len, eps, gate_first, out, items, stream) \
-               : launch_state_output<TT, GG, 256, 1>(o, z, z_stride, gain, gain_len, parts, len, eps, gate_first, out, items, stream); \
+      return vec ? launch_state_output<TT, GG, 32, 4>(o, z, z_stride, gain, gain_len, parts, len, eps, gate_first, logistic, out, items, stream) \
+                 : launch_state_output<TT, GG, 32, 1>(o, z, z_stride, gain, gain_len, parts, len, eps, gate_first, logistic, out, items, stream); \
+    return vec ? launch_state_output<TT, GG, 256, 4>(o, z, z_stride, gain, gain_len, parts, len, eps, gate_first, logistic, out, items, stream) \
+               : launch_state_output<TT, GG, 256, 1>(o, z, z_stride, gain, gain_len, parts, len, eps, gate_first, logistic, out, items, stream); \
   } while (0)
   if (dtype == BN_F32 && z_dtype == BN_F32) GS_OUT(float, float);
   if (dtype == BN_BF16 && z_dtype == BN_F32) GS_OUT(__nv_bfloat16, float);

@@ -49,7 +49,7 @@ struct VecLd<__nv_bfloat16> {
 template <typename T>
 __global__ void __launch_bounds__(SK_WARPS * 32)
 linear_skinny_kernel(const T* __restrict__ x, const T* __restrict__ w, void* __restrict__ out, int out_dtype, int M, int N,
-                     int K, int ldo, float* __restrict__ partial) {
+                     int K, int ldo, float* __restrict__ partial, const float* __restrict__ bias) {
   pdl_launch_dependents();  // the next kernel in the stream may begin its prologue
   pdl_wait();               // the kernels before this one have completed and their writes are visible
   __shared__ __align__(16) T xs[SK_MT][SK_KC];
@@ -112,7 +112,7 @@ linear_skinny_kernel(const T* __restrict__ x, const T* __restrict__ w, void* __r
           float v = warp_sum(acc[i][c]);
           if (lane == 0 && c < nc) {
             if (gridDim.y > 1) partial[((size_t)blockIdx.y * M + m0 + i) * N + n0 + c] = v;
-            else store_from_f32(out, out_dtype, (size_t)(m0 + i) * ldo + n0 + c, v);
+            else store_from_f32(out, out_dtype, (size_t)(m0 + i) * ldo + n0 + c, bias ? v + bias[n0 + c] : v);
           }
         }
       }
@@ -122,7 +122,8 @@ linear_skinny_kernel(const T* __restrict__ x, const T* __restrict__ w, void* __r
 
 // out[m, n] = partial[0][m, n] + partial[1][m, n] + ... in that order.
 __global__ void __launch_bounds__(256)
-linear_skinny_sum_kernel(const float* __restrict__ partial, int splits, void* __restrict__ out, int out_dtype, int M, int N, int ldo) {
+linear_skinny_sum_kernel(const float* __restrict__ partial, int splits, void* __restrict__ out, int out_dtype, int M, int N, int ldo,
+                         const float* __restrict__ bias) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -130,6 +131,7 @@ linear_skinny_sum_kernel(const float* __restrict__ partial, int splits, void* __
   const int m = (int)(i / N), n = (int)(i - (size_t)m * N);
   float v = 0.f;
   for (int s = 0; s < splits; ++s) v += partial[(size_t)s * M * N + i];
+  if (bias) v += bias[n];
   store_from_f32(out, out_dtype, (size_t)m * ldo + n, v);
 }
 
@@ -158,9 +160,10 @@ extern "C" int bn_linear_skinny_splits(int N, int K) {
 }
 
 // x and w share the element type `dtype`; K must be a multiple of 8 (16-byte rows).  partial: float32
-// scratch of bn_linear_skinny_splits(N, K) * M * N floats (not used when that is 1).
+// scratch of bn_linear_skinny_splits(N, K) * M * N floats (not used when that is 1).  bias: [N] float32 added to every row, or
+// null.
 extern "C" int bn_linear_skinny(const void* x, const void* w, int dtype, void* out, int out_dtype, int M, int N,
-                                int K, int ldo, float* partial, cudaStream_t stream) {
+                                int K, int ldo, float* partial, const float* bias, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return BN_OK;
   if (K <= 0 || K % 8 || ldo < N) return BN_ERR_BAD_ARG;
   const int splits = bn_linear_skinny_splits(N, K);
@@ -168,16 +171,16 @@ extern "C" int bn_linear_skinny(const void* x, const void* w, int dtype, void* o
   dim3 grid((unsigned)((N + SK_WARPS * SK_COLS - 1) / (SK_WARPS * SK_COLS)), (unsigned)splits);
   if (dtype == BN_F32)
     BN_LAUNCH((linear_skinny_kernel<float>), grid, SK_WARPS * 32, 0, stream, (const float*)x, (const float*)w, out,
-              out_dtype, M, N, K, ldo, partial);
+              out_dtype, M, N, K, ldo, partial, bias);
   else if (dtype == BN_BF16)
     BN_LAUNCH((linear_skinny_kernel<__nv_bfloat16>), grid, SK_WARPS * 32, 0, stream,
-              (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, out, out_dtype, M, N, K, ldo, partial);
+              (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, out, out_dtype, M, N, K, ldo, partial, bias);
   else
     return BN_ERR_BAD_ARG;
   if (splits > 1) {
     const size_t total = (size_t)M * N;
     BN_LAUNCH(linear_skinny_sum_kernel, (unsigned)((total + 255) / 256), 256, 0, stream, (const float*)partial, splits, out,
-              out_dtype, M, N, ldo);
+              out_dtype, M, N, ldo, bias);
   }
   BN_CHECK_LAUNCH();
   return BN_OK;

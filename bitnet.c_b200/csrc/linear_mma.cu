@@ -46,6 +46,7 @@ struct LmArgs {
   int k_per_split;  // multiple of LM_KC
   int mode;         // 0 store, 1 partial, 2 swiglu
   int act;          // mode 2: the gate's activation (BN_ACT_*)
+  const float* bias;  // mode 0: [N] added to every row, or null
   int ldo;
   float* scratch;   // modes 0/2 with gridDim.y > 1: [splits][row blocks][64 rows][8*NT] partial tiles
   int* counters;    // one ticket counter per row block, zero before and after the launch
@@ -177,8 +178,8 @@ __global__ void __launch_bounds__(128) linear_mma_kernel(LmArgs a) {
       if (m >= a.M) continue;
       float v_lo = acc[nt][j], v_hi = acc[nt][2 + j];
       if (a.mode == 0) {
-        if (n_lo < a.N) store_from_f32(a.out, a.out_dtype, (size_t)m * a.ldo + n_lo, v_lo);
-        if (n_hi < a.N) store_from_f32(a.out, a.out_dtype, (size_t)m * a.ldo + n_hi, v_hi);
+        if (n_lo < a.N) store_from_f32(a.out, a.out_dtype, (size_t)m * a.ldo + n_lo, a.bias ? v_lo + a.bias[n_lo] : v_lo);
+        if (n_hi < a.N) store_from_f32(a.out, a.out_dtype, (size_t)m * a.ldo + n_hi, a.bias ? v_hi + a.bias[n_hi] : v_hi);
       } else if (a.mode == 1) {
         float* part = (float*)a.out + ((size_t)blockIdx.y * a.M + m) * a.N;
         if (n_lo < a.N) part[n_lo] = v_lo;
@@ -195,7 +196,7 @@ __global__ void __launch_bounds__(128) linear_mma_kernel(LmArgs a) {
   }
 }
 
-// x [M, K], w [N, K] bfloat16.  mode 0: out [M, ldo] of out_dtype.  mode 1: out is float32
+// x [M, K], w [N, K] bfloat16.  mode 0: out [M, ldo] of out_dtype, plus bias [N] (or null).  mode 1: out is float32
 // [n_splits, M, N] (every split writes its whole slice).  mode 2: w has N = 2 I rows in blocks
 // of 8 gate / 8 up rows, out [M, ldo] holds silu(gate) * up for I columns.
 // With n_splits > 1 in modes 0 and 2, scratch must hold n_splits * ceil(N/64) * 64 * Mp floats
@@ -203,7 +204,7 @@ __global__ void __launch_bounds__(128) linear_mma_kernel(LmArgs a) {
 // shared by launches that do not overlap on the device.
 extern "C" int bn_linear_mma(const void* x, const void* w, void* out, int out_dtype, int M, int N, int K, int ldo,
                              int mode, int n_splits, float* scratch, long long scratch_floats, int* counters,
-                             int n_counters, cudaStream_t stream) {
+                             int n_counters, const float* bias, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return BN_OK;
   const int act = mode >> 8;
   mode &= 255;
@@ -214,6 +215,7 @@ extern "C" int bn_linear_mma(const void* x, const void* w, void* out, int out_dt
   LmArgs a;
   a.x = (const __nv_bfloat16*)x; a.w = (const __nv_bfloat16*)w; a.out = out; a.out_dtype = out_dtype;
   a.M = M; a.N = N; a.K = K; a.mode = mode; a.act = act; a.ldo = ldo; a.scratch = scratch; a.counters = counters;
+  a.bias = bias;
   int chunks = (K + LM_KC - 1) / LM_KC;
   if (n_splits > chunks) n_splits = chunks;
   a.k_per_split = ((chunks + n_splits - 1) / n_splits) * LM_KC;

@@ -73,12 +73,12 @@ struct TcArgs {
   int M, N, K;
   int ldo;
   int mode;        // 0 store, 2 swiglu, 3 residual add + gain + sums of squares
-  int act;         // mode 2: the gate's activation (BN_ACT_*)
+  int act;         // mode 2: the gate's activation (BN_ACT_*); mode 0: BN_ACT_RELU2 squares the positive part, else none
   int k_blocks;    // ceil(K / 64)
   const float* row_ss;   // [ss_parts][ss_stride]: sums of squares of the input rows, or null (rows are plain)
   int ss_parts, ss_stride;
   float inv_width, eps;  // of the norm whose scale the input rows still lack
-  const void* gain;      // mode 3: the next norm's weight [N]
+  const void* gain;      // mode 3: the next norm's weight [N]; mode 0: a bias [N] or null
   int gain_dtype;
   __nv_bfloat16* xg;     // mode 3: [M, N] residual * gain
   float* ss_out;         // mode 3: [tiles * cluster][ss_out_stride] sums of squares of this block's slice of each row
@@ -378,11 +378,16 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
         const int n = tile * TC_BM + r0 + nl;
         if (n < a.N) {
           float v[W];
+          const float bias = a.gain != nullptr ? load_as_f32(a.gain, a.gain_dtype, (size_t)n) : 0.f;
           slice_values(nl, mg, v);
 #pragma unroll
           for (int i = 0; i < W; ++i) {
             const int m = mg * W + i;
-            if (m < a.M) store_from_f32(a.out, a.out_dtype, (size_t)m * a.ldo + n, a.row_ss != nullptr ? v[i] * row_scale[m] : v[i]);
+            if (m < a.M) {
+              float y = (a.row_ss != nullptr ? v[i] * row_scale[m] : v[i]) + bias;
+              if (a.act == BN_ACT_RELU2) y = relu_squared(y);
+              store_from_f32(a.out, a.out_dtype, (size_t)m * a.ldo + n, y);
+            }
           }
         }
         mg += dm; nl += dn;
@@ -573,7 +578,8 @@ extern "C" int bn_linear_tc_auto_cluster(int N, int K) {
 }
 
 // x [M, K], w [N, K] bfloat16, both 16-byte aligned with K a multiple of 8.  mode 0: out [M, ldo]
-// of out_dtype; mode 2: N = 2 I weight rows in blocks of 8 gate / 8 up rows, out holds
+// of out_dtype, plus a bias per column (gain [N] of gain_dtype, or null), with BN_ACT_RELU2 << 8 the square of
+// its positive part; mode 2: N = 2 I weight rows in blocks of 8 gate / 8 up rows, out holds
 // silu(gate) * up in I columns; mode 3: out is a float32 residual [M, ldo] that the product is
 // added to in place, xg [M, N] bfloat16 receives residual * gain (gain [N] of gain_dtype) and
 // ss_out [tiles * cluster][ss_out_stride] the sums of squares of each block's slice of every row
@@ -589,13 +595,14 @@ extern "C" int bn_linear_tc_ex(const void* x, const void* w, void* out, int out_
   if (M <= 0 || N <= 0) return BN_OK;
   const int act = mode >> 8;
   mode &= 255;
-  if (act != BN_ACT_SILU && act != BN_ACT_GELU_TANH) return BN_ERR_BAD_ARG;
+  if (act != BN_ACT_SILU && act != BN_ACT_GELU_TANH && !(act == BN_ACT_RELU2 && mode == 0)) return BN_ERR_BAD_ARG;
   if (M > 64 || K <= 0 || K % 8 || cluster < 0 || cluster > 8 || (mode != 0 && mode != 2 && mode != 3) || !status)
     return BN_ERR_BAD_ARG;
   if (mode == 2 && (N % 16)) return BN_ERR_BAD_ARG;
   if (mode == 3 && (!gain || !xg || !ss_out || ss_out_stride < M || cluster == 0 || out_dtype != BN_F32 ||
                     (gain_dtype != BN_F32 && gain_dtype != BN_BF16)))
     return BN_ERR_BAD_ARG;
+  if (mode == 0 && gain && gain_dtype != BN_F32 && gain_dtype != BN_BF16) return BN_ERR_BAD_ARG;
   if (row_ss && (ss_parts <= 0 || ss_stride < M)) return BN_ERR_BAD_ARG;
   if (((uintptr_t)x | (uintptr_t)w) & 15) return BN_ERR_BAD_ARG;
   int mp = M <= 16 ? 16 : (M <= 32 ? 32 : 64);

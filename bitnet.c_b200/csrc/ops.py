@@ -59,6 +59,12 @@ def _need(t: torch.Tensor, name: str, dtype=None, dims: Optional[int] = None) ->
         raise KernelError(f"{name} must have {dims} dimensions, got {tuple(t.shape)}")
 
 
+def _need_rows(t: torch.Tensor, name: str, dtype=None) -> None:
+    """A matrix whose rows may lie apart (columns of a wider one): unit inner stride."""
+    if not isinstance(t, torch.Tensor) or not t.is_cuda or t.dim() != 2 or t.stride(1) != 1 or (dtype is not None and t.dtype != dtype):
+        raise KernelError(f"{name} must be a CUDA matrix with unit inner stride" + (f" of type {dtype}" if dtype is not None else ""))
+
+
 def _check(status: int, what: str) -> None:
     if status == 0:
         return
@@ -298,6 +304,13 @@ def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float, out_dtype: torch.
     _check(_fn("act", "bn_poly_norm")(_ptr(z), int(_code(z)), _ptr(coef), c_float(eps), _ptr(out), int(_code(out)), int(n), int(length),
                                       int(row), _stream()), "poly_norm")
     return out
+
+
+def relu_squared(x: torch.Tensor) -> torch.Tensor:
+    """The square of relu, in place."""
+    _need(x, "x")
+    _check(_fn("act", "bn_relu_squared")(_ptr(x), _ptr(x), int(_code(x)), ctypes.c_longlong(x.numel()), _stream()), "relu_squared")
+    return x
 
 
 def scale_softcap(x: torch.Tensor, scale: float, softcap: float) -> torch.Tensor:
@@ -568,7 +581,7 @@ def attention_general(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_token
                       k_cache: torch.Tensor, v_cache: torch.Tensor, *, keep_first: int = 0,
                       rel: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
                       gate_stride: int = 0, max_keys: int = 0, chunk: int = 0, v_dim: int = 0,
-                      sink: Optional[torch.Tensor] = None, v_share: int = 1) -> torch.Tensor:
+                      sink: Optional[torch.Tensor] = None, v_share: int = 1, out_scale: float = 1.0) -> torch.Tensor:
     """Causal attention of every new token over its sequence's pages; q may be a view into a wider row.
     ``max_keys`` (optional): a bound on the keys any of the tokens sees; with few tokens and many keys the
     keys of a token are then shared out over several blocks whose results a second kernel merges.
@@ -582,7 +595,8 @@ def attention_general(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_token
     ``v_cache`` None with ``v_dim``: the values are the first ``v_dim`` numbers of the key rows.
     ``sink`` float32 ``[n_heads]``: a score per head that stands in the softmax's denominator once, with no key
     and no value.  ``v_share`` > 1: so many consecutive key heads read one value head (``v_cache`` has
-    ``n_kv_heads / v_share`` heads): several maps of scores over the same values."""
+    ``n_kv_heads / v_share`` heads): several maps of scores over the same values.  ``out`` may be columns of a wider
+    matrix (its first ``n_heads * v_dim`` ones are written); ``out_scale``: a factor on all of them."""
     if not q.is_cuda or q.stride(-1) != 1:
         raise KernelError("attention: q must be a CUDA tensor with unit inner stride")
     if v_share < 1 or n_kv_heads % v_share or (v_share > 1 and v_cache is None):
@@ -598,7 +612,7 @@ def attention_general(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_token
         v_cache, v_row, inner = k_cache, head_dim, v_dim
     else:
         inner = v_cache.shape[3]
-    _need(out, "out", dims=2)
+    _need_rows(out, "out")
     out_wide = out.dtype == torch.float32 and q.dtype != torch.float32  # the sums unrounded, whatever the compute type
     if out.dtype != q.dtype and not out_wide:
         raise KernelError(f"attention: out must be of q's type or float32, not {out.dtype}")
@@ -618,7 +632,7 @@ def attention_general(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_token
         raise KernelError("attention: chunks take the place of a window")
     if n_heads % n_kv_heads:
         raise KernelError(f"attention: {n_heads} heads are not a multiple of {n_kv_heads} key/value heads")
-    if out.shape[0] < n_tokens or out.shape[1] != n_heads * v_dim:
+    if out.shape[0] < n_tokens or out.shape[1] < n_heads * v_dim:
         raise KernelError("attention: out does not fit")
     n_rel = 0
     if rel is not None:
@@ -641,21 +655,21 @@ def attention_general(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_token
     if max_keys > 2 * DECODE_CHUNK and blocks < 2 * n_sms(q.device):
         splits = min(16, (max_keys + DECODE_CHUNK - 1) // DECODE_CHUNK, max(1, 4 * n_sms(q.device) // blocks))
     if (keep_first or rel is not None or gate is not None or v_dim != head_dim or splits > 1 or chunk or v_row
-            or sink is not None or v_share > 1 or out_wide):
+            or sink is not None or v_share > 1 or out_wide or out_scale != 1.0):
         part = None
         if splits > 1:
             part = torch.empty(n_tokens * n_heads * splits * (v_dim + 2), dtype=torch.float32, device=q.device)
             global LAUNCHES
             LAUNCHES += 1  # the kernel that merges the splits
         _check(_fn("attention", "bn_attention_general_ex")(
-            _ptr(q), int(q_stride), _ptr(out), int(out.shape[1]), int(_code(q)), int(n_tokens), int(n_heads),
+            _ptr(q), int(q_stride), _ptr(out), int(out.stride(0)), int(_code(q)), int(n_tokens), int(n_heads),
             int(n_kv_heads), int(head_dim), int(v_dim), c_float(scale), int(window), int(keep_first), int(chunk), int(v_row),
             _ptr(rel), int(n_rel), _ptr(gate), int(gate_stride), _ptr(tok_seq), _ptr(tok_pos), _ptr(slots), _ptr(page_table),
             int(page_table.shape[1]), _ptr(k_cache), _ptr(v_cache), _ptr(part), int(splits), _ptr(sink), int(v_share),
-            int(out_wide), _stream()), "attention_general")
+            int(out_wide), c_float(out_scale), _stream()), "attention_general")
         return out
     _check(_fn("attention", "bn_attention_general")(
-        _ptr(q), int(q_stride), _ptr(out), int(out.shape[1]), int(_code(q)), int(n_tokens), int(n_heads),
+        _ptr(q), int(q_stride), _ptr(out), int(out.stride(0)), int(_code(q)), int(n_tokens), int(n_heads),
         int(n_kv_heads), int(head_dim), c_float(scale), int(window), _ptr(tok_seq), _ptr(tok_pos),
         _ptr(slots), _ptr(page_table), int(page_table.shape[1]), _ptr(k_cache), _ptr(v_cache), _stream()),
         "attention_general")
@@ -668,12 +682,12 @@ def attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_heads
                       k_cache: torch.Tensor, v_cache: torch.Tensor, *, keep_first: int = 0,
                       rel: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_stride: int = 0,
                       precise: bool = False, chunk: int = 0, v_dim: int = 0, sink: Optional[torch.Tensor] = None,
-                      v_share: int = 1) -> torch.Tensor:
+                      v_share: int = 1, out_scale: float = 1.0) -> torch.Tensor:
     """bfloat16 causal attention of runs of new tokens on the tensor cores; block i handles up to 64
     new tokens of sequence tile_seq[i] from its row tile_row0[i] on.  ``keep_first``, ``rel`` and ``gate`` as
     for ``attention_general``; a value head may have a width of its own (``v_cache``'s rows; with ``precise``); ``precise``: the softmax weights enter the second product with 16 bits of
     mantissa (as two bfloat16 terms) instead of 8.  ``chunk``, ``v_cache`` None with ``v_dim``, ``sink``, ``v_share``
-    and a float32 ``out`` as for ``attention_general``."""
+    a float32 ``out``, an ``out`` of columns and ``out_scale`` as for ``attention_general``."""
     if not q.is_cuda or q.stride(-1) != 1 or q.dtype != torch.bfloat16:
         raise KernelError("attention_prefill: q must be a bfloat16 CUDA tensor with unit inner stride")
     v_row = 0
@@ -683,7 +697,7 @@ def attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_heads
         v_cache, v_row, inner = k_cache, head_dim, v_dim
     else:
         inner = v_cache.shape[3]
-    _need(out, "out", dims=2)
+    _need_rows(out, "out")
     out_wide = out.dtype == torch.float32
     if out.dtype not in (torch.bfloat16, torch.float32):
         raise KernelError("attention_prefill: out must be bfloat16 or float32")
@@ -708,7 +722,7 @@ def attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_heads
         raise KernelError(f"attention_prefill: head_dim={head_dim}, value width {v_dim}, heads {n_heads}/{n_kv_heads} not supported")
     if v_dim != head_dim and not precise:
         raise KernelError("attention_prefill: a value width of its own is built for precise weights only")
-    if out.shape[1] != n_heads * v_dim or q_stride % 8:
+    if out.shape[1] < n_heads * v_dim or q_stride % 8:
         raise KernelError("attention_prefill: out or q_stride does not fit")
     n_rel = 0
     if rel is not None:
@@ -719,17 +733,17 @@ def attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_heads
     if gate is not None and (not gate.is_cuda or gate.dtype != torch.bfloat16 or gate.stride(-1) != 1
                              or gate.shape[-1] < n_heads or gate_stride <= 0):
         raise KernelError("attention_prefill: gate must be a bfloat16 CUDA view with unit inner stride and one number per head")
-    if keep_first or rel is not None or gate is not None or precise or chunk or v_row or sink is not None or v_share > 1 or out_wide:
+    if keep_first or rel is not None or gate is not None or precise or chunk or v_row or sink is not None or v_share > 1 or out_wide or out_scale != 1.0:
         _check(_fn("attention_prefill", "bn_attention_prefill_ex")(
-            _ptr(q), int(q_stride), _ptr(out), int(out.shape[1]), int(tile_seq.shape[0]), int(n_heads),
+            _ptr(q), int(q_stride), _ptr(out), int(out.stride(0)), int(tile_seq.shape[0]), int(n_heads),
             int(n_kv_heads), int(head_dim), int(v_dim), c_float(scale), int(window), int(keep_first), int(chunk), int(v_row),
             _ptr(rel), int(n_rel), _ptr(gate),
             int(gate_stride), int(bool(precise)), _ptr(tile_seq), _ptr(tile_row0), _ptr(seq_start), _ptr(seq_pos0), _ptr(slots),
             _ptr(page_table), int(page_table.shape[1]), _ptr(k_cache), _ptr(v_cache), _ptr(sink), int(v_share), int(out_wide),
-            _stream()), "attention_prefill")
+            c_float(out_scale), _stream()), "attention_prefill")
         return out
     _check(_fn("attention_prefill", "bn_attention_prefill")(
-        _ptr(q), int(q_stride), _ptr(out), int(out.shape[1]), int(tile_seq.shape[0]), int(n_heads),
+        _ptr(q), int(q_stride), _ptr(out), int(out.stride(0)), int(tile_seq.shape[0]), int(n_heads),
         int(n_kv_heads), int(head_dim), c_float(scale), int(window), _ptr(tile_seq), _ptr(tile_row0),
         _ptr(seq_start), _ptr(seq_pos0), _ptr(slots), _ptr(page_table), int(page_table.shape[1]), _ptr(k_cache),
         _ptr(v_cache), _stream()), "attention_prefill")
@@ -743,14 +757,19 @@ def attention_prefill_tc(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_he
                          scale: float, window: int, tile_seq: torch.Tensor, tile_row0: torch.Tensor,
                          seq_start: torch.Tensor, seq_pos0: torch.Tensor, slots: torch.Tensor, page_table: torch.Tensor,
                          k_cache: torch.Tensor, v_cache: torch.Tensor, *, precise: bool = False,
-                         sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                         sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_stride: int = 0,
+                         out_scale: float = 1.0) -> torch.Tensor:
     """bfloat16 causal attention of runs of new tokens on tcgen05 tensor cores with TMA-fed operands;
     block i handles up to 128 new tokens of sequence tile_seq[i] from its row tile_row0[i] on.
     Key and value widths up to 128 (a value head has the width of ``v_cache``'s rows).  ``precise``: the softmax weights
-    enter the value product with 16 bits of mantissa instead of 8; ``sink`` as for ``attention_general``."""
+    enter the value product with 16 bits of mantissa instead of 8; ``sink``, ``gate``, an ``out`` of columns and ``out_scale`` as for
+    ``attention_general``."""
     if not q.is_cuda or q.dim() != 2 or q.stride(-1) != 1 or q.stride(0) != q_stride or q.dtype != torch.bfloat16:
         raise KernelError("attention_prefill_tc: q must be a bfloat16 CUDA matrix with unit inner stride")
-    _need(out, "out", torch.bfloat16, 2)
+    _need_rows(out, "out", torch.bfloat16)
+    if gate is not None and (not gate.is_cuda or gate.dtype != torch.bfloat16 or gate.stride(-1) != 1
+                             or gate.shape[-1] < n_heads or gate_stride <= 0):
+        raise KernelError("attention_prefill_tc: gate must be a bfloat16 CUDA view with unit inner stride and one number per head")
     for t, nm in ((tile_seq, "tile_seq"), (tile_row0, "tile_row0"), (seq_start, "seq_start"), (seq_pos0, "seq_pos0"),
                   (slots, "slots")):
         _need(t, nm, torch.int32, 1)
@@ -767,17 +786,17 @@ def attention_prefill_tc(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_he
         _need(sink, "sink", torch.float32, 1)
         if sink.shape[0] != n_heads:
             raise KernelError(f"attention_prefill_tc: {sink.shape[0]} sink scores for {n_heads} heads")
-    if out.shape[1] != n_heads * v_dim or q_stride % 8 or n_heads * head_dim > q_stride or out.shape[0] < q.shape[0]:
+    if out.shape[1] < n_heads * v_dim or q_stride % 8 or n_heads * head_dim > q_stride or out.shape[0] < q.shape[0]:
         raise KernelError("attention_prefill_tc: out or q_stride does not fit")
-    if precise or sink is not None or v_dim != head_dim:
+    if precise or sink is not None or v_dim != head_dim or gate is not None or out_scale != 1.0:
         _check(_fn("attention_prefill_tc", "bn_attention_prefill_tc_ex")(
-            _ptr(q), int(q_stride), int(q.shape[0]), _ptr(out), int(out.shape[1]), int(tile_seq.shape[0]), int(n_heads),
-            int(n_kv_heads), int(head_dim), int(v_dim), c_float(scale), int(window), int(bool(precise)), _ptr(sink), _ptr(tile_seq),
-            _ptr(tile_row0), _ptr(seq_start), _ptr(seq_pos0), _ptr(slots), _ptr(page_table), int(page_table.shape[1]), _ptr(k_cache),
+            _ptr(q), int(q_stride), int(q.shape[0]), _ptr(out), int(out.stride(0)), int(tile_seq.shape[0]), int(n_heads),
+            int(n_kv_heads), int(head_dim), int(v_dim), c_float(scale), int(window), int(bool(precise)), _ptr(sink), _ptr(gate),
+            int(gate_stride), c_float(out_scale), _ptr(tile_seq), _ptr(tile_row0), _ptr(seq_start), _ptr(seq_pos0), _ptr(slots), _ptr(page_table), int(page_table.shape[1]), _ptr(k_cache),
             _ptr(v_cache), int(k_cache.shape[0]), _ptr(tc_status(q.device)), _stream()), "attention_prefill_tc")
         return out
     _check(_fn("attention_prefill_tc", "bn_attention_prefill_tc")(
-        _ptr(q), int(q_stride), int(q.shape[0]), _ptr(out), int(out.shape[1]), int(tile_seq.shape[0]),
+        _ptr(q), int(q_stride), int(q.shape[0]), _ptr(out), int(out.stride(0)), int(tile_seq.shape[0]),
         int(n_heads), int(n_kv_heads), int(head_dim), c_float(scale), int(window), _ptr(tile_seq), _ptr(tile_row0),
         _ptr(seq_start), _ptr(seq_pos0), _ptr(slots), _ptr(page_table), int(page_table.shape[1]), _ptr(k_cache),
         _ptr(v_cache), int(k_cache.shape[0]), _ptr(tc_status(q.device)), _stream()), "attention_prefill_tc")
@@ -1099,16 +1118,19 @@ USE_FUSED_NORM = True  # products of few rows add to the residual and prepare th
 
 
 ACT_SILU, ACT_GELU_TANH = 0, 1  # the gate's activation in a gated product (BN_ACT_* in common.cuh)
+ACT_RELU2 = 2  # the activation of a unit without a gate: the square of relu
 ACTIVATIONS = {"silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH}
 
 
 def linear_tc(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu: bool = False,
-              cluster: int = 0, sink: Optional[NormSink] = None, _checked: bool = False, act: int = 0):
+              cluster: int = 0, sink: Optional[NormSink] = None, _checked: bool = False, act: int = 0,
+              bias: Optional[torch.Tensor] = None):
     """x[M, K] . w[N, K]^T for M <= 64 in bfloat16 on tcgen05 tensor cores with TMA-fed operands.
     ``cluster`` blocks (1 to 8) share the inner dimension of each 128-row tile of w and add their
     parts up through distributed shared memory (0: chosen from the number of tiles).  ``x`` may be
     ``RowScaled``.  With ``sink`` the product is added to ``sink.residual`` in place and the result
-    is the ``RowScaled`` output of the norm that follows.  (``_checked``: ``linear`` has looked at w
+    is the ``RowScaled`` output of the norm that follows.  ``bias`` (float32, one number per row of w) is added to a plain
+    product, and ``act`` ACT_RELU2 then squares its positive part.  (``_checked``: ``linear`` has looked at w
     and at the sizes already.)"""
     scaled = x if isinstance(x, RowScaled) else None
     if scaled is not None:
@@ -1150,7 +1172,8 @@ def linear_tc(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swigl
     cols = N // 2 if swiglu else N
     out = torch.empty((M, cols), dtype=out_dtype, device=dev)
     _check(fn(c_void_p(x.data_ptr()), c_void_p(w.data_ptr()), c_void_p(out.data_ptr()), _DT[out_dtype], M, N, K, cols,
-              (2 | act << 8) if swiglu else 0, cluster, *row, _NULL, 0, _NULL, _NULL, 0, _tc_status_arg(dev), _stream()), "linear_tc")
+              (2 | act << 8) if swiglu else (act << 8 if act == ACT_RELU2 else 0), cluster, *row,
+              _NULL if bias is None else c_void_p(bias.data_ptr()), 0, _NULL, _NULL, 0, _tc_status_arg(dev), _stream()), "linear_tc")
     return out
 
 
@@ -1262,7 +1285,7 @@ def _own_gemm_fits(x, w: torch.Tensor, swiglu: bool, out_dtype, kind: str) -> bo
 
 
 def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu: bool = False,
-           partial_sums: bool = False, sink: Optional[NormSink] = None, act: int = 0):
+           partial_sums: bool = False, sink: Optional[NormSink] = None, act: int = 0, bias: Optional[torch.Tensor] = None):
     """x[M, K] . w[N, K]^T.  A weight kept in float32 makes the product float32 whatever x is.
 
     ``x`` may be ``RowScaled`` (the output of a norm that a product's epilogue prepared).  With
@@ -1273,13 +1296,21 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu: 
     ``swiglu``: w holds gate and up rows in alternating blocks of 8 and the result is
     act(gate) * up, ``[M, N / 2]`` (``act``: ACT_SILU or ACT_GELU_TANH).  ``partial_sums``: return the float32 partial sums
     ``[parts, M, N]`` of a product that split its inner dimension instead of their sum
-    (``add_rmsnorm`` can add them up); by default the product sums them itself.
+    (``add_rmsnorm`` can add them up); by default the product sums them itself.  ``bias``: float32 ``[N]``, added to a
+    plain product's rows before they are rounded; ``act`` ACT_RELU2 then takes the square of their positive part.
     """
     _need(w, "w", dims=2)
     if x.shape[1] != w.shape[1] or len(x.shape) != 2:
         raise KernelError(f"linear: x {tuple(x.shape)} and w {tuple(w.shape)} do not share the inner size")
     M, K = x.shape
     N = w.shape[0]
+    squared = act == ACT_RELU2
+    if bias is not None:
+        _need(bias, "bias", torch.float32, 1)
+        if bias.shape[0] != N:
+            raise KernelError(f"linear: {bias.shape[0]} biases for {N} rows")
+    if (bias is not None or squared) and (swiglu or partial_sums or sink is not None):
+        raise KernelError("linear: a bias or a unit without a gate goes with plain products only")
     few = w.dtype == torch.bfloat16 and K % 8 == 0 and (not swiglu or N % 16 == 0)
     small = few and M <= MMA_MAX_ROWS
     streams = few and M <= TC_MAX_ROWS and not partial_sums and USE_TCGEN05
@@ -1295,8 +1326,8 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu: 
         return add_rmsnorm(sink.residual, delta, sink.weight, sink.eps, normed)
     if isinstance(x, RowScaled):
         if fast:
-            return linear_tc(x, w, out_dtype=out_dtype or x.dtype, swiglu=swiglu, _checked=True, act=act)
-        if _own_gemm_fits(x.x, w, swiglu, out_dtype, "scaled") and not partial_sums:
+            return linear_tc(x, w, out_dtype=out_dtype or x.dtype, swiglu=swiglu, _checked=True, act=act, bias=bias)
+        if _own_gemm_fits(x.x, w, swiglu, out_dtype, "scaled") and not partial_sums and bias is None and not squared:
             return gemm_tc(x, w, out_dtype=out_dtype or x.dtype, swiglu=swiglu, act=act)
         x = x.dense()
     _need(x, "x", dims=2)
@@ -1304,14 +1335,14 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu: 
     if x.dtype != w.dtype:
         x = x.to(w.dtype)
     if streams:
-        return linear_tc(x, w, out_dtype=out_dtype, swiglu=swiglu, _checked=True, act=act)
-    if _own_gemm_fits(x, w, swiglu, out_dtype, "swiglu" if swiglu else "plain") and not partial_sums:
+        return linear_tc(x, w, out_dtype=out_dtype, swiglu=swiglu, _checked=True, act=act, bias=bias)
+    if _own_gemm_fits(x, w, swiglu, out_dtype, "swiglu" if swiglu else "plain") and not partial_sums and bias is None and not squared:
         return gemm_tc(x, w, out_dtype=out_dtype, swiglu=swiglu, act=act)
     if small:
         fn = _fn("linear_mma", "bn_linear_mma")
         splits = _mma_splits(M, N, K, n_sms(x.device))
         scratch, counters = _split_scratch(x.device)
-        tail = (_ptr(scratch), ctypes.c_longlong(scratch.numel()), _ptr(counters), int(counters.numel()), _stream())
+        tail = (_ptr(scratch), ctypes.c_longlong(scratch.numel()), _ptr(counters), int(counters.numel()), _ptr(bias), _stream())
         if swiglu:
             out = torch.empty((M, N // 2), dtype=out_dtype, device=x.device)
             _check(fn(_ptr(x), _ptr(w), _ptr(out), int(_DT[out_dtype]), int(M), int(N), int(K), int(N // 2),
@@ -1325,7 +1356,7 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu: 
         out = torch.empty((M, N), dtype=out_dtype, device=x.device)
         _check(fn(_ptr(x), _ptr(w), _ptr(out), int(_DT[out_dtype]), int(M), int(N), int(K), int(N), int(0),
                   int(splits), *tail), "linear_mma")
-        return out
+        return relu_squared(out) if squared else out
     if M <= SKINNY_MAX_ROWS and K % 8 == 0:
         out = torch.empty((M, N), dtype=out_dtype, device=x.device)
         # a matrix with few rows shares its inner dimension out over several blocks (a property of the matrix alone)
@@ -1335,7 +1366,7 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu: 
         partial = torch.empty((splits, M, N), dtype=torch.float32, device=x.device) if splits > 1 else None
         _check(_fn("linear", "bn_linear_skinny")(_ptr(x), _ptr(w), int(_code(w)), _ptr(out), int(_DT[out_dtype]),
                                                  int(M), int(N), int(K), int(N),
-                                                 _ptr(partial) if partial is not None else c_void_p(None), _stream()),
+                                                 _ptr(partial) if partial is not None else c_void_p(None), _ptr(bias), _stream()),
                "linear_skinny")
         if splits > 1:
             global LAUNCHES
@@ -1345,13 +1376,15 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu: 
         if w.dtype == torch.float32:
             if torch.backends.cuda.matmul.allow_tf32:
                 raise KernelError("float32 products need torch.backends.cuda.matmul.allow_tf32 = False")
-            product = lambda: torch.matmul(x, w.t())
+            product = lambda: torch.matmul(x, w.t()) if bias is None else torch.addmm(bias, x, w.t())
         elif out_dtype == torch.float32:
-            product = lambda: torch.mm(x, w.t(), out_dtype=torch.float32)
-        else:
-            product = lambda: torch.matmul(x, w.t())
+            product = lambda: torch.mm(x, w.t(), out_dtype=torch.float32) if bias is None else torch.mm(x, w.t(), out_dtype=torch.float32).add_(bias)
+        else:  # (biases that come from the file in the compute type lose nothing by going back to it)
+            product = lambda: torch.matmul(x, w.t()) if bias is None else torch.addmm(bias.to(w.dtype), x, w.t())
         out = product() if PROFILE is None else _timed("library.matmul", product)
         out = out if out.dtype == out_dtype else out.to(out_dtype)
+    if squared:
+        return relu_squared(out)
     if swiglu:
         res = torch.empty((M, N // 2), dtype=out.dtype, device=x.device)
         return glu_mul(out, res, act)
@@ -1639,11 +1672,12 @@ def gated_state_floats(heads: int, groups: int, dim: int, vdim: int, taps: int) 
     return (n + 3) // 4 * 4
 
 
-def gated_state(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: torch.Tensor, a_off: int, b_off: int,
-                conv_w: torch.Tensor, conv_b: Optional[torch.Tensor], dt_bias: torch.Tensor, a_log: torch.Tensor,
+def gated_state(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: Optional[torch.Tensor], a_off: int, b_off: int,
+                conv_w: Optional[torch.Tensor], conv_b: Optional[torch.Tensor], dt_bias: Optional[torch.Tensor], a_log: Optional[torch.Tensor],
                 skip: Optional[torch.Tensor], state: torch.Tensor, tok_seq: torch.Tensor, seq_start: torch.Tensor,
                 seq_pos0: torch.Tensor, slots: torch.Tensor, n_seqs: int, heads: int, groups: int, dim: int, vdim: int,
-                one_token: bool, tile_seq: Optional[torch.Tensor] = None, tile_row0: Optional[torch.Tensor] = None) -> torch.Tensor:
+                one_token: bool, tile_seq: Optional[torch.Tensor] = None, tile_row0: Optional[torch.Tensor] = None,
+                log_decay: Optional[torch.Tensor] = None) -> torch.Tensor:
     """A matrix state per head over the new tokens of every sequence, from and into ``state`` ``[slots,
     gated_state_floats]`` (float32), under one decay per head and token.  ``proj`` ``[T, n]``: rows with the channels of
     q and k (``groups * dim`` each) and v (``heads * vdim``) at their offsets; each channel passes a causal convolution
@@ -1653,25 +1687,31 @@ def gated_state(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: t
     softplus(a + ``dt_bias``), b = sigmoid(.); S <- e^l S; u = b (v - S^T k); S <- S + k u^T; o = S^T q.
     ``b_off`` < 0, the state-space update: b = softplus(a + ``dt_bias``), l = -exp(``a_log``) b;
     S <- e^l S + b k v^T; o = S^T q + ``skip`` v.
+    ``log_decay`` (float32 ``[heads]``; ``b_off`` < 0): the latter with these log decays for every token and b = 1; ``gates``,
+    ``dt_bias`` and ``a_log`` are None.  ``conv_w`` None: no convolution, SiLU alone.
     ``one_token``: every sequence brings one token (one launch does it all).  ``tile_seq`` / ``tile_row0``: the runs of 64
     new tokens (sequence, first row); with them the recurrence goes chunk by chunk instead of token by token (``dim`` a
     multiple of four).  Returns o, float32 ``[T, heads * vdim]``."""
     _need(proj, "proj", dims=2)
-    _need(conv_w, "conv_w", torch.float32, 2)
+    n_ch = 2 * groups * dim + heads * vdim
+    if conv_w is not None:
+        _need(conv_w, "conv_w", torch.float32, 2)
     _need(state, "state", torch.float32, 2)
-    for t, nm, n in ((dt_bias, "dt_bias", heads), (a_log, "a_log", heads), (skip, "skip", heads), (conv_b, "conv_b", conv_w.shape[1])):
+    if log_decay is None and (gates is None or dt_bias is None or a_log is None) or log_decay is not None and b_off >= 0:
+        raise KernelError("gated_state: decays come from gates, or (without a delta rule) from log_decay")
+    for t, nm, n in ((dt_bias, "dt_bias", heads), (a_log, "a_log", heads), (skip, "skip", heads), (conv_b, "conv_b", n_ch), (log_decay, "log_decay", heads)):
         if t is not None:
             _need(t, nm, torch.float32, 1)
             if t.shape[0] != n:
                 raise KernelError(f"gated_state: {nm} holds {t.shape[0]} numbers, {n} are needed")
     for t, nm in ((tok_seq, "tok_seq"), (seq_start, "seq_start"), (seq_pos0, "seq_pos0"), (slots, "slots")):
         _need(t, nm, torch.int32, 1)
-    T, taps = tok_seq.shape[0], conv_w.shape[0]
+    T, taps = tok_seq.shape[0], conv_w.shape[0] if conv_w is not None else 1
     n_qk, n_v = groups * dim, heads * vdim
-    if (not gates.is_cuda or gates.dtype != torch.float32 or gates.dim() != 2 or gates.stride(1) != 1 or gates.shape[0] < T
+    if gates is not None and (not gates.is_cuda or gates.dtype != torch.float32 or gates.dim() != 2 or gates.stride(1) != 1 or gates.shape[0] < T
             or max(a_off, b_off) + heads > gates.shape[1]):
         raise KernelError("gated_state: gates must be a float32 CUDA matrix with unit inner stride that holds the pre-activations")
-    if (conv_w.shape[1] != 2 * n_qk + n_v or proj.shape[0] < T or state.shape[1] != gated_state_floats(heads, groups, dim, vdim, taps)
+    if (conv_w is not None and conv_w.shape[1] != n_ch or proj.shape[0] < T or state.shape[1] != gated_state_floats(heads, groups, dim, vdim, taps)
             or seq_start.shape[0] < n_seqs + 1 or seq_pos0.shape[0] < n_seqs or slots.shape[0] < n_seqs or heads % groups
             or (one_token and T != n_seqs)):
         raise KernelError("gated_state: sizes do not fit")
@@ -1679,9 +1719,9 @@ def gated_state(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: t
         raise KernelError(f"gated_state: dim={dim} (at most {GATED_STATE_MAX_DIM}) or {taps} taps (at most {GATED_STATE_MAX_TAPS})")
     dev = proj.device
     out = torch.empty((T, n_v), dtype=torch.float32, device=dev)
-    args = (_ptr(proj), int(_code(proj)), int(T), int(proj.shape[1]), int(q_off), int(k_off), int(v_off), c_void_p(gates.data_ptr()),
-            int(gates.stride(0)), int(a_off), int(b_off), int(groups), int(heads), int(dim), int(vdim), int(taps), _ptr(conv_w),
-            _ptr(conv_b), _ptr(dt_bias), _ptr(a_log), _ptr(skip), c_float(dim ** -0.5), _ptr(state),
+    args = (_ptr(proj), int(_code(proj)), int(T), int(proj.shape[1]), int(q_off), int(k_off), int(v_off), _ptr(gates),
+            int(gates.stride(0)) if gates is not None else 0, int(a_off), int(b_off), int(groups), int(heads), int(dim), int(vdim), int(taps), _ptr(conv_w),
+            _ptr(conv_b), _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(log_decay), c_float(dim ** -0.5), _ptr(state),
             ctypes.c_longlong(state.shape[1]), _ptr(tok_seq), _ptr(seq_start), _ptr(seq_pos0), _ptr(slots), int(n_seqs))
     if one_token:
         _check(_fn("gated_state", "bn_gated_state_token")(*args, _ptr(out), _stream()), "gated_state_token")
@@ -1707,9 +1747,10 @@ def gated_state(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: t
 
 
 def state_output(o: torch.Tensor, z: torch.Tensor, gain: torch.Tensor, parts: int, eps: float, gate_first: bool,
-                 dtype: torch.dtype) -> torch.Tensor:
+                 dtype: torch.dtype, logistic: bool = False) -> torch.Tensor:
     """Rows of o (float32) in ``parts`` equal parts: o silu(z) divided by its root mean square per part, times ``gain``
-    (``gate_first``), or o divided by its root mean square per part, times ``gain``, times silu(z).  ``z``: a view of
+    (``gate_first``), or o divided by its root mean square per part, times ``gain``, times silu(z) (``logistic``: the logistic
+    function of z).  ``z``: a view of
     o's width with unit inner stride; ``gain`` float32, as long as a row or as a part (shared by the parts)."""
     _need(o, "o", torch.float32, 2)
     _need(gain, "gain", torch.float32, 1)
@@ -1720,11 +1761,80 @@ def state_output(o: torch.Tensor, z: torch.Tensor, gain: torch.Tensor, parts: in
     out = torch.empty((n, row), dtype=dtype, device=o.device)
     _check(_fn("gated_state", "bn_state_output")(_ptr(o), c_void_p(z.data_ptr()), int(_code(z)), int(z.stride(0)), _ptr(gain),
                                                  int(gain.shape[0]), int(_DT[dtype]), int(n), int(parts), int(row // parts),
-                                                 c_float(eps), int(bool(gate_first)), _ptr(out), _stream()), "state_output")
+                                                 c_float(eps), int(bool(gate_first)), int(bool(logistic)), _ptr(out), _stream()), "state_output")
     return out
 
 
 # ---- a residual of several streams ----------------------------------------------------------------
+def gated_linear_floats(width: int, taps: int) -> int:
+    """Floats of one sequence's state: the recurrence's, then a ring of the convolution's last ``taps`` inputs."""
+    n = width * (1 + (taps if taps > 1 else 0))
+    return (n + 3) // 4 * 4
+
+
+GATED_LINEAR_MAX_TAPS = 16
+GATED_LINEAR_MAX_PART = 6144  # channels per part: eight sequences of them fit a block's shared memory
+
+
+def gated_linear(x: torch.Tensor, y: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, w_gates: torch.Tensor,
+                 gate_b: torch.Tensor, lam: torch.Tensor, state: torch.Tensor, tok_seq: torch.Tensor, seq_start: torch.Tensor,
+                 seq_pos0: torch.Tensor, slots: torch.Tensor, n_seqs: int, out: torch.Tensor, *, scale: float = 1.0, tail: int = 0,
+                 one_token: bool = False, tile_seq: Optional[torch.Tensor] = None, tile_row0: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """A real-gated linear recurrence per channel over the new tokens of every sequence, from and into ``state`` ``[slots,
+    gated_linear_floats]`` (float32).  ``x`` and ``y`` are matrices of ``width`` columns (they may be columns of one wider
+    matrix): u = a causal convolution of x (``conv_w`` float32 ``[taps, width]``, ``conv_b``), rounded to x's type;
+    [r | i] = the logistic function of W u + ``gate_b`` part by part (``w_gates`` ``[parts, 2 part, part]`` in x's type, r's rows
+    first; ``gate_b`` float32 ``[parts, 2 part]``); l = -8 r softplus(``lam``); S <- e^l S + sqrt(1 - e^(2 l)) i u.
+    ``out`` (columns of a matrix in x's type) receives ``scale`` * gelu_tanh(y) * S and, in ``tail`` more columns, 1, 1, 0, ...
+    ``one_token``: every sequence brings one token (one launch); else ``tile_seq`` / ``tile_row0`` are the step's runs of 64
+    new tokens."""
+    parts, rows, part = w_gates.shape
+    width, taps, T = parts * part, conv_w.shape[0], tok_seq.shape[0]
+    for t, nm in ((x, "x"), (y, "y"), (out, "out")):
+        _need_rows(t, nm, w_gates.dtype)
+    _need(w_gates, "w_gates", dims=3)
+    _need(state, "state", torch.float32, 2)
+    for t, nm, shape in ((conv_w, "conv_w", (taps, width)), (conv_b, "conv_b", (width,)), (gate_b, "gate_b", (parts, 2 * part)),
+                         (lam, "lam", (width,))):
+        _need(t, nm, torch.float32)
+        if tuple(t.shape) != shape:
+            raise KernelError(f"gated_linear: {nm} {tuple(t.shape)} is not {shape}")
+    for t, nm in ((tok_seq, "tok_seq"), (seq_start, "seq_start"), (seq_pos0, "seq_pos0"), (slots, "slots")):
+        _need(t, nm, torch.int32, 1)
+    if (rows != 2 * part or x.shape[1] != width or y.shape[1] != width or x.stride(0) != y.stride(0) or min(x.shape[0], y.shape[0], out.shape[0]) < T
+            or out.shape[1] < width + tail or state.shape[1] != gated_linear_floats(width, taps) or seq_start.shape[0] < n_seqs + 1
+            or seq_pos0.shape[0] < n_seqs or slots.shape[0] < n_seqs or (one_token and T != n_seqs)):
+        raise KernelError("gated_linear: sizes do not fit")
+    if part > GATED_LINEAR_MAX_PART or not 1 <= taps <= GATED_LINEAR_MAX_TAPS:
+        raise KernelError(f"gated_linear: parts of {part} channels (at most {GATED_LINEAR_MAX_PART}) or {taps} taps (1 to {GATED_LINEAR_MAX_TAPS})")
+    args = (_ptr(x), _ptr(y), int(_code(x)), int(T), int(x.stride(0)), int(width), int(parts), int(taps), _ptr(conv_w), _ptr(conv_b),
+            _ptr(gate_b), _ptr(lam), _ptr(state), ctypes.c_longlong(state.shape[1]), _ptr(tok_seq), _ptr(seq_start), _ptr(seq_pos0),
+            _ptr(slots), int(n_seqs), c_float(scale), _ptr(out), int(out.stride(0)), int(tail))
+    if one_token:
+        _check(_fn("gated_linear", "bn_gated_linear_token")(*args, _ptr(w_gates), _stream()), "gated_linear_token")
+        return out
+    _need(tile_seq, "tile_seq", torch.int32, 1)
+    _need(tile_row0, "tile_row0", torch.int32, 1)
+    u = torch.empty((T, width), dtype=x.dtype, device=x.device)
+    _check(_fn("gated_linear", "bn_gated_linear_conv")(*args, _ptr(u), _stream()), "gated_linear_conv")
+    up = u.view(T, parts, part).transpose(0, 1)
+    if x.dtype == torch.float32:
+        if torch.backends.cuda.matmul.allow_tf32:
+            raise KernelError("float32 products need torch.backends.cuda.matmul.allow_tf32 = False")
+        product = lambda: torch.bmm(up, w_gates.transpose(1, 2))
+    else:
+        product = lambda: torch.bmm(up, w_gates.transpose(1, 2), out_dtype=torch.float32)
+    gates = product() if PROFILE is None else _timed("library.bmm", product)
+    gates = gates.contiguous()
+    n_pieces = tile_seq.shape[0]
+    sums = torch.empty((n_pieces, 2, width), dtype=torch.float32, device=x.device)
+    global LAUNCHES
+    LAUNCHES += 2  # the pieces alone, the states carried through them, the pieces again
+    _check(_fn("gated_linear", "bn_gated_linear_scan")(*args, _ptr(u), _ptr(gates), _ptr(tile_seq), _ptr(tile_row0), int(n_pieces),
+                                                       _ptr(sums), _stream()), "gated_linear_scan")
+    return out
+
+
 MAX_STREAMS = 16
 STREAMS_MAX_TAPS = 16
 STREAMS_MAX_WIDTH = (200 * 1024) // 4
@@ -1878,26 +1988,38 @@ def sigmoid_attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor,
 
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, top: int, renormalise: bool = False, softmax: bool = False,
-              weight_scale: float = 1.0, sum_eps: float = 0.0, bias: Optional[torch.Tensor] = None):
+              weight_scale: float = 1.0, sum_eps: float = 0.0, bias: Optional[torch.Tensor] = None,
+              correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1, gate: bool = False):
     """Per token the ``top`` experts with the largest router logits (float32 products, plus ``bias``), and their scores as
     weights: the logistic function of each logit, or with ``softmax`` the softmax over all experts; divided by
     the chosen ones' sum (+ ``sum_eps``) with ``renormalise``, then times ``weight_scale``:
-    ``(ids int32 [T, top], weights float32 [T, top])``."""
+    ``(ids int32 [T, top], weights float32 [T, top])``.  ``correction`` (float32, one number per expert): the choice goes by
+    score + correction, and with ``keep`` < ``groups`` only among the experts of the ``keep`` best of ``groups`` equal groups of
+    neighbours (a group counts by its best); the weights stay the scores.  ``gate``: the router's last row is no expert; a
+    third result holds the logistic function of its product, float32 ``[T]``."""
     _need(h, "h", dims=2)
     _need(w_router, "w_router", dims=2)
-    if w_router.shape[1] != h.shape[1] or not 0 < top <= min(w_router.shape[0], 32) or w_router.shape[0] > 1024:
+    n = w_router.shape[0] - int(bool(gate))
+    if w_router.shape[1] != h.shape[1] or not 0 < top <= min(n, 32) or n > 1024:
         raise KernelError(f"moe_route: router {tuple(w_router.shape)}, top {top} do not fit rows of width {h.shape[1]}")
     if bias is not None:
         _need(bias, "bias", torch.float32, 1)
-        if bias.shape[0] != w_router.shape[0]:
-            raise KernelError(f"moe_route: {bias.shape[0]} biases for {w_router.shape[0]} experts")
+        if bias.shape[0] != n:
+            raise KernelError(f"moe_route: {bias.shape[0]} biases for {n} experts")
+    if correction is not None:
+        _need(correction, "correction", torch.float32, 1)
+        if correction.shape[0] != n:
+            raise KernelError(f"moe_route: {correction.shape[0]} corrections for {n} experts")
+    if groups < 1 or n % groups or not 0 < keep <= groups or (keep < groups and (correction is None or keep * (n // groups) < top)):
+        raise KernelError(f"moe_route: {n} experts cannot be chosen {top} at a time from {keep} of {groups} groups")
+    g = torch.empty(h.shape[0], dtype=torch.float32, device=h.device) if gate else None
     ids = torch.empty((h.shape[0], top), dtype=torch.int32, device=h.device)
     weights = torch.empty((h.shape[0], top), dtype=torch.float32, device=h.device)
     _check(_fn("moe", "bn_moe_route_ex")(_ptr(h), int(_code(h)), int(h.shape[0]), int(h.shape[1]), _ptr(w_router),
-                                         int(_code(w_router)), _ptr(bias), int(w_router.shape[0]), int(top), int(bool(renormalise)),
-                                         int(bool(softmax)), c_float(weight_scale), c_float(sum_eps), _ptr(ids), _ptr(weights),
-                                         _stream()), "moe_route")
-    return ids, weights
+                                         int(_code(w_router)), _ptr(bias), int(n), int(top), int(bool(renormalise)),
+                                         int(bool(softmax)), c_float(weight_scale), c_float(sum_eps), _ptr(correction), int(groups),
+                                         int(keep), _ptr(g), _ptr(ids), _ptr(weights), _stream()), "moe_route")
+    return (ids, weights, g) if gate else (ids, weights)
 
 
 def moe_table_route(tokens: torch.Tensor, table: torch.Tensor, top: int, n_experts: int):
@@ -1927,10 +2049,12 @@ def moe_few_fits(width: int, top: int, ff: int) -> bool:
 
 def moe_experts_few(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
                     w_down: torch.Tensor, limit: float, slope: float, scale_input: bool,
-                    add: Optional[torch.Tensor] = None, act: int = -1) -> torch.Tensor:
+                    add: Optional[torch.Tensor] = None, act: int = -1, add_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The chosen experts of every token, streamed once per (token, expert): float32 ``[T, width]``, the sum over
     a token's experts plus ``add``.  The weight multiplies the expert's input (``scale_input``) or its output.
-    ``act`` < 0: the clamped unit with ``limit`` and ``slope``; ACT_SILU / ACT_GELU_TANH: act(gate) * up.
+    ``act`` < 0: the clamped unit with ``limit`` and ``slope``; ACT_SILU / ACT_GELU_TANH: act(gate) * up; ACT_RELU2: no gate,
+    the square of relu(up), and ``w_gate_up`` is ``[experts, ff, width]``.  Ids from the number of experts on are identity experts:
+    their output is h itself.  ``add_scale`` (float32 ``[T]``): a factor on each row of ``add``.
     ``w_gate_up`` ``[experts, 2 * ff, width]`` holds an expert's gate rows and then its up rows, ``w_down``
     ``[experts, width, ff]``; both in h's type."""
     _need(h, "h", dims=2)
@@ -1940,32 +2064,38 @@ def moe_experts_few(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w
     top = ids.shape[1]
     _need(w_gate_up, "w_gate_up", h.dtype, 3)
     _need(w_down, "w_down", h.dtype, 3)
-    E, ff = w_gate_up.shape[0], w_gate_up.shape[1] // 2
-    if (tuple(w_gate_up.shape) != (E, 2 * ff, width) or tuple(w_down.shape) != (E, width, ff)
+    per = 1 if act == ACT_RELU2 else 2
+    E, ff = w_gate_up.shape[0], w_gate_up.shape[1] // per
+    if (tuple(w_gate_up.shape) != (E, per * ff, width) or tuple(w_down.shape) != (E, width, ff)
             or tuple(ids.shape) != (T, top) or tuple(weights.shape) != (T, top) or not moe_few_fits(width, top, ff)):
         raise KernelError("moe_experts_few: sizes do not fit")
     if add is not None:
         _need(add, "add", dims=2)
         if tuple(add.shape) != (T, width):
             raise KernelError("moe_experts_few: add does not fit")
+    if add_scale is not None:
+        _need(add_scale, "add_scale", torch.float32, 1)
+        if add_scale.shape[0] != T:
+            raise KernelError("moe_experts_few: add_scale does not fit")
     y = torch.empty((T * top, ff), dtype=h.dtype, device=h.device)
-    w_up = w_gate_up[:, ff:]
+    w_up = w_gate_up[:, ff:] if per == 2 else w_gate_up
     _check(_fn("moe", "bn_moe_gate_up_ex")(_ptr(h), int(_code(h)), int(T), int(width), _ptr(ids), _ptr(weights),
-                                           int(bool(scale_input)), _ptr(w_gate_up), c_void_p(w_up.data_ptr()),
-                                           ctypes.c_longlong(2 * ff * width), int(ff), int(top), c_float(limit),
-                                           c_float(slope), int(act), _ptr(y), _stream()), "moe_gate_up")
+                                           int(bool(scale_input)), _ptr(w_gate_up if per == 2 else None), c_void_p(w_up.data_ptr()),
+                                           ctypes.c_longlong(per * ff * width), int(ff), int(top), c_float(limit),
+                                           c_float(slope), int(act), int(E), _ptr(y), _stream()), "moe_gate_up")
     out = torch.empty((T, width), dtype=torch.float32, device=h.device)
     _check(_fn("moe", "bn_moe_down")(_ptr(y), int(_code(y)), int(T), int(ff), _ptr(ids), _ptr(weights),
                                      int(not scale_input), _ptr(w_down), int(width), int(top), _ptr(add),
-                                     int(_code(add) if add is not None else 0), _ptr(out), _stream()), "moe_down")
+                                     int(_code(add) if add is not None else 0), _ptr(add_scale), int(E), _ptr(h), _ptr(out), _stream()),
+           "moe_down")
     return out
 
 
 def moe_count(ids: torch.Tensor, n_experts: int) -> torch.Tensor:
-    """int32 ``[experts]``: how many (token, expert) items chose each expert."""
+    """int32 ``[experts]``: how many (token, expert) items chose each expert (identity experts behind them are not counted)."""
     _need(ids, "ids", torch.int32, 2)
     counts = torch.zeros(n_experts, dtype=torch.int32, device=ids.device)
-    _check(_fn("moe", "bn_moe_count")(_ptr(ids), int(ids.numel()), _ptr(counts), _stream()), "moe_count")
+    _check(_fn("moe", "bn_moe_count")(_ptr(ids), int(ids.numel()), int(n_experts), _ptr(counts), _stream()), "moe_count")
     return counts
 
 
@@ -1975,7 +2105,8 @@ def moe_sort(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, counts: 
     Item i went to row ``place[i]`` of ``x_sorted``, which holds its token's row of h (times its weight with
     ``scale_input``).  ``cap`` = 0: the experts' rows are packed, expert e's are rows ``offsets[e] ..
     offsets[e + 1]`` of ``[T * top, width]``.  ``cap`` > 0 (at least the largest of ``counts``): expert e's rows
-    begin at ``e * cap`` of ``[experts * cap, width]``; rows that no item took hold nothing."""
+    begin at ``e * cap`` of ``[experts * cap, width]``; rows that no item took hold nothing.  Items of identity experts (ids from
+    the number of ``counts`` on) get the place -1."""
     _need(h, "h", dims=2)
     _need(ids, "ids", torch.int32, 2)
     _need(weights, "weights", torch.float32, 2)
@@ -1996,9 +2127,10 @@ def moe_sort(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, counts: 
 
 
 def moe_gather(y_sorted: torch.Tensor, place: torch.Tensor, weights: torch.Tensor, scale_output: bool,
-               add: Optional[torch.Tensor] = None) -> torch.Tensor:
+               add: Optional[torch.Tensor] = None, add_scale: Optional[torch.Tensor] = None,
+               h: Optional[torch.Tensor] = None) -> torch.Tensor:
     """float32 ``[T, width]``: per token the sum of its experts' rows of ``y_sorted`` (times their weight with
-    ``scale_output``), plus ``add``."""
+    ``scale_output``), plus ``add`` (its rows times ``add_scale``, if given).  A place of -1 stands for the token's row of ``h``."""
     _need(y_sorted, "y_sorted", dims=2)
     _need(place, "place", torch.int32, 1)
     _need(weights, "weights", torch.float32, 2)
@@ -2010,10 +2142,16 @@ def moe_gather(y_sorted: torch.Tensor, place: torch.Tensor, weights: torch.Tenso
         _need(add, "add", dims=2)
         if tuple(add.shape) != (T, width):
             raise KernelError("moe_gather: add does not fit")
+    if add_scale is not None:
+        _need(add_scale, "add_scale", torch.float32, 1)
+    if h is not None:
+        _need(h, "h", y_sorted.dtype, 2)
+        if tuple(h.shape) != (T, width):
+            raise KernelError("moe_gather: h does not fit")
     out = torch.empty((T, width), dtype=torch.float32, device=y_sorted.device)
     _check(_fn("moe", "bn_moe_gather")(_ptr(y_sorted), int(_code(y_sorted)), int(T), int(width), _ptr(place), _ptr(weights),
                                        int(bool(scale_output)), int(top), _ptr(add), int(_code(add) if add is not None else 0),
-                                       _ptr(out), _stream()), "moe_gather")
+                                       _ptr(add_scale), _ptr(h), _ptr(out), _stream()), "moe_gather")
     return out
 
 

@@ -123,6 +123,14 @@ class Model:
             per_part.setdefault(id(part), (part, {}))[1][name] = tensors[path]
         for part, group in per_part.values():
             part.bind(group)
+        def settle(part) -> None:
+            for child in part.children().values():
+                settle(child)
+            part.bound()
+
+        for part in (*self.blocks, self.final_norm, self.embedding_norm, self.head_part):
+            if part is not None:
+                settle(part)
         self.embedding = tensors["embedding.table"]
         self.head = tensors["head.weight"] if not self.spec.tie_embeddings else self.embedding
         self._bad_token = torch.zeros(1, dtype=torch.int32, device=self.device)

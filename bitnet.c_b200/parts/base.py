@@ -117,6 +117,9 @@ class Part:
         if tensors:
             raise ValueError(f"{type(self).__name__} takes no parameters, got {sorted(tensors)}")
 
+    def bound(self) -> None:
+        """Called once when this part's and all of its children's parameters are in place (children first)."""
+
     def children(self) -> Dict[str, "Part"]:
         return {}
 
@@ -139,6 +142,14 @@ class Mixer(Part):
     # itself and returns the output of the norm that follows (``ops.linear(..., sink=sink)``)
     # instead of the delta.
     accepts_sink = False
+    # A mixer that sets ``shares_products`` is one product of its input, an inner part, and one product of what that leaves,
+    # and lets a part that runs it beside another mixer take both products together: ``w_in`` / ``b_in`` and ``w_o`` / ``b_o``
+    # (a bias: float32 or None; the rows of ``w_in`` a multiple of 8), ``inner_dim`` the columns between them, and
+    # ``inner(proj, at, out, out_at, factor, ctx, kv, state, tail=0)``: proj's columns from ``at`` (a multiple of 8) on are the
+    # first product; ``factor`` times the inner result goes to out's columns from ``out_at`` on, and behind it, where
+    # ``leaves_tail`` is set, ``tail`` more columns 1, 1, 0, 0, ...
+    shares_products = False
+    leaves_tail = False
 
     def cache_request(self) -> Optional[KvRequest]:
         return None

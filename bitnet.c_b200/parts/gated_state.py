@@ -1,7 +1,8 @@
 """Recurrent mixers with a matrix state per head under one decay per head and token: the gated delta rule with
-head-wise decays, and the Mamba-2 state-space layer."""
+head-wise decays, the Mamba-2 state-space layer, and linear attention under fixed decays."""
 from __future__ import annotations
 
+import math
 from typing import Dict, Optional, Sequence, Tuple
 
 import torch
@@ -12,7 +13,7 @@ from .registry import register_mixer
 
 
 class GatedStateMixer(Mixer):
-    """What both mixers share: one stacked product of the mixer's input whose last rows are the heads' gate
+    """What the mixers share: one stacked product of the mixer's input whose last rows are the heads' gate
     pre-activations, the recurrence from the sequence's state (matrices, and the convolutions' last inputs, float32),
     a gated norm and the output projection.  Steps of one token per sequence take the whole product in float32 and
     the recurrence in one launch; runs of tokens in bfloat16 take the gates' rows as a float32 product of their own
@@ -22,6 +23,7 @@ class GatedStateMixer(Mixer):
     graph_safe = True
     CHUNKED_MIN_TOKENS = 16  # steps with a run of so many new tokens take the recurrence chunk by chunk
     n_heads = n_groups = dim = vdim = taps = 0  # set by the mixers
+    log_decay = None  # fixed log decays per head, in place of gates
 
     def _check_sizes(self) -> None:
         if min(self.n_heads, self.n_groups, self.dim, self.vdim) <= 0 or self.n_heads % self.n_groups:
@@ -56,7 +58,8 @@ class GatedStateMixer(Mixer):
         tiles = dict(tile_seq=ctx.tile_seq, tile_row0=ctx.tile_row0) if chunked else {}
         o = ops.gated_state(proj, self.q_off, self.k_off, self.v_off, gates, self.a_off, self.b_off, self.conv_w, self.conv_b,
                             self.dt_bias, self.a_log, self.skip, state, ctx.tok_seq, ctx.seq_start, ctx.seq_pos0, ctx.slots,
-                            ctx.n_seqs, self.n_heads, self.n_groups, self.dim, self.vdim, one_token=ctx.decode, **tiles)
+                            ctx.n_seqs, self.n_heads, self.n_groups, self.dim, self.vdim, one_token=ctx.decode,
+                            log_decay=self.log_decay, **tiles)
         ctx.tap("state_raw", o)
         return o
 
@@ -152,4 +155,49 @@ class Mamba2(GatedStateMixer):
         proj, gates = self._project(h, ctx)
         o = self._recur(proj, gates, ctx, state)
         y = ops.state_output(o, proj[:, : self.inner], self.gain, s.norm_groups, s.norm_eps, True, self.build.dtype)
+        return ops.linear(y, self.w_o, out_dtype=torch.float32)
+
+
+@register_mixer("lightning")
+class Lightning(GatedStateMixer):
+    """q, k (heads x dim) and v (heads x vdim) = SiLU(W h); per head, from the sequence's state S (zero at first), under one
+    fixed decay per head
+
+        S = decay S_before + k v^T;  o = S^T q
+
+    Then one RMS norm over all heads with a gain, the logistic function of W_g h, and the output projection."""
+
+    NO_DECAY_LEFT = -100.0  # log decay of a head that forgets everything: e^-100 is zero in single precision
+
+    def __init__(self, spec, build):
+        super().__init__(spec, build)
+        self.n_heads = self.n_groups = spec.n_heads
+        self.dim, self.vdim, self.taps = spec.head_dim, spec.v_head_dim, 1
+        self._check_sizes()
+        if len(spec.decay) != spec.n_heads or not all(0.0 <= d <= 1.0 for d in spec.decay):
+            raise ValueError(f"lightning: one decay from 0 to 1 for each of {spec.n_heads} heads, not {spec.decay!r}")
+        self.w_in: Optional[torch.Tensor] = None
+
+    def params(self) -> Dict[str, ParamSpec]:
+        s = self.spec
+        qk, vv = s.n_heads * s.head_dim, s.n_heads * s.v_head_dim
+        return {"q": ParamSpec((qk, s.width)), "k": ParamSpec((qk, s.width)), "v": ParamSpec((vv, s.width)),
+                "g": ParamSpec((vv, s.width)), "o": ParamSpec((s.width, vv)), "norm": ParamSpec((vv,), init="ones")}
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        s = self.spec
+        qk, vv = s.n_heads * s.head_dim, s.n_heads * s.v_head_dim
+        self._stack([tensors[n] for n in ("q", "k", "v", "g")], 0)
+        self.q_off, self.k_off, self.v_off, self.g_off = 0, qk, 2 * qk, 2 * qk + vv
+        self.a_off, self.b_off = 0, -1
+        self.conv_w = self.conv_b = self.dt_bias = self.a_log = self.skip = None
+        self.log_decay = torch.tensor([max(math.log(d), self.NO_DECAY_LEFT) if d > 0 else self.NO_DECAY_LEFT for d in s.decay],
+                                      dtype=torch.float32, device=self.w_in.device)
+        self.gain, self.w_o = tensors["norm"].float().contiguous(), tensors["o"]
+
+    def forward(self, h, ctx, kv, state):
+        s = self.spec
+        proj = ops.linear(h, self.w_in, out_dtype=self.build.dtype)
+        o = self._recur(proj, None, ctx, state)
+        y = ops.state_output(o, proj[:, self.g_off: self.g_off + o.shape[1]], self.gain, 1, s.norm_eps, False, self.build.dtype, logistic=True)
         return ops.linear(y, self.w_o, out_dtype=torch.float32)

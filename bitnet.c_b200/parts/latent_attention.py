@@ -29,7 +29,10 @@ class LatentAttention(Mixer):
     Runs of new tokens whose key rows are too wide for the tensor-core kernel (more than 256 numbers) take the
     other order: the rows every new token sees are read back from the cache, W_uk and W_uv make per-head keys
     [W_uk c | k_rot] and values of them (two products over all those rows), which go into scratch pages of the
-    step, and the tensor-core kernel runs on these with the queries as projected."""
+    step, and the tensor-core kernel runs on these with the queries as projected.
+
+    A run without a latent of its own (``own_kv`` False) reads the rows of the run its schedule entry names, with its own
+    queries, W_uk and W_uv."""
 
     kernels = ("linear", "linear_mma", "linear_tc", "gemm_tc", "attention", "attention_prefill", "rotary_pairs", "norm")
     TILED_MIN_TOKENS = 16  # runs of new tokens from this many on take the tensor-core kernel (bfloat16)
@@ -57,9 +60,9 @@ class LatentAttention(Mixer):
 
     def params(self) -> Dict[str, ParamSpec]:
         s = self.spec
-        p = {"dkv": ParamSpec((self.key_row, s.width)), "dkv.norm": ParamSpec((s.kv_rank,), init="ones"),
-             "uk": ParamSpec((s.n_heads * s.head_dim, s.kv_rank)), "uv": ParamSpec((s.n_heads * s.v_head_dim, s.kv_rank)),
-             "o": ParamSpec((s.width, s.n_heads * s.v_head_dim))}
+        p = {"uk": ParamSpec((s.n_heads * s.head_dim, s.kv_rank)), "uv": ParamSpec((s.n_heads * s.v_head_dim, s.kv_rank)), "o": ParamSpec((s.width, s.n_heads * s.v_head_dim))}
+        if s.own_kv:
+            p.update({"dkv": ParamSpec((self.key_row, s.width)), "dkv.norm": ParamSpec((s.kv_rank,), init="ones")})
         if s.q_rank:
             p.update({"dq": ParamSpec((s.q_rank, s.width)), "dq.norm": ParamSpec((s.q_rank,), init="ones"),
                       "uq": ParamSpec((s.n_heads * (s.head_dim + s.rot_dim), s.q_rank))})
@@ -80,26 +83,28 @@ class LatentAttention(Mixer):
         s = self.spec
         if s.q_rank:
             self.w_dq, self.g_dq, self.w_uq = tensors["dq"], tensors["dq.norm"], tensors["uq"]
-        self.g_dkv, self.w_o = tensors["dkv.norm"], tensors["o"]
+        self.g_dkv, self.w_o = tensors.get("dkv.norm"), tensors["o"]
         self.sink = tensors["sink"].float().contiguous() if self.has_sink else None
         # the latent, the rotated key part, the gates and (without a query latent) the queries are one product of
         # the mixer's input
-        parts = [tensors["dkv"]] + ([tensors["g"]] if self.gate_len else [])
-        self.g_off = self.key_row
-        at = self.key_row + self.gate_len
+        parts = ([tensors["dkv"]] if s.own_kv else []) + ([tensors["g"]] if self.gate_len else [])
+        self.g_off = self.key_row if s.own_kv else 0
+        at = self.g_off + self.gate_len
         if not s.q_rank:
             gap = -at % 8  # the queries start at a 16-byte boundary of the row
             if gap:
-                parts.append(torch.zeros((gap, s.width), dtype=parts[0].dtype, device=parts[0].device))
+                parts.append(torch.zeros((gap, s.width), dtype=tensors["q"].dtype, device=tensors["q"].device))
             self.q_off = at + gap
             parts.append(tensors["q"])
             at = self.q_off + s.n_heads * (s.head_dim + s.rot_dim)
-        dt = parts[0].dtype if all(t.dtype == parts[0].dtype for t in parts) else torch.float32
-        pad = -at % 8  # rows of the product's result stay 16-byte aligned
-        if pad:
-            parts.append(torch.zeros((pad, s.width), dtype=dt, device=parts[0].device))
-        self.w_kv = torch.cat([t.to(dt) for t in parts], dim=0).contiguous()
-        self.row = at + pad
+        self.w_kv, self.row = None, 0  # (nothing at all where a run has a query latent, no gates and no latent of its own)
+        if parts:
+            dt = parts[0].dtype if all(t.dtype == parts[0].dtype for t in parts) else torch.float32
+            pad = -at % 8  # rows of the product's result stay 16-byte aligned
+            if pad:
+                parts.append(torch.zeros((pad, s.width), dtype=dt, device=parts[0].device))
+            self.w_kv = torch.cat([t.to(dt) for t in parts], dim=0).contiguous()
+            self.row = at + pad
         # per head: W_uk as [dim, kv_rank] (plain query part -> latent space), W_uv as [vdim, kv_rank]
         self.w_uk = tensors["uk"].reshape(s.n_heads, s.head_dim, s.kv_rank).contiguous()
         self.w_uv = tensors["uv"].reshape(s.n_heads, s.v_head_dim, s.kv_rank).contiguous()
@@ -114,7 +119,9 @@ class LatentAttention(Mixer):
         n = h.shape[0]
         H, d, dr, rank, row = s.n_heads, s.head_dim, s.rot_dim, s.kv_rank, self.key_row
         dt = self.build.dtype
-        ckv = ops.linear(h, self.w_kv, out_dtype=dt)  # [n, latent | rotated key part | gates | (queries) | padding]
+        if kv.owner != s.own_kv:
+            raise ValueError("a latent mixer with a latent of its own owns its cache plane, one without reads another's")
+        ckv = ops.linear(h, self.w_kv, out_dtype=dt) if self.w_kv is not None else None  # [n, latent | rotated key part | gates | (queries) | padding]
         if s.q_rank:
             cq = ops.linear(h, self.w_dq, out_dtype=dt)
             ops.rmsnorm_slices(cq, s.norm_eps, 0, s.q_rank, self.g_dq)
@@ -123,9 +130,13 @@ class LatentAttention(Mixer):
             q, q_off = ckv, self.q_off
         # the latent normed, the heads' rotated query parts and the shared key part rotated, the key row [c | k_rot]
         # to the cache: one launch
-        self.position.apply(ckv, ctx, xq=q, q_off=q_off, n_q_heads=H, q_head_stride=d + dr, q_rot_off=d, k_off=0, n_k_heads=1,
-                            k_head_stride=row, k_rot_off=rank, k_row=row, tok_seq=ctx.tok_seq, slots=ctx.slots,
-                            page_table=kv.page_table, k_cache=kv.k, norm_len=rank, norm_w=self.g_dkv, norm_eps=s.norm_eps)
+        places = dict(q_off=q_off, n_q_heads=H, q_head_stride=d + dr, q_rot_off=d)
+        if s.own_kv:
+            self.position.apply(ckv, ctx, xq=q, k_off=0, n_k_heads=1, k_head_stride=row, k_rot_off=rank, k_row=row, tok_seq=ctx.tok_seq,
+                                slots=ctx.slots, page_table=kv.page_table, k_cache=kv.k, norm_len=rank, norm_w=self.g_dkv,
+                                norm_eps=s.norm_eps, **places)
+        else:
+            self.position.apply(q, ctx, **places)
         gate = ckv[:, self.g_off:] if s.head_gate else None
         egate = ckv[:, self.g_off: self.g_off + self.gate_len] if self.element_gate else None
         tiled = dt == torch.bfloat16 and not ctx.decode and ctx.tile_seq is not None and ctx.max_new >= self.TILED_MIN_TOKENS

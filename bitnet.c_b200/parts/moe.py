@@ -1,4 +1,4 @@
-"""Mixture of gated experts: logistic or softmax router scores, clamped or plain gated units."""
+"""Mixture of experts: logistic or softmax router scores, clamped or plain gated units, or units without a gate."""
 from __future__ import annotations
 
 from typing import Dict
@@ -21,7 +21,10 @@ class Moe(FeedForward):
     over all experts as scores; ``renormalise`` divides the chosen ones' by their sum (+ ``renormalise_eps``);
     ``router_bias`` adds a number per expert to the logits; ``weight_scale`` multiplies the weights; ``activation`` "silu" / "gelu_tanh" makes an expert
     down(act(gate x) * (up x)) without clamps; ``scores`` "table": no router, a table of expert ids by token id
-    chooses and every chosen expert weighs 1 / top.
+    chooses and every chosen expert weighs 1 / top; ``correction`` chooses by score + a learned number per expert, within the
+    ``keep_groups`` best of ``groups`` equal groups, and weighs by the score alone; ``identity``: the router's last outputs stand for
+    the input itself; ``activation`` "relu2": down(max(up x, 0)^2), no gate; ``shared_gate``: the shared expert's output times the
+    logistic function of one number per token, a row of the router's product.
 
     Few rows (a decode step): two kernels stream the chosen experts once per (token, expert), from
     device memory alone.  Many rows: the (token, expert) items are sorted by expert and every expert's
@@ -40,64 +43,88 @@ class Moe(FeedForward):
         self.by_table = scores == "table"
         if self.by_table and (getattr(spec, "table_rows", 0) <= 0 or spec.shared_ff or spec.weight_on_input):
             raise ValueError("experts chosen by a table need its number of rows, weigh their outputs and have no shared expert")
-        if activation != "limited" and activation not in ops.ACTIVATIONS:
-            raise ValueError(f"expert activation {activation!r} is not built; known: limited, {', '.join(sorted(ops.ACTIVATIONS))}")
+        if activation not in ("limited", "relu2") and activation not in ops.ACTIVATIONS:
+            raise ValueError(f"expert activation {activation!r} is not built; known: limited, relu2, {', '.join(sorted(ops.ACTIVATIONS))}")
+        self.gated = activation != "relu2"
+        self.outputs = spec.n_experts + spec.identity  # what the router chooses among
+        if self.by_table and (spec.identity or spec.correction) or spec.groups > 1 and not spec.correction:
+            raise ValueError("identity experts need a router; groups go with a correction")
+        if spec.shared_gate and (self.by_table or not spec.shared_ff):
+            raise ValueError("a gate on the shared expert needs a router and a shared expert")
+        if spec.identity and spec.weight_on_input:
+            raise ValueError("identity experts are built for weights on the output")
         self.softmax = scores == "softmax"
-        self.act = -1 if activation == "limited" else ops.ACTIVATIONS[activation]  # -1: the clamped unit
+        # -1: the clamped unit
+        self.act = -1 if activation == "limited" else ops.ACT_RELU2 if not self.gated else ops.ACTIVATIONS[activation]
         # experts too wide for the streaming kernels' shared memory always take the sorted path, which asks the
         # device for the experts' counts: such a model's steps are not recorded
         self.few_fits = ops.moe_few_fits(spec.width, spec.top, spec.expert_ff)
         self.graph_safe = self.few_fits
 
-    def _activate(self, gate_up, out, limit):
+    def _activate(self, up, limit):
+        """The unit on rows of [gate | up], or of up alone."""
+        if not self.gated:
+            return ops.relu_squared(up)
+        out = torch.empty((up.shape[0], up.shape[1] // 2), dtype=up.dtype, device=up.device)
         if self.act < 0:
-            return ops.glu_limited(gate_up, out, limit, self.spec.slope)
-        return ops.glu_halves(gate_up, out, self.act)
+            return ops.glu_limited(up, out, limit, self.spec.slope)
+        return ops.glu_halves(up, out, self.act)
 
     def params(self) -> Dict[str, ParamSpec]:
         s = self.spec
         if self.by_table:  # token id -> the ids of its experts, different within a row
             p = {"table": ParamSpec((s.table_rows, s.top), init="distinct", integer=True, high=s.n_experts)}
         else:
-            p = {"router": ParamSpec((s.n_experts, s.width))}
+            p = {"router": ParamSpec((self.outputs, s.width))}
             if s.router_bias:
-                p["router.b"] = ParamSpec((s.n_experts,))
+                p["router.b"] = ParamSpec((self.outputs,))
+            if s.correction:
+                p["correction"] = ParamSpec((self.outputs,))
         for e in range(s.n_experts):
-            p[f"e{e}.gate"] = ParamSpec((s.expert_ff, s.width))
+            if self.gated:
+                p[f"e{e}.gate"] = ParamSpec((s.expert_ff, s.width))
             p[f"e{e}.up"] = ParamSpec((s.expert_ff, s.width))
             p[f"e{e}.down"] = ParamSpec((s.width, s.expert_ff))
         if s.shared_ff:
-            p["shared.gate"] = ParamSpec((s.shared_ff, s.width))
+            if self.gated:
+                p["shared.gate"] = ParamSpec((s.shared_ff, s.width))
             p["shared.up"] = ParamSpec((s.shared_ff, s.width))
             p["shared.down"] = ParamSpec((s.width, s.shared_ff))
+            if s.shared_gate:
+                p["shared.sg"] = ParamSpec((1, s.width))
         return p
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         s = self.spec
         dt = self.build.dtype
         self.w_router = tensors.get("router")
+        if s.shared_gate:
+            r, g = self.w_router, tensors["shared.sg"]
+            wd = r.dtype if r.dtype == g.dtype else torch.float32
+            self.w_router = torch.cat([r.to(wd), g.to(wd)]).contiguous()
+        self.correction = tensors["correction"].float().contiguous() if s.correction else None
         self.b_router = tensors["router.b"].float().contiguous() if s.router_bias else None
         self.table = tensors.get("table")
         # the table on the host too: how many tokens of a step take each expert is then known without asking the device
         self.table_host = self.table.cpu().numpy() if self.table is not None else None
-        # [experts, 2 ff, width]: an expert's gate rows, then its up rows; [experts, width, ff]
-        self.w_gate_up = torch.stack([torch.cat([tensors[f"e{e}.gate"].to(dt), tensors[f"e{e}.up"].to(dt)], dim=0)
-                                      for e in range(s.n_experts)]).contiguous()
+        up_of = lambda n: torch.cat([tensors[f"{n}.gate"].to(dt), tensors[f"{n}.up"].to(dt)], dim=0) if self.gated else tensors[f"{n}.up"].to(dt)
+        # [experts, 2 ff, width]: an expert's gate rows, then its up rows (up rows alone without a gate); [experts, width, ff]
+        self.w_gate_up = torch.stack([up_of(f"e{e}") for e in range(s.n_experts)]).contiguous()
         self.w_down = torch.stack([tensors[f"e{e}.down"].to(dt) for e in range(s.n_experts)]).contiguous()
         if s.shared_ff:
-            self.w_shared_gate_up = torch.cat([tensors["shared.gate"].to(dt), tensors["shared.up"].to(dt)], dim=0).contiguous()
+            self.w_shared_gate_up = up_of("shared").contiguous()
             self.w_shared_down = tensors["shared.down"]
 
     def _expert(self, x, w_gate_up, w_down, limit, out_dtype):
-        gu = ops.linear(x, w_gate_up, out_dtype=self.build.dtype)
-        act = torch.empty((x.shape[0], gu.shape[1] // 2), dtype=gu.dtype, device=gu.device)
-        self._activate(gu, act, limit)
-        return ops.linear(act, w_down, out_dtype=out_dtype)
+        if not self.gated:
+            return ops.linear(ops.linear(x, w_gate_up, out_dtype=self.build.dtype, act=ops.ACT_RELU2), w_down, out_dtype=out_dtype)
+        return ops.linear(self._activate(ops.linear(x, w_gate_up, out_dtype=self.build.dtype), limit), w_down, out_dtype=out_dtype)
 
     def forward(self, h, ctx):
         s = self.spec
         T = h.shape[0]
         shared = self._expert(h, self.w_shared_gate_up, self.w_shared_down, s.shared_limit, torch.float32) if s.shared_ff else None
+        shared_scale = None  # a factor per token on the shared expert's output
         if self.by_table:
             # the choice depends on the step's token ids alone: runs that share a table share its rows of the step
             key = ("moe.table", self.table.data_ptr(), s.top)
@@ -105,14 +132,17 @@ class Moe(FeedForward):
                 ctx.memo[key] = ops.moe_table_route(ctx.tokens, self.table, s.top, s.n_experts)
             ids, weights = ctx.memo[key]
         else:
-            ids, weights = ops.moe_route(h, self.w_router, s.top, s.renormalise, softmax=self.softmax,
-                                         weight_scale=getattr(s, "weight_scale", 1.0), sum_eps=getattr(s, "renormalise_eps", 0.0),
-                                         bias=self.b_router)
+            ids, weights, *gate = ops.moe_route(
+                h, self.w_router, s.top, s.renormalise, softmax=self.softmax, weight_scale=getattr(s, "weight_scale", 1.0),
+                sum_eps=getattr(s, "renormalise_eps", 0.0), bias=self.b_router, correction=self.correction, groups=s.groups,
+                keep=s.keep_groups, gate=s.shared_gate)
+            if gate:
+                shared_scale = gate[0]
         if ctx.diag is not None:
             ctx.tap("moe_ids", lambda: ids.float())
         if self.few_fits and (ctx.decode or T * s.top <= self.FEW_ITEMS):
             return ops.moe_experts_few(h, ids, weights, self.w_gate_up, self.w_down, s.expert_limit, s.slope,
-                                       s.weight_on_input, add=shared, act=self.act)
+                                       s.weight_on_input, add=shared, act=self.act, add_scale=shared_scale)
         counts = ops.moe_count(ids, s.n_experts)
         host_tokens = getattr(ctx, "host_tokens", None)
         if self.by_table and host_tokens is not None:
@@ -128,29 +158,28 @@ class Moe(FeedForward):
         else:
             per_expert = counts.cpu().tolist()  # the one place where the host waits for the device
         dt, dev_ = self.build.dtype, h.device
-        cap = -(-max(per_expert) // 8) * 8
+        rest = dict(add_scale=shared_scale, h=h if s.identity else None)
+        cap = max(-(-max(per_expert) // 8) * 8, 8)
         if cap * s.n_experts <= self.PAD_FACTOR * T * s.top:
             # the experts are about evenly used: each gets a block of ``cap`` rows, and all of them run as
             # one batched product each way (rows that no token took compute nothing that is read)
             x_pad, place, _ = ops.moe_sort(h, ids, weights, counts, s.weight_on_input, cap=cap)
             gate_up = ops.batched_matmul(x_pad.view(s.n_experts, cap, s.width), self.w_gate_up)
-            act = torch.empty((s.n_experts * cap, s.expert_ff), dtype=dt, device=dev_)
-            self._activate(gate_up.view(s.n_experts * cap, 2 * s.expert_ff), act, s.expert_limit)
+            act = self._activate(gate_up.view(s.n_experts * cap, -1), s.expert_limit)
             y_pad = ops.batched_matmul(act.view(s.n_experts, cap, s.expert_ff), self.w_down)
-            return ops.moe_gather(y_pad.view(s.n_experts * cap, s.width), place, weights, not s.weight_on_input, add=shared)
+            return ops.moe_gather(y_pad.view(s.n_experts * cap, s.width), place, weights, not s.weight_on_input, add=shared, **rest)
         # uneven: the experts' rows packed side by side, their products one after another into slices
         x_sorted, place, _ = ops.moe_sort(h, ids, weights, counts, s.weight_on_input)
         at = [0]
         for c in per_expert:
             at.append(at[-1] + c)
-        gate_up = torch.empty((T * s.top, 2 * s.expert_ff), dtype=dt, device=dev_)
+        gate_up = torch.empty((T * s.top, self.w_gate_up.shape[1]), dtype=dt, device=dev_)
         for e in range(s.n_experts):
             if at[e + 1] > at[e]:
                 ops.matmul_into(x_sorted[at[e]: at[e + 1]], self.w_gate_up[e], gate_up[at[e]: at[e + 1]])
-        act = torch.empty((T * s.top, s.expert_ff), dtype=dt, device=dev_)
-        self._activate(gate_up, act, s.expert_limit)
+        act = self._activate(gate_up, s.expert_limit)
         y_sorted = torch.empty((T * s.top, s.width), dtype=dt, device=dev_)
         for e in range(s.n_experts):
             if at[e + 1] > at[e]:
                 ops.matmul_into(act[at[e]: at[e + 1]], self.w_down[e], y_sorted[at[e]: at[e + 1]])
-        return ops.moe_gather(y_sorted, place, weights, not s.weight_on_input, add=shared)
+        return ops.moe_gather(y_sorted, place, weights, not s.weight_on_input, add=shared, **rest)

@@ -102,7 +102,7 @@ def blended_frequencies(spec, wide: bool = False):
     The magnitude multiplies cos and sin alike."""
     dims = spec.dims
     i = np.arange(dims // 2, dtype=np.float64)
-    f = np.float64(spec.base) ** (-2.0 * i / dims)
+    f = np.float64(spec.base) ** (-2.0 * i / dims) / getattr(spec, "slowdown", 1.0)
     if spec.factor == 1.0 or spec.original <= 0:
         return (f if wide else f.astype(np.float32)), 1.0
 
