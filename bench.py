@@ -586,6 +586,43 @@ RUDOLIX_SIZES = {
 }
 
 
+def lakadra_sizes(width, heads, kv_heads, dim, rot_dim, q_rank, kv_rank, l_heads, l_dim, l_vdim, window, inner, blocks, taps, ff, experts,
+                  identity, groups, keep, top, vocab):
+    """A Lakadra configuration of four layers (lightning attention; latent attention; windowed attention beside the gated
+    linear recurrence; latent attention on the second layer's rows; every layer with experts, of which a token uses ``top``
+    of a quarter of the dense unit's width each, and a shared expert of half its width), the Llama configuration of the same
+    width, heads, layers, vocabulary and feed-forward width, and Lotilix and Rudolix configurations of that size, which hold
+    the nearest relatives of its mixers."""
+    latent = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": dim, "q_rank": q_rank, "kv_rank": kv_rank,
+              "scale": (dim + rot_dim) ** -0.5, "rot": {"base": 1e6, "dims": rot_dim}}
+    lightning = {"heads": l_heads, "dim": l_dim, "vdim": l_vdim, "decay": [1.0 - 2.0 ** (-3.0 - 5.0 * h / l_heads) for h in range(l_heads)]}
+    pair = {"left_scale": 0.5, "right_scale": 0.5,
+            "left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window},
+                     "rot": {"base": 5e5, "dims": dim, "scaling": {"factor": 8.0}}},
+            "right": {"width": inner, "blocks": blocks, "conv": taps}}
+    mlp = {"kind": "moe", "router": {"experts": experts, "top": top, "identity": identity, "groups": {"count": groups, "keep": keep}},
+           "expert": {"ff": ff // 4}, "shared": {"ff": ff // 2}}
+    layers = [{"type": "lightning", "mixer": lightning, "mlp": mlp}, {"type": "latent_attention", "mixer": latent, "mlp": mlp},
+              {"type": "parallel", "mixer": pair, "mlp": mlp}, {"type": "latent_attention", "mixer": dict(latent, kv_from=1), "mlp": mlp}]
+    lak = {"architecture": "Lakadra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0, "logit_softcap": 30.0,
+           "layers": layers, "max_positions": 8192}
+    llama = {"architectures": ["LlamaForCausalLM"], "model_type": "llama", "hidden_size": width, "intermediate_size": ff,
+             "num_hidden_layers": len(layers), "num_attention_heads": heads, "num_key_value_heads": kv_heads, "head_dim": dim,
+             "vocab_size": vocab, "max_position_embeddings": 8192, "rope_theta": 500000.0, "rms_norm_eps": 1e-5,
+             "tie_word_embeddings": False, "hidden_act": "silu"}
+    return lak, llama, {"lotilix": lotilix_sizes(**LOTILIX_SIZES[f"w{width}"])[0], "rudolix": rudolix_sizes(**RUDOLIX_SIZES[f"w{width}"])[0]}
+
+
+LAKADRA_SIZES = {
+    "w1024": dict(width=1024, heads=8, kv_heads=2, dim=128, rot_dim=64, q_rank=384, kv_rank=192, l_heads=8, l_dim=128, l_vdim=128,
+                  window=1024, inner=1024, blocks=8, taps=4, ff=4096, experts=14, identity=2, groups=4, keep=2, top=2, vocab=32000),
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, rot_dim=64, q_rank=768, kv_rank=192, l_heads=16, l_dim=128, l_vdim=128,
+                  window=1024, inner=2048, blocks=16, taps=4, ff=8192, experts=14, identity=2, groups=4, keep=2, top=2, vocab=32000),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, rot_dim=64, q_rank=1536, kv_rank=512, l_heads=32, l_dim=128, l_vdim=128,
+                  window=1024, inner=4096, blocks=16, taps=4, ff=14336, experts=14, identity=2, groups=4, keep=2, top=2, vocab=32000),
+}
+
+
 def kernel_classes(model, vocab, tokens, batch, prompt_len):
     """Device time by entry point (ms) of one step of ``tokens`` prompt tokens and of one decode step of
     ``batch`` sequences behind prompts of ``prompt_len``, each kernel between two events (no graph, so the
@@ -626,7 +663,7 @@ def kernel_classes(model, vocab, tokens, batch, prompt_len):
 
 
 def run_design(args):
-    """``--design fesorax | lotilix | mekevik | netanex | rudolix``: prefill and decode throughput of that design at layer sizes of real
+    """``--design fesorax | lakadra | lotilix | mekevik | netanex | rudolix``: prefill and decode throughput of that design at layer sizes of real
     models (random weights, bfloat16), beside the Llama decoder of equal width, heads, layers, vocabulary and
     feed-forward work per token, with each step's device time by kernel entry point."""
     import torch
@@ -637,6 +674,7 @@ def run_design(args):
            "decode_batch": args.batch, "decode_prompt": PROMPT_LEN, "sizes": {}}
     sizes, maker = {"lotilix": (LOTILIX_SIZES, lotilix_sizes), "mekevik": (MEKEVIK_SIZES, mekevik_sizes),
                     "netanex": (NETANEX_SIZES, netanex_sizes), "rudolix": (RUDOLIX_SIZES, rudolix_sizes),
+                    "lakadra": (LAKADRA_SIZES, lakadra_sizes),
                     "fesorax": (DESIGN_SIZES, fesorax_sizes)}[args.design]
     rec["metric"] = rec["metric"].replace("Fesorax", args.design.capitalize())
     names = [n for n in sizes if not args.sizes or n in args.sizes.split(",")]
@@ -677,7 +715,7 @@ def main():
                          "(comparisons, profiling)")
     ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16",
                     help="compute type of the main decode run (float32: profiling of the 32-bit path, with --skip-points)")
-    ap.add_argument("--design", choices=["fesorax", "lotilix", "mekevik", "netanex", "rudolix"],
+    ap.add_argument("--design", choices=["fesorax", "lakadra", "lotilix", "mekevik", "netanex", "rudolix"],
                     help="measure another design of the library beside Llama at equal size instead (prefill, decode, "
                          "time by kernel); the default workload and its record stay as they are")
     ap.add_argument("--sizes", default="", help="with --design: which size sets, with commas (default: all)")
