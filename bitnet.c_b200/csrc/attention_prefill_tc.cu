@@ -27,7 +27,7 @@
 // width of their own (VD), and a sink, a score per head without a key or a value, may enlarge the rows' sums at the end.
 // The new tokens' own keys and values must already be in the cache, so the same kernel serves
 // whole prompts, pieces of prompts and ragged batches (a table gives each block its sequence and
-// first row).  Head sizes in steps of 16 up to 128 run on the instantiation for 64 or 128: columns
+// first row).  Head sizes in steps of 16 up to 192 run on the instantiation for 64, 128 or 192: columns
 // past the head size read as zero (TMA fills what lies outside the tensor).  Value rows behind a
 // sequence's last position are cleared in shared memory, whatever the cache holds there.
 //
@@ -448,7 +448,7 @@ static int launch_pt(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
 // tile_seq / tile_row0: for each block its sequence and the first of its 128 new-token rows;
 // seq_start [n_seqs+1]: first packed row of each sequence; seq_pos0: its length before the step.
 // The caches are [n_cache_pages, n_kv_heads, 64, head_dim], contiguous and 16-byte aligned, and
-// already hold the new tokens.  head_dim: a multiple of 16 up to 128.  status: one int on the
+// already hold the new tokens.  head_dim: a multiple of 16 up to 192.  status: one int on the
 // device, left as it is unless a wait inside the kernel gave up (then 5; nothing is stored by
 // that block).
 // The values' cache is [n_cache_pages, n_kv_heads, 64, v_dim] with v_dim a multiple of 16 up to 128.  precise: the weights
@@ -462,7 +462,7 @@ extern "C" int bn_attention_prefill_tc_ex(const void* q, int q_stride, int n_tok
                                           const void* k_cache, const void* v_cache, int n_cache_pages, int* status,
                                           cudaStream_t stream) {
   if (n_tiles <= 0) return BN_OK;
-  if (head_dim <= 0 || head_dim % 16 || head_dim > 128 || v_dim <= 0 || v_dim % 16 || v_dim > 128 || !(scale > 0.f) || n_kv_heads <= 0 || n_heads % n_kv_heads || window < 0 ||
+  if (head_dim <= 0 || head_dim % 16 || head_dim > 192 || v_dim <= 0 || v_dim % 16 || v_dim > 128 || !(scale > 0.f) || n_kv_heads <= 0 || n_heads % n_kv_heads || window < 0 ||
       n_heads > 65535 || (q_stride % 8) || (out_stride % 8) || n_tokens <= 0 || n_cache_pages <= 0 || !status ||
       (((uintptr_t)q | (uintptr_t)out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15))
     return BN_ERR_BAD_ARG;
@@ -487,6 +487,9 @@ extern "C" int bn_attention_prefill_tc_ex(const void* q, int q_stride, int n_tok
   return precise ? launch_pt<HD, VD, KS, VS, true>(mq, mk, mv, a, n_tiles, stream) : launch_pt<HD, VD, KS, VS, false>(mq, mk, mv, a, n_tiles, stream)
   if (head_dim <= 64 && v_dim <= 64) PT_RUN(64, 64, 3, 3);
   if (head_dim <= 64) PT_RUN(64, 128, 3, 2);
+  // keys of up to 192 numbers (a latent layer's heads, unrotated and rotated part): 120 and 128 KB, one block per SM
+  if (head_dim > 128 && v_dim <= 64) PT_RUN(192, 64, 2, 3);
+  if (head_dim > 128) PT_RUN(192, 128, 2, 2);
   if (v_dim <= 64) PT_RUN(128, 64, 2, 3);
   PT_RUN(128, 128, 2, 2);
 #undef PT_RUN

@@ -52,6 +52,7 @@ SOURCES: Dict[str, str] = {
     "streams": "streams.cu",
     "gated_state": "gated_state.cu",
     "gated_linear": "gated_linear.cu",
+    "latent": "latent.cu",
     "sigmoid_attention": "sigmoid_attention.cu",
     "sigmoid_attention_prefill": "sigmoid_attention_prefill.cu",
 }

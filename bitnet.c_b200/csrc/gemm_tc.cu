@@ -9,7 +9,7 @@
 // stage) into one of two accumulators of 256 columns in tensor memory; while it works on the next
 // tile's accumulator, four epilogue warps read the finished one (a thread owns a row: its TMEM
 // lane) and finish it:
-//   mode 0  store (bfloat16 or float32);
+//   mode 0  store (bfloat16 or float32), with BN_ACT_RELU2 the square of the positive part;
 //   mode 2  SwiGLU: columns hold gate and up values in alternating blocks of 8 (the layout of the
 //           stacked weight), out[m, i] = silu(gate_i) * up_i, [M, N / 2];
 //   mode 3  residual[m, n] += result (float32, in place); xg[m, n] = residual * gain[n] (the next
@@ -17,6 +17,10 @@
 //           residual values of these 256 columns: the rows of xg still lack the norm's scale
 //           1 / sqrt(sum of the parts / N + eps), which the product that consumes them applies
 //           to its own result rows, W (s x) = s (W x): modes 0 and 2 take such rows (row_ss).
+// Grouped: the rows of x belong to groups, packed one behind another (offsets on the device), and every group has a matrix of its
+// own in a stack of W: the experts of a mixture in one launch, however their rows are shared out, without asking the
+// device for the counts.  The tiles of all groups form one list; a tile's rows past its group's end are not stored.
+//
 // This removes the separate passes over the activations that a library product leaves to other
 // kernels: the SwiGLU pass over [M, 2 I] and both residual + norm passes of a layer.
 //
@@ -41,7 +45,7 @@ struct GmArgs {
   void* out;        // modes 0, 2: [M, ldo]
   int out_dtype;
   int M, N, K, ldo, mode;
-  int act;          // mode 2: the gate's activation (BN_ACT_*)
+  int act;          // mode 2: the gate's activation (BN_ACT_*); mode 0: BN_ACT_RELU2 or none
   int k_blocks, m_tiles, n_tiles;
   const float* row_ss;  // [ss_parts][ss_stride]: sums of squares of the input rows, or null (rows are plain)
   int ss_parts, ss_stride;
@@ -53,20 +57,51 @@ struct GmArgs {
   float* ss_out;        // mode 3: [n_tiles][ss_out_stride]
   int ss_out_stride;
   int* status;
+  const int* offsets;   // grouped: [groups + 1] first row of each group, or null
+  int groups;
 };
+
+// Which tile a number stands for: the matrix's rows (wrow0: in the stack), the output's rows from m0 to m_end, the columns' tile.
+struct GmTile {
+  int m0, m_end, nt, wrow0;
+};
+// Grouped: prefix[g] = the number of tiles of the groups before g; g only moves forward along a block's tiles.
+__device__ __forceinline__ GmTile gm_tile(const GmArgs& a, const int* prefix, int t, int rows_per_tile, int m_tiles, int* g) {
+  GmTile r;
+  if (a.offsets == nullptr) {
+    r.m0 = (t % m_tiles) * rows_per_tile;
+    r.nt = t / m_tiles;
+    r.m_end = a.M;
+    r.wrow0 = 0;
+    return r;
+  }
+  while (t >= prefix[*g + 1]) ++*g;
+  const int first = a.offsets[*g], end = a.offsets[*g + 1], tiles = (end - first + rows_per_tile - 1) / rows_per_tile;
+  const int local = t - prefix[*g];
+  r.m0 = first + (local % tiles) * rows_per_tile;
+  r.nt = local / tiles;
+  r.m_end = end;
+  r.wrow0 = *g * a.N;
+  return r;
+}
 
 __device__ __forceinline__ float gm_glu_mul(float g, float u, int act) { return glu_activation(g, act) * u; }
 
 // The epilogue of one tile for one thread in modes 0 and 2: row m of the output, the 256 columns
 // from n0 on, read from the thread's TMEM lane at acc_addr (see the modes at the top of this file).
-__device__ __forceinline__ void gm_finish_tile(const GmArgs& a, unsigned acc_addr, int m, int n0, float scale) {
-  const bool live = m < a.M;
+__device__ __forceinline__ void gm_finish_tile(const GmArgs& a, unsigned acc_addr, int m, int m_end, int n0, float scale) {
+  const bool live = m < m_end;
 #pragma unroll 1
   for (int c = 0; c < GM_BN; c += 32) {
     float v[32];
     tmem_ld32(acc_addr + c, v);
     if (!live || n0 + c >= a.N) continue;
     if (a.mode == 0) {
+      if (a.act == BN_ACT_RELU2) {
+#pragma unroll
+        for (int e = 0; e < 32; ++e) v[e] = relu_squared(v[e] * scale);
+        scale = 1.0f;
+      }
       if (a.out_dtype == BN_BF16) {
         __nv_bfloat16* o = (__nv_bfloat16*)a.out + (size_t)m * a.ldo + n0 + c;
 #pragma unroll
@@ -292,7 +327,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
         gm_finish_tile_rows(a, lane_addr + buf * GM_BN, mt * GM_BM + quad * 32, n0, nt, gain_s + buf * GM_BN,
                             stage_s + (warp - 2) * 32 * GM_STG, lane);
       else
-        gm_finish_tile(a, lane_addr + buf * GM_BN, m, n0, scale);
+        gm_finish_tile(a, lane_addr + buf * GM_BN, m, a.M, n0, scale);
       // the accumulator may be written again
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       __syncwarp();
@@ -383,13 +418,14 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
   volatile int* failed = (volatile int*)(tmem_slot + 1);
   float* gain_s = (float*)(tmem_slot + 4);
   float* stage_s = gain_s + 2 * GM_BN;
+  int* prefix = (int*)(stage_s + 4 * 32 * GM_STG);  // grouped: [groups + 1]
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const unsigned rank = gm_cluster_rank();
   const bool leader = rank == 0;
   const int pair = blockIdx.x >> 1, n_pairs = gridDim.x >> 1;
   const int m_pairs = (a.m_tiles + 1) / 2;
-  const int n_tiles_total = m_pairs * a.n_tiles;
+  int n_tiles_total = m_pairs * a.n_tiles;
 
   if (tid == 0) {
     *failed = 0;
@@ -416,14 +452,36 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
   asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
   const unsigned tmem_base = *tmem_slot;
   pdl_wait();
+  if (a.offsets != nullptr) {
+    // both blocks of a pair count the same tiles
+    if (warp == 0) {
+      const int per = (a.groups + 31) / 32, g0 = min(lane * per, a.groups), g1 = min(g0 + per, a.groups);
+      int mine = 0;
+      for (int g = g0; g < g1; ++g) mine += (a.offsets[g + 1] - a.offsets[g] + 2 * GM_BM - 1) / (2 * GM_BM) * a.n_tiles;
+      int upto = mine;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int up = __shfl_up_sync(0xffffffffu, upto, o);
+        if (lane >= o) upto += up;
+      }
+      int at = upto - mine;
+      for (int g = g0; g < g1; ++g) {
+        prefix[g] = at;
+        at += (a.offsets[g + 1] - a.offsets[g] + 2 * GM_BM - 1) / (2 * GM_BM) * a.n_tiles;
+      }
+      if (lane == 31) prefix[a.groups] = upto;
+    }
+    __syncthreads();
+    n_tiles_total = prefix[a.groups];
+  }
 
   if (warp == 0) {
     // ---- producer: this block's halves of the operands; the bytes count on the leader's barrier
     if (lane == 0) {
-      int it = 0;
+      int it = 0, group = 0;
       bool ok = true;
       for (int t = pair; ok && t < n_tiles_total; t += n_pairs) {
-        const int mp = t % m_pairs, nt = t / m_pairs;
+        const GmTile tile = gm_tile(a, prefix, t, 2 * GM_BM, m_pairs, &group);
         for (int kb = 0; kb < a.k_blocks; ++kb, ++it) {
           const int s = it % GM2_STAGES, round = it / GM2_STAGES;
           if (round > 0 && (!mbar_wait(empty0 + 8 * s, (unsigned)(round - 1) & 1u, a.status, GM_ERR_WAIT) || *failed)) {
@@ -434,8 +492,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
           const unsigned dst = smem_u32(base + s * STAGE_BYTES);
           if (leader) mbar_expect_tx(full0 + 8 * s, 2 * STAGE_BYTES);
           const unsigned bar = gm_map_to_rank(full0 + 8 * s, 0);
-          gm_tma_load_2d_pair(dst, &map_x, bar, kb * GM_BK, mp * 2 * GM_BM + (int)rank * GM_BM);
-          gm_tma_load_2d_pair(dst + A_BYTES, &map_w, bar, kb * GM_BK, nt * GM_BN + (int)rank * (GM_BN / 2));
+          gm_tma_load_2d_pair(dst, &map_x, bar, kb * GM_BK, tile.m0 + (int)rank * GM_BM);
+          gm_tma_load_2d_pair(dst + A_BYTES, &map_w, bar, kb * GM_BK, tile.wrow0 + tile.nt * GM_BN + (int)rank * (GM_BN / 2));
         }
       }
     }
@@ -474,11 +532,12 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
     const int quad = warp & 3, et = tid - 64;
     const int row = quad * 32 + lane;
     const unsigned lane_addr = tmem_base + ((unsigned)(quad * 32) << 16);
-    int tile_i = 0;
+    int tile_i = 0, group = 0;
     bool ok = true;
     for (int t = pair; t < n_tiles_total; t += n_pairs, ++tile_i) {
-      const int mp = t % m_pairs, nt = t / m_pairs, buf = tile_i & 1;
-      const int m = mp * 2 * GM_BM + (int)rank * GM_BM + row, n0 = nt * GM_BN;
+      const GmTile tile = gm_tile(a, prefix, t, 2 * GM_BM, m_pairs, &group);
+      const int nt = tile.nt, buf = tile_i & 1;
+      const int m = tile.m0 + (int)rank * GM_BM + row, n0 = nt * GM_BN;
       float scale = 1.0f;
       if (a.row_ss != nullptr && m < a.M) {
         float ss = 0.f;
@@ -497,10 +556,10 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
       if (!ok) continue;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       if (a.mode == 3)
-        gm_finish_tile_rows(a, lane_addr + buf * GM_BN, mp * 2 * GM_BM + (int)rank * GM_BM + quad * 32, n0, nt,
+        gm_finish_tile_rows(a, lane_addr + buf * GM_BN, tile.m0 + (int)rank * GM_BM + quad * 32, n0, nt,
                             gain_s + buf * GM_BN, stage_s + (warp - 2) * 32 * GM_STG, lane);
       else
-        gm_finish_tile(a, lane_addr + buf * GM_BN, m, n0, scale);
+        gm_finish_tile(a, lane_addr + buf * GM_BN, m, tile.m_end, n0, scale);
       // the pair's accumulator may be written again once all eight epilogue warps have said so
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       __syncwarp();
@@ -534,6 +593,20 @@ static int gm_sm_count() {
   return n;
 }
 
+// The pair kernel's shared memory; grouped products keep their tiles' counts behind it.
+#define GM_MAX_GROUPS 1024
+#define GM2_SMEM ((size_t)GM2_STAGES * (GM_BM + GM_BN / 2) * GM_BK * 2 + (2 * GM2_STAGES + 4) * 8 + 16 + 2 * GM_BN * 4 + 4 * 32 * GM_STG * 4 + 1024)
+static int gm_grant_pair_smem() {
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(gemm_tc_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         (int)(GM2_SMEM + (GM_MAX_GROUPS + 1) * sizeof(int)));
+    if (e != cudaSuccess) return BN_ERR_LAUNCH + (int)e;
+    configured = true;
+  }
+  return BN_OK;
+}
+
 // How many parts of sums of squares a mode-3 product of N columns writes (rows of ss_out).
 extern "C" int bn_gemm_tc_parts(int N) { return N <= 0 ? 0 : (N + GM_BN - 1) / GM_BN; }
 
@@ -550,7 +623,7 @@ extern "C" int bn_gemm_tc(const void* x, const void* w, int M, int N, int K, voi
   if (M <= 0 || N <= 0) return BN_OK;
   const int act = mode >> 8;
   mode &= 255;
-  if (act != BN_ACT_SILU && act != BN_ACT_GELU_TANH) return BN_ERR_BAD_ARG;
+  if (act != BN_ACT_SILU && act != BN_ACT_GELU_TANH && !(act == BN_ACT_RELU2 && mode == 0)) return BN_ERR_BAD_ARG;
   if (K <= 0 || K % 8 || N % 8 || !status || (((uintptr_t)x | (uintptr_t)w) & 15)) return BN_ERR_BAD_ARG;
   if (mode == 0 || mode == 2) {
     if (!out || (out_dtype != BN_BF16 && out_dtype != BN_F32) || ((uintptr_t)out & 15)) return BN_ERR_BAD_ARG;
@@ -576,13 +649,8 @@ extern "C" int bn_gemm_tc(const void* x, const void* w, int M, int N, int K, voi
   a.residual = residual; a.gain = gain; a.gain_dtype = gain_dtype; a.xg = (__nv_bfloat16*)xg; a.ss_out = ss_out;
   a.ss_out_stride = ss_out_stride; a.status = status;
   if (pairs) {
-    size_t smem = (size_t)GM2_STAGES * (GM_BM + GM_BN / 2) * GM_BK * 2 + (2 * GM2_STAGES + 4) * 8 + 16 + 2 * GM_BN * 4 + 4 * 32 * GM_STG * 4 + 1024;
-    static bool configured = false;
-    if (!configured) {
-      cudaError_t e = cudaFuncSetAttribute(gemm_tc_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-      if (e != cudaSuccess) return BN_ERR_LAUNCH + (int)e;
-      configured = true;
-    }
+    const size_t smem = GM2_SMEM;
+    if (int rc = gm_grant_pair_smem()) return rc;
     long long tiles = (long long)((a.m_tiles + 1) / 2) * a.n_tiles;
     long long want = tiles < gm_sm_count() / 2 ? tiles : gm_sm_count() / 2;
     cudaError_t e = bn_launch_cluster(gemm_tc_pair_kernel, dim3((unsigned)(2 * want)), dim3(GM_THREADS), smem, stream, dim3(2, 1, 1),
@@ -600,6 +668,33 @@ extern "C" int bn_gemm_tc(const void* x, const void* w, int M, int N, int K, voi
   long long tiles = (long long)a.m_tiles * a.n_tiles;
   unsigned blocks = (unsigned)(tiles < gm_sm_count() ? tiles : gm_sm_count());
   BN_LAUNCH(gemm_tc_kernel, blocks, GM_THREADS, smem, stream, mx, mw, a);
+  return BN_OK;
+}
+
+// out[rows of group g] = x[rows of group g] . w[g]^T for all groups in one launch (pairs of blocks).  x: [rows, K] bfloat16, the
+// groups' rows packed one behind another, group g's at offsets[g] .. offsets[g + 1] (on the device; offsets[groups] <= rows); w:
+// [groups, N, K]; out: [rows, N] bfloat16, rows past offsets[groups] are left alone.  act: BN_ACT_RELU2, or 0 for none.
+extern "C" int bn_gemm_tc_grouped(const void* x, const void* w, int rows, int groups, int N, int K, const int* offsets, void* out, int act,
+                                  int* status, cudaStream_t stream) {
+  if (rows <= 0 || N <= 0 || groups <= 0) return BN_OK;
+  if (!x || !w || !out || !offsets || !status || groups > GM_MAX_GROUPS || K <= 0 || K % 8 || N % 8 || (act != 0 && act != BN_ACT_RELU2) ||
+      (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15))
+    return BN_ERR_BAD_ARG;
+  CUtensorMap mx, mw;
+  if (!tma_map_bf16_rows(&mx, x, (unsigned long long)rows, (unsigned long long)K, GM_BM) ||
+      !tma_map_bf16_rows(&mw, w, (unsigned long long)groups * N, (unsigned long long)K, GM_BN / 2))
+    return BN_ERR_BAD_ARG;
+  GmArgs a = {};
+  a.out = out; a.out_dtype = BN_BF16; a.M = rows; a.N = N; a.K = K; a.ldo = N; a.mode = 0; a.act = act;
+  a.k_blocks = (K + GM_BK - 1) / GM_BK; a.m_tiles = (rows + GM_BM - 1) / GM_BM; a.n_tiles = (N + GM_BN - 1) / GM_BN;
+  a.status = status; a.offsets = offsets; a.groups = groups;
+  const size_t smem = GM2_SMEM + (size_t)(GM_MAX_GROUPS + 1) * sizeof(int);
+  if (int rc = gm_grant_pair_smem()) return rc;
+  // at most one tile of rows more per group than the rows alone would make
+  const long long tiles = ((long long)(rows + 2 * GM_BM - 1) / (2 * GM_BM) + groups) * a.n_tiles;
+  const long long want = tiles < gm_sm_count() / 2 ? tiles : gm_sm_count() / 2;
+  cudaError_t e = bn_launch_cluster(gemm_tc_pair_kernel, dim3((unsigned)(2 * want)), dim3(GM_THREADS), smem, stream, dim3(2, 1, 1), mx, mw, a);
+  if (e != cudaSuccess) return BN_ERR_LAUNCH + (int)e;
   return BN_OK;
 }
 

@@ -59,6 +59,77 @@ __device__ __forceinline__ int moe_pick(const float* v, int n, int lane, float* 
   return arg < n ? arg : 0;
 }
 
+// A token's experts from its logits z [n_experts] (which are used up), by one warp; score and group_best: working space of
+// n_experts numbers each.
+__device__ __forceinline__ void moe_choose(float* z, float* score, float* group_best, int n_experts, int top, int renormalise, int softmax,
+                                           float weight_scale, float sum_eps, const MoeChoice& choice, int t, int lane,
+                                           int* __restrict__ ids, float* __restrict__ weights) {
+  // softmax scores: e^(z - max) over the sum of all experts' (the order of the scores is the logits')
+  float z_max = -INFINITY, z_sum = 0.f;
+  if (softmax) {
+    for (int e = lane; e < n_experts; e += 32) z_max = fmaxf(z_max, z[e]);
+    z_max = warp_max(z_max);
+    for (int e = lane; e < n_experts; e += 32) z_sum += expf(z[e] - z_max);
+    z_sum = warp_sum(z_sum);
+  }
+  if (choice.correction) {
+    // z becomes the choice scores, the scores themselves wait in score
+    for (int e = lane; e < n_experts; e += 32) {
+      const float s = softmax ? expf(z[e] - z_max) / z_sum : 1.0f / (1.0f + expf(-z[e]));
+      score[e] = s;
+      z[e] = s + choice.correction[e];
+    }
+    __syncwarp();
+    if (choice.keep < choice.groups) {
+      const int size = n_experts / choice.groups;
+      for (int g = lane; g < choice.groups; g += 32) {
+        float m = -INFINITY;
+        for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, z[e]);
+        group_best[g] = m;
+      }
+      __syncwarp();
+      // the groups that stay are marked by +infinity, which is looked past
+      for (int k = 0; k < choice.keep; ++k) {
+        float best = -INFINITY;
+        int arg = choice.groups;
+        for (int g = lane; g < choice.groups; g += 32)
+          if (group_best[g] > best && group_best[g] != INFINITY) { best = group_best[g]; arg = g; }
+        for (int o = 16; o > 0; o >>= 1) {
+          float ob = __shfl_xor_sync(0xffffffffu, best, o);
+          int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+          if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+        }
+        if (lane == 0 && arg < choice.groups) group_best[arg] = INFINITY;
+        __syncwarp();
+      }
+      for (int e = lane; e < n_experts; e += 32)
+        if (group_best[e / size] != INFINITY) z[e] = -INFINITY;
+      __syncwarp();
+    }
+  }
+  float total = 0.f;
+  for (int k = 0; k < top; ++k) {
+    // the largest logit (or choice score) left; among equal ones the lowest index
+    float best;
+    const int arg = moe_pick(z, n_experts, lane, &best);
+    float s = choice.correction ? score[arg] : softmax ? expf(best - z_max) / z_sum : 1.0f / (1.0f + expf(-best));
+    __syncwarp();
+    total += s;
+    if (lane == 0) {
+      ids[(size_t)t * top + k] = arg;
+      weights[(size_t)t * top + k] = s;
+      z[arg] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  __syncwarp();
+  if (lane < top && (renormalise || weight_scale != 1.0f)) {
+    float wt = weights[(size_t)t * top + lane];
+    if (renormalise) wt /= total + sum_eps;
+    weights[(size_t)t * top + lane] = wt * weight_scale;
+  }
+}
+
 template <typename T, typename W>
 __global__ void moe_route_kernel(const T* __restrict__ h, int width, const W* __restrict__ w, const float* __restrict__ bias,
                                  int n_experts, int top,
@@ -82,71 +153,41 @@ __global__ void moe_route_kernel(const T* __restrict__ h, int width, const W* __
   }
   __syncthreads();
   if (warp == 0) {
-    // softmax scores: e^(z - max) over the sum of all experts' (the order of the scores is the logits')
-    float z_max = -INFINITY, z_sum = 0.f;
-    if (softmax) {
-      for (int e = lane; e < n_experts; e += 32) z_max = fmaxf(z_max, z[e]);
-      z_max = warp_max(z_max);
-      for (int e = lane; e < n_experts; e += 32) z_sum += expf(z[e] - z_max);
-      z_sum = warp_sum(z_sum);
-    }
-    if (choice.correction) {
-      // z becomes the choice scores, the scores themselves wait in score
-      for (int e = lane; e < n_experts; e += 32) {
-        const float s = softmax ? expf(z[e] - z_max) / z_sum : 1.0f / (1.0f + expf(-z[e]));
-        score[e] = s;
-        z[e] = s + choice.correction[e];
-      }
-      __syncwarp();
-      if (choice.keep < choice.groups) {
-        const int size = n_experts / choice.groups;
-        for (int g = lane; g < choice.groups; g += 32) {
-          float m = -INFINITY;
-          for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, z[e]);
-          group_best[g] = m;
-        }
-        __syncwarp();
-        // the groups that stay are marked by +infinity, which is looked past
-        for (int k = 0; k < choice.keep; ++k) {
-          float best = -INFINITY;
-          int arg = choice.groups;
-          for (int g = lane; g < choice.groups; g += 32)
-            if (group_best[g] > best && group_best[g] != INFINITY) { best = group_best[g]; arg = g; }
-          for (int o = 16; o > 0; o >>= 1) {
-            float ob = __shfl_xor_sync(0xffffffffu, best, o);
-            int oa = __shfl_xor_sync(0xffffffffu, arg, o);
-            if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
-          }
-          if (lane == 0 && arg < choice.groups) group_best[arg] = INFINITY;
-          __syncwarp();
-        }
-        for (int e = lane; e < n_experts; e += 32)
-          if (group_best[e / size] != INFINITY) z[e] = -INFINITY;
-        __syncwarp();
-      }
-    }
-    float total = 0.f;
-    for (int k = 0; k < top; ++k) {
-      // the largest logit (or choice score) left; among equal ones the lowest index
-      float best;
-      const int arg = moe_pick(z, n_experts, lane, &best);
-      float s = choice.correction ? score[arg] : softmax ? expf(best - z_max) / z_sum : 1.0f / (1.0f + expf(-best));
-      __syncwarp();
-      total += s;
-      if (lane == 0) {
-        ids[(size_t)t * top + k] = arg;
-        weights[(size_t)t * top + k] = s;
-        z[arg] = -INFINITY;
-      }
-      __syncwarp();
-    }
-    __syncwarp();
-    if (lane < top && (renormalise || weight_scale != 1.0f)) {
-      float wt = weights[(size_t)t * top + lane];
-      if (renormalise) wt /= total + sum_eps;
-      weights[(size_t)t * top + lane] = wt * weight_scale;
-    }
+    moe_choose(z, score, group_best, n_experts, top, renormalise, softmax, weight_scale, sum_eps, choice, t, lane, ids, weights);
   }
+}
+
+// The same from logits that a product has left: a warp per token.  logits [tokens, stride] float32; with choice.gate the logit of
+// the gate follows the experts'.
+#define MOE_CHOOSE_WARPS 4
+__global__ void moe_choose_kernel(const float* __restrict__ logits, int stride, int n_tokens, const float* __restrict__ bias, int n_experts,
+                                  int top, int renormalise, int softmax, float weight_scale, float sum_eps, MoeChoice choice,
+                                  int* __restrict__ ids, float* __restrict__ weights) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float sm[];  // per warp: logits, scores, groups
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x * MOE_CHOOSE_WARPS + warp;
+  if (t >= n_tokens) return;
+  float* z = sm + (size_t)warp * 3 * n_experts;
+  const float* row = logits + (size_t)t * stride;
+  for (int e = lane; e < n_experts; e += 32) z[e] = bias ? row[e] + bias[e] : row[e];
+  if (choice.gate && lane == 0) choice.gate[t] = 1.0f / (1.0f + expf(-row[n_experts]));
+  __syncwarp();
+  moe_choose(z, z + n_experts, z + 2 * n_experts, n_experts, top, renormalise, softmax, weight_scale, sum_eps, choice, t, lane, ids, weights);
+}
+
+extern "C" int bn_moe_choose(const float* logits, int stride, int n_tokens, const float* bias, int n_experts, int top, int renormalise,
+                             int softmax, float weight_scale, float sum_eps, const float* correction, int groups, int keep, float* gate,
+                             int* ids, float* weights, cudaStream_t stream) {
+  if (n_tokens <= 0) return BN_OK;
+  if (!logits || !ids || !weights || n_experts <= 0 || n_experts > MOE_MAX_EXPERTS || stride < n_experts + (gate ? 1 : 0) || top <= 0 ||
+      top > n_experts || top > 32 || groups <= 0 || n_experts % groups || keep <= 0 || keep > groups || (keep < groups && !correction))
+    return BN_ERR_BAD_ARG;
+  const MoeChoice choice = {correction, groups, keep, gate};
+  const size_t smem = (size_t)MOE_CHOOSE_WARPS * 3 * n_experts * sizeof(float);  // at most 48 KB
+  BN_LAUNCH(moe_choose_kernel, (n_tokens + MOE_CHOOSE_WARPS - 1) / MOE_CHOOSE_WARPS, MOE_CHOOSE_WARPS * 32, smem, stream, logits, stride, n_tokens,
+            bias, n_experts, top, renormalise, softmax, weight_scale, sum_eps, choice, ids, weights);
+  return BN_OK;
 }
 
 // softmax: the scores are the softmax over all experts instead of each logit's logistic function; the chosen
@@ -399,8 +440,22 @@ __global__ void moe_scatter_kernel(const T* __restrict__ h, int width, const int
   }
   __syncthreads();
   const float wt = scale_input ? weights[item] : 1.0f;
-  for (int c = threadIdx.x; c < width; c += blockDim.x)
-    x_sorted[(size_t)row * width + c] = from_f32<T>(to_f32<T>(h[(size_t)t * width + c]) * wt);
+  constexpr int V = 16 / (int)sizeof(T);
+  const T* src = h + (size_t)t * width;
+  T* dst = x_sorted + (size_t)row * width;
+  if (width % V == 0 && (((uintptr_t)h | (uintptr_t)x_sorted) & 15) == 0) {  // rows of whole 16-byte pieces
+    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+      uint4 raw = *reinterpret_cast<const uint4*>(src + c);
+      if (scale_input) {
+        T* v = reinterpret_cast<T*>(&raw);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = from_f32<T>(to_f32<T>(v[e]) * wt);
+      }
+      *reinterpret_cast<uint4*>(dst + c) = raw;
+    }
+    return;
+  }
+  for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = from_f32<T>(to_f32<T>(src[c]) * wt);
 }
 
 // out[t] = sum_k (weight) y_sorted[place[t * top + k]] (+ add_scale[t] add[t]), float32; a place below zero: the row of h
@@ -412,6 +467,35 @@ __global__ void moe_gather_kernel(const T* __restrict__ y_sorted, int width, con
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
+  constexpr int V = 16 / (int)sizeof(T);
+  if (width % V == 0 && (!add || add_dtype == BN_F32) &&
+      (((uintptr_t)y_sorted | (uintptr_t)h | (uintptr_t)out | (uintptr_t)add) & 15) == 0) {  // rows of whole 16-byte pieces
+    const float factor = add_scale ? add_scale[t] : 1.0f;
+    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+      float total[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) total[e] = 0.f;
+      for (int k = 0; k < top; ++k) {
+        const int row = place[(size_t)t * top + k];
+        const float wt = scale_output ? weights[(size_t)t * top + k] : 1.0f;
+        const T* src = row >= 0 ? y_sorted + (size_t)row * width : h ? h + (size_t)t * width : nullptr;
+        if (!src) continue;
+        const uint4 raw = *reinterpret_cast<const uint4*>(src + c);
+        const T* v = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int e = 0; e < V; ++e) total[e] = scale_output ? fmaf(to_f32<T>(v[e]), wt, total[e]) : total[e] + to_f32<T>(v[e]);
+      }
+      float4* dst = reinterpret_cast<float4*>(out + (size_t)t * width + c);
+#pragma unroll
+      for (int e = 0; e < V; e += 4) {
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (add) a = *reinterpret_cast<const float4*>((const float*)add + (size_t)t * width + c + e);
+        dst[e / 4] = make_float4(fmaf(a.x, factor, total[e]), fmaf(a.y, factor, total[e + 1]), fmaf(a.z, factor, total[e + 2]),
+                                 fmaf(a.w, factor, total[e + 3]));
+      }
+    }
+    return;
+  }
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
     float total = 0.f;
     for (int k = 0; k < top; ++k) {

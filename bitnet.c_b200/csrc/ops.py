@@ -761,7 +761,7 @@ def attention_prefill_tc(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_he
                          out_scale: float = 1.0) -> torch.Tensor:
     """bfloat16 causal attention of runs of new tokens on tcgen05 tensor cores with TMA-fed operands;
     block i handles up to 128 new tokens of sequence tile_seq[i] from its row tile_row0[i] on.
-    Key and value widths up to 128 (a value head has the width of ``v_cache``'s rows).  ``precise``: the softmax weights
+    Key widths up to 192 and value widths up to 128 (a value head has the width of ``v_cache``'s rows).  ``precise``: the softmax weights
     enter the value product with 16 bits of mantissa instead of 8; ``sink``, ``gate``, an ``out`` of columns and ``out_scale`` as for
     ``attention_general``."""
     if not q.is_cuda or q.dim() != 2 or q.stride(-1) != 1 or q.stride(0) != q_stride or q.dtype != torch.bfloat16:
@@ -780,7 +780,7 @@ def attention_prefill_tc(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_he
     if tuple(k_cache.shape[1:]) != (n_kv_heads, PAGE, head_dim) or k_cache.shape[:3] != v_cache.shape[:3]:
         raise KernelError(f"attention_prefill_tc: cache {tuple(k_cache.shape)} / {tuple(v_cache.shape)} is not "
                           f"[pages, {n_kv_heads}, {PAGE}, {head_dim} / value width]")
-    if head_dim % 16 or head_dim > 128 or v_dim % 16 or v_dim > 128 or n_heads % n_kv_heads:
+    if head_dim % 16 or head_dim > 192 or v_dim % 16 or v_dim > 128 or n_heads % n_kv_heads:
         raise KernelError(f"attention_prefill_tc: head_dim={head_dim}, value width {v_dim}, heads {n_heads}/{n_kv_heads} not supported")
     if sink is not None:
         _need(sink, "sink", torch.float32, 1)
@@ -801,6 +801,43 @@ def attention_prefill_tc(q: torch.Tensor, q_stride: int, out: torch.Tensor, n_he
         _ptr(seq_start), _ptr(seq_pos0), _ptr(slots), _ptr(page_table), int(page_table.shape[1]), _ptr(k_cache),
         _ptr(v_cache), int(k_cache.shape[0]), _ptr(tc_status(q.device)), _stream()), "attention_prefill_tc")
     return out
+
+
+def latent_gather(k_cache: torch.Tensor, rank: int, seen_seq: torch.Tensor, seen_pos: torch.Tensor, slots: torch.Tensor,
+                  page_table: torch.Tensor) -> torch.Tensor:
+    """``[seen, rank]``: the first ``rank`` numbers of the cached rows (one key head) of the positions ``seen_pos`` of the step's
+    sequences ``seen_seq``.  bfloat16, rows of whole 16-byte pieces."""
+    _need(k_cache, "k_cache", torch.bfloat16, 4)
+    _need(page_table, "page_table", torch.int32, 2)
+    for t, nm in ((seen_seq, "seen_seq"), (seen_pos, "seen_pos"), (slots, "slots")):
+        _need(t, nm, torch.int32, 1)
+    row = k_cache.shape[3]
+    if k_cache.shape[1] != 1 or k_cache.shape[2] != PAGE or row % 8 or rank % 8 or not 0 < rank <= row or seen_seq.shape != seen_pos.shape:
+        raise KernelError(f"latent_gather: cache {tuple(k_cache.shape)} does not hold latents of {rank}")
+    out = torch.empty((seen_seq.shape[0], rank), dtype=torch.bfloat16, device=k_cache.device)
+    _check(_fn("latent", "bn_latent_gather")(_ptr(k_cache), int(row), int(rank), _ptr(seen_seq), _ptr(seen_pos), int(seen_seq.shape[0]), _ptr(slots),
+                                             _ptr(page_table), int(page_table.shape[1]), _ptr(out), _stream()), "latent_gather")
+    return out
+
+
+def latent_pages(keys: torch.Tensor, values: torch.Tensor, k_cache: torch.Tensor, rank: int, heads: int, seen_seq: torch.Tensor,
+                 seen_pos: torch.Tensor, slots: torch.Tensor, page_table: torch.Tensor, scratch_table: torch.Tensor,
+                 k_pages: torch.Tensor, v_pages: torch.Tensor) -> None:
+    """Per-head keys and values of the seen positions into scratch pages: ``keys`` ``[seen, heads * dim]`` with the cached row's rotated
+    part behind every head's, ``values`` ``[seen, heads * vdim]``; ``scratch_table``: by the step's sequence and its page, the
+    scratch page."""
+    for t, nm, d in ((keys, "keys", 2), (values, "values", 2), (k_cache, "k_cache", 4), (k_pages, "k_pages", 4), (v_pages, "v_pages", 4)):
+        _need(t, nm, torch.bfloat16, d)
+    for t, nm, d in ((seen_seq, "seen_seq", 1), (seen_pos, "seen_pos", 1), (slots, "slots", 1), (page_table, "page_table", 2),
+                     (scratch_table, "scratch_table", 2)):
+        _need(t, nm, torch.int32, d)
+    n, row, dim, vdim = seen_seq.shape[0], k_cache.shape[3], keys.shape[1] // heads, values.shape[1] // heads
+    if (k_cache.shape[1:3] != (1, PAGE) or keys.shape != (n, heads * dim) or values.shape != (n, heads * vdim) or dim % 8 or vdim % 8 or row % 8
+            or rank % 8 or tuple(k_pages.shape[1:]) != (heads, PAGE, dim + row - rank) or tuple(v_pages.shape[1:]) != (heads, PAGE, vdim)):
+        raise KernelError("latent_pages: sizes do not fit")
+    _check(_fn("latent", "bn_latent_pages")(_ptr(keys), _ptr(values), _ptr(k_cache), int(row), int(rank), int(heads), int(dim), int(vdim),
+                                            _ptr(seen_seq), _ptr(seen_pos), int(n), _ptr(slots), _ptr(page_table), int(page_table.shape[1]),
+                                            _ptr(scratch_table), int(scratch_table.shape[1]), _ptr(k_pages), _ptr(v_pages), _stream()), "latent_pages")
 
 
 DECODE_CHUNK = 128  # positions per block of the decode attention; must equal DEC_CHUNK in attention_decode.cu
@@ -1213,7 +1250,7 @@ def own_gemm_sink_rows(rows: int) -> bool:
 def gemm_tc(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu: bool = False,
             sink: Optional[NormSink] = None, act: int = 0):
     """x[M, K] . w[N, K]^T for many rows in bfloat16 on tcgen05 tensor cores (gemm_tc.cu).  ``x`` may be
-    ``RowScaled``; ``swiglu`` and ``sink`` as for ``linear`` (the activation, or the residual add with
+    ``RowScaled``; ``swiglu``, ACT_RELU2 and ``sink`` as for ``linear`` (the activation, or the residual add with
     the next norm's gain and sums of squares, happen in the product's epilogue)."""
     scaled = x if isinstance(x, RowScaled) else None
     if scaled is not None:
@@ -1253,9 +1290,32 @@ def gemm_tc(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu:
     cols = N // 2 if swiglu else N
     out = torch.empty((M, cols), dtype=out_dtype, device=x.device)
     _check(fn(_ptr(x), _ptr(w), int(M), int(N), int(K), _ptr(out), int(_DT[out_dtype]), int(cols),
-              int((2 | act << 8) if swiglu else 0), *row, c_void_p(None), c_void_p(None), int(0), c_void_p(None), c_void_p(None),
+              int((2 | act << 8) if swiglu else (act << 8 if act == ACT_RELU2 else 0)), *row, c_void_p(None), c_void_p(None), int(0), c_void_p(None), c_void_p(None),
               int(0), status, _stream()), "gemm_tc")
     return out
+
+
+GROUPED_MAX = 1024  # groups of a grouped product (GM_MAX_GROUPS in gemm_tc.cu)
+
+
+def grouped_product(x: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, act: int = 0) -> torch.Tensor:
+    """``[rows, N]``: rows ``offsets[g] .. offsets[g + 1]`` of x times ``w[g]`` ``[N, K]`` transposed, for all groups in one launch
+    (gemm_tc.cu); bfloat16.  ``offsets`` int32 ``[groups + 1]`` on the device; rows past its last number hold nothing.  ``act``
+    ACT_RELU2: the square of the results' positive part."""
+    _need(x, "x", torch.bfloat16, 2)
+    _need(w, "w", torch.bfloat16, 3)
+    _need(offsets, "offsets", torch.int32, 1)
+    G, N, K = w.shape
+    if x.shape[1] != K or offsets.shape[0] != G + 1 or not grouped_fits(w) or act not in (0, ACT_RELU2):
+        raise KernelError(f"grouped_product: x {tuple(x.shape)}, w {tuple(w.shape)}, {offsets.shape[0]} offsets do not fit")
+    out = torch.empty((x.shape[0], N), dtype=torch.bfloat16, device=x.device)
+    _check(_fn("gemm_tc", "bn_gemm_tc_grouped")(_ptr(x), _ptr(w), int(x.shape[0]), int(G), int(N), int(K), _ptr(offsets), _ptr(out), int(act),
+                                                _ptr(tc_status(x.device)), _stream()), "gemm_tc_grouped")
+    return out
+
+
+def grouped_fits(w: torch.Tensor) -> bool:
+    return w.dtype == torch.bfloat16 and w.shape[0] <= GROUPED_MAX and w.shape[1] % 8 == 0 and w.shape[2] % 8 == 0
 
 
 def gemm_pairs(on: Optional[bool] = None) -> bool:
@@ -1327,7 +1387,7 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu: 
     if isinstance(x, RowScaled):
         if fast:
             return linear_tc(x, w, out_dtype=out_dtype or x.dtype, swiglu=swiglu, _checked=True, act=act, bias=bias)
-        if _own_gemm_fits(x.x, w, swiglu, out_dtype, "scaled") and not partial_sums and bias is None and not squared:
+        if _own_gemm_fits(x.x, w, swiglu, out_dtype, "scaled") and not partial_sums and bias is None:
             return gemm_tc(x, w, out_dtype=out_dtype or x.dtype, swiglu=swiglu, act=act)
         x = x.dense()
     _need(x, "x", dims=2)
@@ -1336,7 +1396,7 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None, swiglu: 
         x = x.to(w.dtype)
     if streams:
         return linear_tc(x, w, out_dtype=out_dtype, swiglu=swiglu, _checked=True, act=act, bias=bias)
-    if _own_gemm_fits(x, w, swiglu, out_dtype, "swiglu" if swiglu else "plain") and not partial_sums and bias is None and not squared:
+    if _own_gemm_fits(x, w, swiglu, out_dtype, "swiglu" if swiglu or squared else "plain") and not partial_sums and bias is None:
         return gemm_tc(x, w, out_dtype=out_dtype, swiglu=swiglu, act=act)
     if small:
         fn = _fn("linear_mma", "bn_linear_mma")
@@ -2022,6 +2082,31 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, top: int, renormalise: bo
     return (ids, weights, g) if gate else (ids, weights)
 
 
+def moe_choose(logits: torch.Tensor, n_experts: int, top: int, renormalise: bool = False, softmax: bool = False, weight_scale: float = 1.0,
+               sum_eps: float = 0.0, bias: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None, groups: int = 1,
+               keep: int = 1, gate: bool = False):
+    """``moe_route`` behind a product of its own: float32 ``logits`` ``[T, at least n_experts]`` (with ``gate`` the gate's logit
+    follows the experts')."""
+    _need(logits, "logits", torch.float32, 2)
+    T = logits.shape[0]
+    if logits.shape[1] < n_experts + int(bool(gate)) or not 0 < top <= min(n_experts, 32) or n_experts > 1024:
+        raise KernelError(f"moe_choose: logits {tuple(logits.shape)} do not hold {n_experts} experts, top {top}")
+    for t, nm in ((bias, "bias"), (correction, "correction")):
+        if t is not None:
+            _need(t, nm, torch.float32, 1)
+            if t.shape[0] != n_experts:
+                raise KernelError(f"moe_choose: {t.shape[0]} numbers of {nm} for {n_experts} experts")
+    if groups < 1 or n_experts % groups or not 0 < keep <= groups or (keep < groups and (correction is None or keep * (n_experts // groups) < top)):
+        raise KernelError(f"moe_choose: {n_experts} experts cannot be chosen {top} at a time from {keep} of {groups} groups")
+    ids = torch.empty((T, top), dtype=torch.int32, device=logits.device)
+    weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
+    g = torch.empty(T, dtype=torch.float32, device=logits.device) if gate else None
+    _check(_fn("moe", "bn_moe_choose")(_ptr(logits), int(logits.shape[1]), int(T), _ptr(bias), int(n_experts), int(top), int(bool(renormalise)),
+                                       int(bool(softmax)), c_float(weight_scale), c_float(sum_eps), _ptr(correction), int(groups), int(keep),
+                                       _ptr(g), _ptr(ids), _ptr(weights), _stream()), "moe_choose")
+    return (ids, weights, g) if gate else (ids, weights)
+
+
 def moe_table_route(tokens: torch.Tensor, table: torch.Tensor, top: int, n_experts: int):
     """Experts by token id: ``(ids int32 [T, top], weights float32 [T, top])`` with ids = ``table[token, :top]`` and
     every weight 1 / top (an id or an entry out of range takes weight 0)."""
@@ -2136,7 +2221,7 @@ def moe_gather(y_sorted: torch.Tensor, place: torch.Tensor, weights: torch.Tenso
     _need(weights, "weights", torch.float32, 2)
     T, top = weights.shape
     width = y_sorted.shape[1]
-    if y_sorted.shape[0] < T * top or place.shape[0] != T * top:
+    if (h is None and y_sorted.shape[0] < T * top) or place.shape[0] != T * top:  # (items of identity experts have no row)
         raise KernelError("moe_gather: sizes do not fit")
     if add is not None:
         _need(add, "add", dims=2)

@@ -26,16 +26,17 @@ class LatentAttention(Mixer):
     the head's output in the latent space, and W_uv brings it back (another small product per head).  The
     values are a part of the key rows, so the cache holds no value plane.
 
-    Runs of new tokens whose key rows are too wide for the tensor-core kernel (more than 256 numbers) take the
-    other order: the rows every new token sees are read back from the cache, W_uk and W_uv make per-head keys
-    [W_uk c | k_rot] and values of them (two products over all those rows), which go into scratch pages of the
-    step, and the tensor-core kernel runs on these with the queries as projected.
+    Runs of new tokens take the other order where the tcgen05 kernel has room for a head's keys (192 numbers) and values (128),
+    or the key rows are too wide for the mma.sync one (more than 256 numbers): the rows every new token sees are read back
+    from the cache, W_uk and W_uv make per-head keys [W_uk c | k_rot] and values of them (two products over all those
+    rows), which go into scratch pages of the step, and the attention runs on these with the queries as projected.
 
     A run without a latent of its own (``own_kv`` False) reads the rows of the run its schedule entry names, with its own
     queries, W_uk and W_uv."""
 
-    kernels = ("linear", "linear_mma", "linear_tc", "gemm_tc", "attention", "attention_prefill", "rotary_pairs", "norm")
+    kernels = ("linear", "linear_mma", "linear_tc", "gemm_tc", "attention", "attention_prefill", "attention_prefill_tc", "rotary_pairs", "norm", "latent")
     TILED_MIN_TOKENS = 16  # runs of new tokens from this many on take the tensor-core kernel (bfloat16)
+    SEEN_PER_NEW = 64  # keys and values are made per head while a step's tokens see at most so many rows each, on average
     graph_safe = True
 
     def __init__(self, spec, build):
@@ -48,6 +49,11 @@ class LatentAttention(Mixer):
             raise ValueError("latent_attention: a gate per head or a gate per output number, not both")
         if spec.kv_rank + spec.rot_dim > 2048:
             raise ValueError(f"latent_attention: kv_rank + rot_dim = {spec.kv_rank + spec.rot_dim} must be at most 2048")
+        s = spec
+        # which forms of attention over runs of tokens its sizes allow
+        self.per_head = (build.dtype == torch.bfloat16 and (s.head_dim + s.rot_dim) % 16 == 0 and s.v_head_dim % 16 == 0
+                         and max(s.head_dim + s.rot_dim, s.v_head_dim) <= 256 and not (s.head_dim % 8 or s.rot_dim % 8 or s.kv_rank % 8))
+        self.on_tcgen05 = self.per_head and ops.USE_TCGEN05_ATTENTION and s.head_dim + s.rot_dim <= 192 and s.v_head_dim <= 128 and s.scale > 0
         self.position = build_part("position", spec.position, build)
         self.w_dq: Optional[torch.Tensor] = None
 
@@ -142,8 +148,9 @@ class LatentAttention(Mixer):
         tiled = dt == torch.bfloat16 and not ctx.decode and ctx.tile_seq is not None and ctx.max_new >= self.TILED_MIN_TOKENS
         if q_off:
             q = q[:, q_off: q_off + H * (d + dr)]
-        if (tiled and (row > 256 or row % 16 or rank % 16) and (d + dr) % 16 == 0 and s.v_head_dim % 16 == 0 and d + dr <= 256
-                and s.v_head_dim <= 256 and ctx.host_new):
+        in_latent_space = row <= 256 and row % 16 == 0 and rank % 16 == 0  # the tensor-core kernel takes the cached rows as they are
+        if (tiled and self.per_head and ctx.host_new and q.stride(0) % 8 == 0
+                and (not in_latent_space or self.on_tcgen05 and sum(ctx.host_pos0) <= (self.SEEN_PER_NEW - 1) * ctx.n_tokens)):
             return self._per_head_keys(q, gate, ctx, kv, egate)
         # queries in the latent space: [W_uk^T q_plain | q_rot] per head
         q3 = q.unflatten(1, (H, d + dr))
@@ -153,7 +160,7 @@ class LatentAttention(Mixer):
         if ctx.diag is not None:
             ctx.tap("attn_q", lambda: ql.view(n, H * row))
         out = torch.empty((n, H * rank), dtype=dt, device=h.device)
-        if tiled and row % 16 == 0 and rank % 16 == 0 and row <= 256:
+        if tiled and in_latent_space:
             # runs of new tokens: 64 tokens of a sequence and a head per block on the tensor cores, the
             # softmax weights with 16 bits of mantissa
             ops.attention_prefill(ql, H * row, out, H, 1, row, s.scale, s.window, ctx.tile_seq, ctx.tile_row0, ctx.seq_start,
@@ -182,8 +189,8 @@ class LatentAttention(Mixer):
             seq, pos, spans = [], [], []
             for i, (p0, n) in enumerate(zip(ctx.host_pos0, ctx.host_new)):
                 lo = max(0, p0 - w + 1) if w > 0 else 0
-                seq.append(np.full(p0 + n - lo, i, dtype=np.int64))
-                pos.append(np.arange(lo, p0 + n, dtype=np.int64))
+                seq.append(np.full(p0 + n - lo, i, dtype=np.int32))
+                pos.append(np.arange(lo, p0 + n, dtype=np.int32))
                 spans.append((lo // ops.PAGE, (p0 + n - 1) // ops.PAGE))
             table = np.zeros((len(spans), max(b for _a, b in spans) + 1), dtype=np.int32)
             at = 0
@@ -200,22 +207,23 @@ class LatentAttention(Mixer):
         H, d, dr, dv, rank = s.n_heads, s.head_dim, s.rot_dim, s.v_head_dim, s.kv_rank
         dt, dev = self.build.dtype, q.device
         seq, pos, table, n_pages, rows_of = self._seen_rows(ctx, dev)
-        page, r = pos // ops.PAGE, pos % ops.PAGE
-        rows = kv.k[kv.page_table[ctx.slots[seq].long(), page].long(), 0, r]  # [seen, latent | rotated key part]
-        c = rows[:, :rank].contiguous()
-        keys = torch.empty((rows.shape[0], H, d + dr), dtype=dt, device=dev)
-        keys[:, :, :d] = ops.linear(c, self.w_uk_flat, out_dtype=dt).view(-1, H, d)
-        keys[:, :, d:] = rows[:, None, rank:]
-        values = ops.linear(c, self.w_uv_flat, out_dtype=dt).view(-1, H, dv)
-        # scratch pages start as zeros: rows of a page that no position fills are masked, and zero times them is zero
-        k_s = torch.zeros((n_pages, H, ops.PAGE, d + dr), dtype=dt, device=dev)
-        v_s = torch.zeros((n_pages, H, ops.PAGE, dv), dtype=dt, device=dev)
-        to = table[seq, page].long()
-        k_s[to, :, r] = keys
-        v_s[to, :, r] = values
+        c = ops.latent_gather(kv.k, rank, seq, pos, ctx.slots, kv.page_table)
+        keys, values = ops.linear(c, self.w_uk_flat, out_dtype=dt), ops.linear(c, self.w_uv_flat, out_dtype=dt)
+        on_tcgen05 = self.on_tcgen05 and ctx.wide_tile_seq is not None and q.dim() == 2
+        # rows of a page that no position fills are masked, but zero times what lies there must be zero: scratch pages start as
+        # zeros where the kernel does not see to it (it does for what lies behind a sequence's last position on tcgen05)
+        new = torch.empty if on_tcgen05 and s.window <= 0 else torch.zeros
+        k_s = new((n_pages, H, ops.PAGE, d + dr), dtype=dt, device=dev)
+        v_s = new((n_pages, H, ops.PAGE, dv), dtype=dt, device=dev)
+        ops.latent_pages(keys, values, kv.k, rank, H, seq, pos, ctx.slots, kv.page_table, table, k_s, v_s)
         out = torch.empty((q.shape[0], H * dv), dtype=dt, device=dev)
-        ops.attention_prefill(q, q.stride(0), out, H, H, d + dr, s.scale, s.window, ctx.tile_seq, ctx.tile_row0, ctx.seq_start,
-                              ctx.seq_pos0, rows_of, table, k_s, v_s, gate=gate, gate_stride=self.row, precise=True, sink=self.sink)
+        if on_tcgen05:
+            ops.attention_prefill_tc(q, q.stride(0), out, H, H, d + dr, s.scale, s.window, ctx.wide_tile_seq, ctx.wide_tile_row0,
+                                     ctx.seq_start, ctx.seq_pos0, rows_of, table, k_s, v_s, precise=True, sink=self.sink, gate=gate,
+                                     gate_stride=self.row)
+        else:
+            ops.attention_prefill(q, q.stride(0), out, H, H, d + dr, s.scale, s.window, ctx.tile_seq, ctx.tile_row0, ctx.seq_start,
+                                  ctx.seq_pos0, rows_of, table, k_s, v_s, gate=gate, gate_stride=self.row, precise=True, sink=self.sink)
         ctx.tap("attn_out", out)
         if egate is not None:
             ops.gate_rows(out, egate)

@@ -27,12 +27,14 @@ class Moe(FeedForward):
     logistic function of one number per token, a row of the router's product.
 
     Few rows (a decode step): two kernels stream the chosen experts once per (token, expert), from
-    device memory alone.  Many rows: the (token, expert) items are sorted by expert and every expert's
-    rows go through the ordinary products; the host then needs the experts' row counts, one copy per call."""
+    device memory alone.  Many rows: the (token, expert) items are sorted by expert, and in bfloat16 all experts run as one
+    grouped product each way, which reads the experts' row counts on the device.  Otherwise (float32, odd sizes) every
+    expert's rows go through the ordinary products; the host then needs the counts, one copy per call."""
 
     kernels = ("linear", "linear_mma", "linear_tc", "gemm_tc", "act", "moe")
     graph_safe = True  # the steps that are recorded are decode steps, which take the path without the host
     FEW_ITEMS = 64  # up to so many (token, expert) items the streaming kernels run
+    USE_GROUPED = True  # (tests and comparisons set it to False)
     PAD_FACTOR = 2.0  # blocks of equal size for all experts while they hold at most so many times the rows used
 
     def __init__(self, spec, build):
@@ -102,6 +104,9 @@ class Moe(FeedForward):
             r, g = self.w_router, tensors["shared.sg"]
             wd = r.dtype if r.dtype == g.dtype else torch.float32
             self.w_router = torch.cat([r.to(wd), g.to(wd)]).contiguous()
+        if self.w_router is not None and self.w_router.shape[0] % 8:  # rows of the product's result stay whole pieces
+            pad = torch.zeros((-self.w_router.shape[0] % 8, s.width), dtype=self.w_router.dtype, device=self.w_router.device)
+            self.w_router = torch.cat([self.w_router, pad])
         self.correction = tensors["correction"].float().contiguous() if s.correction else None
         self.b_router = tensors["router.b"].float().contiguous() if s.router_bias else None
         self.table = tensors.get("table")
@@ -132,10 +137,11 @@ class Moe(FeedForward):
                 ctx.memo[key] = ops.moe_table_route(ctx.tokens, self.table, s.top, s.n_experts)
             ids, weights = ctx.memo[key]
         else:
-            ids, weights, *gate = ops.moe_route(
-                h, self.w_router, s.top, s.renormalise, softmax=self.softmax, weight_scale=getattr(s, "weight_scale", 1.0),
-                sum_eps=getattr(s, "renormalise_eps", 0.0), bias=self.b_router, correction=self.correction, groups=s.groups,
-                keep=s.keep_groups, gate=s.shared_gate)
+            # the logits are a product of the library's own for few rows; only then the choice is made
+            logits = ops.linear(h, self.w_router, out_dtype=torch.float32)
+            ids, weights, *gate = ops.moe_choose(
+                logits, self.outputs, s.top, s.renormalise, softmax=self.softmax, weight_scale=s.weight_scale, sum_eps=s.renormalise_eps,
+                bias=self.b_router, correction=self.correction, groups=s.groups, keep=s.keep_groups, gate=s.shared_gate)
             if gate:
                 shared_scale = gate[0]
         if ctx.diag is not None:
@@ -144,6 +150,13 @@ class Moe(FeedForward):
             return ops.moe_experts_few(h, ids, weights, self.w_gate_up, self.w_down, s.expert_limit, s.slope,
                                        s.weight_on_input, add=shared, act=self.act, add_scale=shared_scale)
         counts = ops.moe_count(ids, s.n_experts)
+        rest = dict(add_scale=shared_scale, h=h if s.identity else None)
+        if self.USE_GROUPED and h.dtype == torch.bfloat16 and ops.grouped_fits(self.w_gate_up) and ops.grouped_fits(self.w_down):
+            x_sorted, place, offsets = ops.moe_sort(h, ids, weights, counts, s.weight_on_input)
+            up = ops.grouped_product(x_sorted, self.w_gate_up, offsets, act=0 if self.gated else ops.ACT_RELU2)
+            act = self._activate(up, s.expert_limit) if self.gated else up
+            y_sorted = ops.grouped_product(act, self.w_down, offsets)
+            return ops.moe_gather(y_sorted, place, weights, not s.weight_on_input, add=shared, **rest)
         host_tokens = getattr(ctx, "host_tokens", None)
         if self.by_table and host_tokens is not None:
             # chosen by token id: the counts follow from the step's ids on the host, nobody waits for the device
@@ -158,7 +171,6 @@ class Moe(FeedForward):
         else:
             per_expert = counts.cpu().tolist()  # the one place where the host waits for the device
         dt, dev_ = self.build.dtype, h.device
-        rest = dict(add_scale=shared_scale, h=h if s.identity else None)
         cap = max(-(-max(per_expert) // 8) * 8, 8)
         if cap * s.n_experts <= self.PAD_FACTOR * T * s.top:
             # the experts are about evenly used: each gets a block of ``cap`` rows, and all of them run as
