@@ -47,7 +47,7 @@ struct GatedLinearArgs {
   __device__ __forceinline__ float* ring(int s) const { return own(s) + width; }
 };
 
-__device__ __forceinline__ float gl_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float gl_sigmoid(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
 __device__ __forceinline__ float gl_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 // (log decay, what enters the state) from the gates' pre-activations; sp = softplus(lam)
@@ -57,50 +57,75 @@ __device__ __forceinline__ float2 gl_step(float zr, float zi, float u, float sp)
 }
 
 // ---- runs of tokens -------------------------------------------------------------------------------------
-// V neighbouring channels of one token per thread
+// A block takes a piece of a run and GL_CONV_COLS * V channels; a thread four neighbouring tokens of V neighbouring channels, so
+// that a row is read once for the (up to) four outputs that look at it.
+#define GL_CONV_COLS 16
+#define GL_CONV_ROWS 4
 template <typename T, int V>
-__global__ void gated_linear_conv_kernel(const GatedLinearArgs a, T* __restrict__ u) {
+__device__ __forceinline__ void gl_load(const T* p, float* o) {
+  if constexpr (V * sizeof(T) == 16) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const T* v = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+    for (int e = 0; e < V; ++e) o[e] = to_f32<T>(v[e]);
+  } else {
+#pragma unroll
+    for (int e = 0; e < V; ++e) o[e] = to_f32<T>(p[e]);
+  }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(GL_CONV_COLS * GL_PIECE / GL_CONV_ROWS)
+gated_linear_conv_kernel(const GatedLinearArgs a, const int* __restrict__ tile_seq, const int* __restrict__ tile_row0, T* __restrict__ u) {
   pdl_launch_dependents();
+  __shared__ __align__(16) float w[GL_MAX_TAPS][GL_CONV_COLS * V];
+  const int c_block = blockIdx.y * GL_CONV_COLS * V;
+  for (int i = threadIdx.x; i < a.taps * GL_CONV_COLS * V; i += blockDim.x) {
+    const int j = i / (GL_CONV_COLS * V), d = i - j * GL_CONV_COLS * V;
+    w[j][d] = c_block + d < a.width ? a.conv_w[(size_t)j * a.width + c_block + d] : 0.f;
+  }
+  __syncthreads();
   pdl_wait();
-  const int t = blockIdx.x, s = a.tok_seq[t], start = a.seq_start[s], r = t - start, pos = a.seq_pos0[s] + r;
+  const int s = tile_seq[blockIdx.x], start = a.seq_start[s], n = a.seq_start[s + 1] - start, pos0 = a.seq_pos0[s];
+  const int d = (threadIdx.x % GL_CONV_COLS) * V, c = c_block + d;
+  const int r0 = tile_row0[blockIdx.x] + threadIdx.x / GL_CONV_COLS * GL_CONV_ROWS;  // the thread's first row of the run
+  if (c >= a.width || r0 >= n) return;
   const T* x = (const T*)a.x;
   const float* ring = a.ring(s);
-  for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * V; c < a.width; c += gridDim.y * blockDim.x * V) {
-    float acc[V];
+  float acc[GL_CONV_ROWS][V];
 #pragma unroll
-    for (int e = 0; e < V; ++e) acc[e] = a.conv_b[c + e];
-    for (int j = 0; j < a.taps; ++j) {
-      const int back = a.taps - 1 - j;  // how many positions before this token the tap looks
-      if (back > pos) continue;
-      const float* w = a.conv_w + (size_t)j * a.width + c;
-      if (r - back >= 0) {
-        const T* p = x + (size_t)(t - back) * a.stride + c;
-        if (V == 4 && sizeof(T) == 2) {
-          const uint2 raw = *reinterpret_cast<const uint2*>(p);
-          const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-          const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-          acc[0] = fmaf(w[0], lo.x, acc[0]); acc[1 % V] = fmaf(w[1 % V], lo.y, acc[1 % V]);
-          acc[2 % V] = fmaf(w[2 % V], hi.x, acc[2 % V]); acc[3 % V] = fmaf(w[3 % V], hi.y, acc[3 % V]);
-        } else {
+  for (int o = 0; o < GL_CONV_ROWS; ++o)
 #pragma unroll
-          for (int e = 0; e < V; ++e) acc[e] = fmaf(w[e], to_f32<T>(p[e]), acc[e]);
-        }
-      } else {
-        const float* p = ring + (size_t)((pos - back) % a.taps) * a.width + c;
+    for (int e = 0; e < V; ++e) acc[o][e] = a.conv_b[c + e];
+#pragma unroll 4
+  for (int i = 1 - a.taps; i < GL_CONV_ROWS; ++i) {
+    const int r = r0 + i;
+    if (r >= n || pos0 + r < 0) continue;  // behind the run, or before the sequence
+    float xv[V];
+    if (r >= 0) gl_load<T, V>(x + (size_t)(start + r) * a.stride + c, xv);
+    else gl_load<float, V>(ring + (size_t)((pos0 + r) % a.taps) * a.width + c, xv);
 #pragma unroll
-        for (int e = 0; e < V; ++e) acc[e] = fmaf(w[e], p[e], acc[e]);
+    for (int o = 0; o < GL_CONV_ROWS; ++o) {
+      const int j = a.taps - 1 - (o - i);  // the tap of output o that looks at this row
+      if (o >= i && j >= 0) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc[o][e] = fmaf(w[j][d + e], xv[e], acc[o][e]);
       }
     }
-    T* dst = u + (size_t)t * a.width + c;
-    if (V == 4 && sizeof(T) == 2) {
-      const __nv_bfloat162 p = __floats2bfloat162_rn(acc[0], acc[1 % V]), q = __floats2bfloat162_rn(acc[2 % V], acc[3 % V]);
-      uint2 raw;
-      raw.x = *reinterpret_cast<const unsigned*>(&p);
-      raw.y = *reinterpret_cast<const unsigned*>(&q);
-      *reinterpret_cast<uint2*>(dst) = raw;
+  }
+#pragma unroll
+  for (int o = 0; o < GL_CONV_ROWS; ++o) {
+    if (r0 + o >= n) break;
+    T* dst = u + (size_t)(start + r0 + o) * a.width + c;
+    if constexpr (V * sizeof(T) == 16) {
+      uint4 raw;
+      T* v = reinterpret_cast<T*>(&raw);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] = from_f32<T>(acc[o][e]);
+      *reinterpret_cast<uint4*>(dst) = raw;
     } else {
 #pragma unroll
-      for (int e = 0; e < V; ++e) dst[e] = from_f32<T>(acc[e]);
+      for (int e = 0; e < V; ++e) dst[e] = from_f32<T>(acc[o][e]);
     }
   }
 }
@@ -135,25 +160,35 @@ __global__ void __launch_bounds__(GL_THREADS) gated_linear_piece_kernel(const Ga
   const T* yt = (const T*)a.y + (size_t)first * a.stride + c;
   float* mine = piece_sums + (size_t)piece * 2 * a.width + c;
   float S = OUT ? mine[a.width] : 0.f, L = 0.f;
-  // eight tokens at a time: their loads are in flight together
+  // eight tokens at a time, the next eight on their way meanwhile
   constexpr int B = 8;
-  for (int t0 = 0; t0 < n_tok; t0 += B) {
-    float zr[B], zi[B], uu[B], yy[B];
+  float zr[2][B], zi[2][B], uu[2][B], yy[2][B];
+  auto fetch = [&](int t0, int buf) {
 #pragma unroll
     for (int e = 0; e < B; ++e) {
       const int t = min(t0 + e, n_tok - 1);
-      zr[e] = g[(size_t)t * 2 * wb];
-      zi[e] = g[(size_t)t * 2 * wb + wb];
-      uu[e] = to_f32<T>(ut[(size_t)t * a.width]);
-      yy[e] = OUT ? to_f32<T>(yt[(size_t)t * a.stride]) : 0.f;
+      zr[buf][e] = g[(size_t)t * 2 * wb];
+      zi[buf][e] = g[(size_t)t * 2 * wb + wb];
+      uu[buf][e] = to_f32<T>(ut[(size_t)t * a.width]);
+      yy[buf][e] = OUT ? to_f32<T>(yt[(size_t)t * a.stride]) : 0.f;
     }
+  };
+  fetch(0, 0);
+  for (int t2 = 0; t2 < n_tok; t2 += 2 * B) {
 #pragma unroll
-    for (int e = 0; e < B; ++e) {
-      if (t0 + e < n_tok) {
-        const float2 st = gl_step(zr[e] + br, zi[e] + bi, uu[e], sp);
-        S = fmaf(expf(st.x), S, st.y);
-        if (OUT) out[(size_t)(first + t0 + e) * a.out_stride + c] = from_f32<T>(a.scale * glu_activation(yy[e], BN_ACT_GELU_TANH) * S);
-        else L += st.x;
+    for (int half = 0; half < 2; ++half) {
+      const int t0 = t2 + half * B;
+      if (t0 + B < n_tok) fetch(t0 + B, half ^ 1);
+#pragma unroll
+      for (int e = 0; e < B; ++e) {
+        if (t0 + e < n_tok) {
+          const float2 st = gl_step(zr[half][e] + br, zi[half][e] + bi, uu[half][e], sp);
+          S = fmaf(expf(st.x), S, st.y);
+          if (OUT)
+            out[(size_t)(first + t0 + e) * a.out_stride + c] = from_f32<T>(a.scale * glu_activation(yy[half][e], BN_ACT_GELU_TANH) * S);
+          else
+            L += st.x;
+        }
       }
     }
   }
@@ -205,21 +240,38 @@ __global__ void __launch_bounds__(GL_THREADS) gated_linear_carry_kernel(const Ga
 }
 
 // ---- one token per sequence --------------------------------------------------------------------------------
-#define GL_SEQS 8      // sequences a block takes at a time
-#define GL_CHANNELS 16 // channels per block: two per warp
+#define GL_SEQS 8        // sequences a block takes at a time
+#define GL_CHANNELS 8    // channels per block: one per warp
+#define GL_AHEAD 8       // numbers of each row of R and I that a lane asks for before the step's inputs are there
 
-// A block per (part, 16 of its channels): the convolution of the whole part for eight sequences at a time into shared memory,
+// A block per (part, 8 of its channels): the convolution of the whole part for eight sequences at a time into shared memory,
 // then a warp per channel takes its rows of R and I (w_gates [blocks][2 wb][wb], r's rows first) against all of them, and
 // lane s does sequence s's step.
 template <typename T>
 __global__ void __launch_bounds__(256) gated_linear_token_kernel(const GatedLinearArgs a, const T* __restrict__ w_gates) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float us[];  // [GL_SEQS][wb padded to 4]
+  __shared__ int seq_pos[GL_SEQS], seq_row[GL_SEQS];
+  __shared__ float* seq_own[GL_SEQS];
   const int wb = a.width / a.blocks, ld = (wb + 3) / 4 * 4;
   const int b = blockIdx.x, d0 = blockIdx.y * GL_CHANNELS;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const T* x = (const T*)a.x;
   T* out = (T*)a.out;
+  // the warp's channel and what of it are weights
+  const int d = d0 + warp, c = b * wb + d;
+  const bool live = d < wb;
+  const T* rr = w_gates + ((size_t)b * 2 * wb + (live ? d : 0)) * wb;
+  const T* ri = rr + (size_t)wb * wb;
+  float wr[GL_AHEAD], wi[GL_AHEAD];
+#pragma unroll
+  for (int k = 0; k < GL_AHEAD; ++k) {
+    const int jj = lane + 32 * k;
+    wr[k] = jj < wb ? to_f32<T>(rr[jj]) : 0.f;
+    wi[k] = jj < wb ? to_f32<T>(ri[jj]) : 0.f;
+  }
+  const float br = live ? a.gate_b[(size_t)b * 2 * wb + d] : 0.f, bi = live ? a.gate_b[(size_t)b * 2 * wb + wb + d] : 0.f;
+  const float sp = live ? gl_softplus(a.lam[c]) : 0.f;
   pdl_wait();
   if (a.tail > 0 && blockIdx.x == 0 && blockIdx.y == 0)
     for (int i = threadIdx.x; i < a.n_seqs * a.tail; i += blockDim.x) {
@@ -229,57 +281,75 @@ __global__ void __launch_bounds__(256) gated_linear_token_kernel(const GatedLine
   for (int s0 = 0; s0 < a.n_seqs; s0 += GL_SEQS) {
     const int ns = min(GL_SEQS, a.n_seqs - s0);
     __syncthreads();  // the sequences before are done with the inputs
+    if (threadIdx.x < ns) {
+      const int s = s0 + threadIdx.x;
+      seq_pos[threadIdx.x] = a.seq_pos0[s];
+      seq_row[threadIdx.x] = a.seq_start[s];
+      seq_own[threadIdx.x] = a.own(s);
+    }
+    __syncthreads();
+    // lane s: sequence s's state and output gate, on their way during the convolution
+    float S = 0.f, y = 0.f;
+    if (live && lane < ns) {
+      S = seq_own[lane][c];
+      y = to_f32<T>(((const T*)a.y)[(size_t)seq_row[lane] * a.stride + c]);
+    }
+#pragma unroll 4
     for (int i = threadIdx.x; i < GL_SEQS * ld; i += blockDim.x) {
-      const int q = i / ld, d = i - q * ld;
+      const int q = i / ld, dd = i - q * ld;
       float acc = 0.f;
-      if (q < ns && d < wb) {
-        const int s = s0 + q, pos = a.seq_pos0[s], c = b * wb + d;
-        float* ring = a.ring(s);
-        const float now = to_f32<T>(x[(size_t)a.seq_start[s] * a.stride + c]);
-        acc = fmaf(a.conv_w[(size_t)(a.taps - 1) * a.width + c], now, a.conv_b[c]);
-        for (int j = 0; j < a.taps - 1; ++j) {
-          const int p = pos - (a.taps - 1 - j);
-          if (p >= 0) acc = fmaf(a.conv_w[(size_t)j * a.width + c], ring[(size_t)(p % a.taps) * a.width + c], acc);
+      if (q < ns && dd < wb) {
+        const int pos = seq_pos[q], cc = b * wb + dd;
+        float* ring = seq_own[q] + a.width;
+        const float now = to_f32<T>(x[(size_t)seq_row[q] * a.stride + cc]);
+        acc = fmaf(a.conv_w[(size_t)(a.taps - 1) * a.width + cc], now, a.conv_b[cc]);
+        int row = pos % a.taps;  // of this token; the token `back` before it lies `back` rows in front
+        if (a.taps > 1 && dd >= d0 && dd < d0 + GL_CHANNELS) ring[(size_t)row * a.width + cc] = now;
+        for (int back = 1; back < a.taps && back <= pos; ++back) {
+          row = row == 0 ? a.taps - 1 : row - 1;
+          acc = fmaf(a.conv_w[(size_t)(a.taps - 1 - back) * a.width + cc], ring[(size_t)row * a.width + cc], acc);
         }
-        if (a.taps > 1 && d >= d0 && d < d0 + GL_CHANNELS) ring[(size_t)(pos % a.taps) * a.width + c] = now;
         acc = to_f32<T>(from_f32<T>(acc));
       }
       us[i] = acc;
     }
     __syncthreads();
-    for (int k = 0; k < GL_CHANNELS / 8; ++k) {
-      const int d = d0 + warp + 8 * k;
-      if (d >= wb) continue;
-      const T* rr = w_gates + ((size_t)b * 2 * wb + d) * wb;
-      const T* ri = rr + (size_t)wb * wb;
-      float zr[GL_SEQS], zi[GL_SEQS];
+    if (!live) continue;
+    float zr[GL_SEQS], zi[GL_SEQS];
 #pragma unroll
-      for (int q = 0; q < GL_SEQS; ++q) zr[q] = zi[q] = 0.f;
-      for (int j = lane; j < wb; j += 32) {
-        const float wr = to_f32<T>(rr[j]), wi = to_f32<T>(ri[j]);
+    for (int q = 0; q < GL_SEQS; ++q) zr[q] = zi[q] = 0.f;
+#pragma unroll
+    for (int k = 0; k < GL_AHEAD; ++k) {
+      const int j = lane + 32 * k;
+      if (j < wb) {
 #pragma unroll
         for (int q = 0; q < GL_SEQS; ++q) {
           const float v = us[q * ld + j];
-          zr[q] = fmaf(wr, v, zr[q]);
-          zi[q] = fmaf(wi, v, zi[q]);
+          zr[q] = fmaf(wr[k], v, zr[q]);
+          zi[q] = fmaf(wi[k], v, zi[q]);
         }
       }
-      float my_r = 0.f, my_i = 0.f;
+    }
+    for (int j = lane + 32 * GL_AHEAD; j < wb; j += 32) {
+      const float vr = to_f32<T>(rr[j]), vi = to_f32<T>(ri[j]);
 #pragma unroll
       for (int q = 0; q < GL_SEQS; ++q) {
-        const float r = warp_sum(zr[q]), i = warp_sum(zi[q]);
-        if (lane == q) { my_r = r; my_i = i; }
+        const float v = us[q * ld + j];
+        zr[q] = fmaf(vr, v, zr[q]);
+        zi[q] = fmaf(vi, v, zi[q]);
       }
-      if (lane < ns) {
-        const int s = s0 + lane, t = a.seq_start[s], c = b * wb + d;
-        const float2 st = gl_step(my_r + a.gate_b[(size_t)b * 2 * wb + d], my_i + a.gate_b[(size_t)b * 2 * wb + wb + d], us[lane * ld + d],
-                                  gl_softplus(a.lam[c]));
-        float* own = a.own(s) + c;
-        const float S = fmaf(expf(st.x), *own, st.y);
-        *own = S;
-        const float y = to_f32<T>(((const T*)a.y)[(size_t)t * a.stride + c]);
-        out[(size_t)t * a.out_stride + c] = from_f32<T>(a.scale * glu_activation(y, BN_ACT_GELU_TANH) * S);
-      }
+    }
+    float my_r = 0.f, my_i = 0.f;
+#pragma unroll
+    for (int q = 0; q < GL_SEQS; ++q) {
+      const float r = warp_sum(zr[q]), i = warp_sum(zi[q]);
+      if (lane == q) { my_r = r; my_i = i; }
+    }
+    if (lane < ns) {
+      const float2 st = gl_step(my_r + br, my_i + bi, us[lane * ld + d], sp);
+      S = fmaf(expf(st.x), S, st.y);
+      seq_own[lane][c] = S;
+      out[(size_t)seq_row[lane] * a.out_stride + c] = from_f32<T>(a.scale * glu_activation(y, BN_ACT_GELU_TANH) * S);
     }
   }
 }
@@ -308,23 +378,24 @@ static GatedLinearArgs gl_args(GL_PARAMS) {
   x, y, dtype, n_tokens, stride, width, blocks, taps, conv_w, conv_b, gate_b, lam, state, state_stride, tok_seq, seq_start, seq_pos0, \
       slots, n_seqs, scale, out, out_stride, tail
 
-// u [n_tokens, width] in the compute type.
-extern "C" int bn_gated_linear_conv(GL_PARAMS, void* u, cudaStream_t stream) {
+// u [n_tokens, width] in the compute type; tile_seq / tile_row0: the sequence and first row of every piece of 64 new tokens.
+extern "C" int bn_gated_linear_conv(GL_PARAMS, const int* tile_seq, const int* tile_row0, int n_pieces, void* u, cudaStream_t stream) {
   if (n_tokens <= 0) return BN_OK;
   const GatedLinearArgs a = gl_args(GL_PASS);
-  if (!gl_fits(a) || !u) return BN_ERR_BAD_ARG;
-  const bool vec = width % 4 == 0 && stride % 4 == 0 && !((((uintptr_t)x) | ((uintptr_t)u)) & 7);
-  const int per = 256 * (vec ? 4 : 1);
-  const dim3 grid(n_tokens, (width + per - 1) / per);
-  if (dtype == BN_F32) {
-    if (vec) BN_LAUNCH((gated_linear_conv_kernel<float, 4>), grid, 256, 0, stream, a, (float*)u);
-    else BN_LAUNCH((gated_linear_conv_kernel<float, 1>), grid, 256, 0, stream, a, (float*)u);
-  } else if (dtype == BN_BF16) {
-    if (vec) BN_LAUNCH((gated_linear_conv_kernel<__nv_bfloat16, 4>), grid, 256, 0, stream, a, (__nv_bfloat16*)u);
-    else BN_LAUNCH((gated_linear_conv_kernel<__nv_bfloat16, 1>), grid, 256, 0, stream, a, (__nv_bfloat16*)u);
-  } else {
-    return BN_ERR_BAD_ARG;
-  }
+  if (!gl_fits(a) || !u || !tile_seq || !tile_row0 || n_pieces <= 0) return BN_ERR_BAD_ARG;
+#define GL_CONV(TT, VV)                                                                                                              \
+  do {                                                                                                                               \
+    const int per = GL_CONV_COLS * VV, cols = (width + per - 1) / per;                                                               \
+    if (cols > 65535) return BN_ERR_BAD_ARG;                                                                                         \
+    BN_LAUNCH((gated_linear_conv_kernel<TT, VV>), dim3(n_pieces, cols), GL_CONV_COLS * GL_PIECE / GL_CONV_ROWS, 0, stream, a, tile_seq, \
+              tile_row0, (TT*)u);                                                                                                    \
+  } while (0)
+  const int v = dtype == BN_F32 ? 4 : 8;  // whole 16-byte pieces, also of the ring's rows
+  const bool vec = width % v == 0 && stride % v == 0 && state_stride % 4 == 0 && !(((uintptr_t)x | (uintptr_t)u | (uintptr_t)state) & 15);
+  if (dtype == BN_F32) { if (vec) GL_CONV(float, 4); else GL_CONV(float, 1); }
+  else if (dtype == BN_BF16) { if (vec) GL_CONV(__nv_bfloat16, 8); else GL_CONV(__nv_bfloat16, 1); }
+  else return BN_ERR_BAD_ARG;
+#undef GL_CONV
   return BN_OK;
 }
 

@@ -420,6 +420,36 @@ __global__ void moe_offsets_kernel(const int* __restrict__ counts, int n_experts
   }
 }
 
+// The same, packed, from the items themselves (counted in shared memory); one block of 1,024 threads.
+__global__ void __launch_bounds__(1024) moe_count_offsets_kernel(const int* __restrict__ ids, int n_items, int n_experts,
+                                                                 int* __restrict__ offsets, int* __restrict__ cursor) {
+  pdl_launch_dependents();
+  __shared__ int counts[MOE_MAX_EXPERTS], warp_total[32];
+  const int e = threadIdx.x, lane = e & 31, warp = e >> 5;
+  counts[e] = 0;
+  __syncthreads();
+  pdl_wait();
+  for (int i = e; i < n_items; i += 1024) {
+    const int id = ids[i];
+    if (id < n_experts) atomicAdd(&counts[id], 1);
+  }
+  __syncthreads();
+  const int mine = counts[e];
+  int upto = mine;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int up = __shfl_up_sync(0xffffffffu, upto, o);
+    if (lane >= o) upto += up;
+  }
+  if (lane == 31) warp_total[warp] = upto;
+  __syncthreads();
+  for (int w = 0; w < warp; ++w) upto += warp_total[w];
+  if (e < n_experts) {
+    offsets[e] = cursor[e] = upto - mine;
+    if (e == n_experts - 1) offsets[n_experts] = upto;
+  }
+}
+
 // place[i] = row of item i in the sorted order, and x_sorted[place[i]] = weight * h[token of i] (or h itself).
 // Rows of one expert come in any order; every row is computed alone, so the order changes no result.
 template <typename T>
@@ -518,17 +548,20 @@ extern "C" int bn_moe_count(const int* ids, int n_items, int n_experts, int* cou
   return BN_OK;
 }
 
-// counts as bn_moe_count left them; offsets: [n_experts + 1]; cursor: [n_experts]; place: [n_items];
+// counts as bn_moe_count left them (or null: counted here; cap == 0 then); offsets: [n_experts + 1]; cursor: [n_experts]; place: [n_items];
 // x_sorted: [n_items, width] (cap == 0) or [n_experts * cap, width] (cap >= the largest count)
 extern "C" int bn_moe_scatter(const void* h, int dtype, int n_tokens, int width, const int* ids, const float* weights,
                               int scale_input, int top, int n_experts, int cap, const int* counts, int* offsets,
                               int* cursor, int* place, void* x_sorted, cudaStream_t stream) {
   if (n_tokens <= 0) return BN_OK;
-  if (!h || !ids || !weights || !counts || !offsets || !cursor || !place || !x_sorted || width <= 0 || top <= 0 ||
+  if (!h || !ids || !weights || (!counts && (cap > 0 || n_experts > MOE_MAX_EXPERTS)) || !offsets || !cursor || !place || !x_sorted || width <= 0 || top <= 0 ||
       n_experts <= 0 || cap < 0)
     return BN_ERR_BAD_ARG;
   int n_items = n_tokens * top;
-  BN_LAUNCH(moe_offsets_kernel, 1, 32, 0, stream, counts, n_experts, cap, offsets, cursor);
+  if (counts)
+    BN_LAUNCH(moe_offsets_kernel, 1, 32, 0, stream, counts, n_experts, cap, offsets, cursor);
+  else
+    BN_LAUNCH(moe_count_offsets_kernel, 1, 1024, 0, stream, ids, n_items, n_experts, offsets, cursor);
   if (dtype == BN_F32)
     BN_LAUNCH(moe_scatter_kernel<float>, n_items, 128, 0, stream, (const float*)h, width, ids, weights, scale_input, top, n_experts,
               cursor, place, (float*)x_sorted);

@@ -1876,7 +1876,7 @@ def gated_linear(x: torch.Tensor, y: torch.Tensor, conv_w: torch.Tensor, conv_b:
     _need(tile_seq, "tile_seq", torch.int32, 1)
     _need(tile_row0, "tile_row0", torch.int32, 1)
     u = torch.empty((T, width), dtype=x.dtype, device=x.device)
-    _check(_fn("gated_linear", "bn_gated_linear_conv")(*args, _ptr(u), _stream()), "gated_linear_conv")
+    _check(_fn("gated_linear", "bn_gated_linear_conv")(*args, _ptr(tile_seq), _ptr(tile_row0), int(tile_seq.shape[0]), _ptr(u), _stream()), "gated_linear_conv")
     up = u.view(T, parts, part).transpose(0, 1)
     if x.dtype == torch.float32:
         if torch.backends.cuda.matmul.allow_tf32:
@@ -2184,20 +2184,24 @@ def moe_count(ids: torch.Tensor, n_experts: int) -> torch.Tensor:
     return counts
 
 
-def moe_sort(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, counts: torch.Tensor, scale_input: bool,
-             cap: int = 0):
+def moe_sort(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, counts: Optional[torch.Tensor], scale_input: bool,
+             cap: int = 0, n_experts: int = 0):
     """Sort the (token, expert) items by expert: ``(x_sorted, place int32 [T * top], offsets int32 [experts + 1])``.
     Item i went to row ``place[i]`` of ``x_sorted``, which holds its token's row of h (times its weight with
     ``scale_input``).  ``cap`` = 0: the experts' rows are packed, expert e's are rows ``offsets[e] ..
     offsets[e + 1]`` of ``[T * top, width]``.  ``cap`` > 0 (at least the largest of ``counts``): expert e's rows
     begin at ``e * cap`` of ``[experts * cap, width]``; rows that no item took hold nothing.  Items of identity experts (ids from
-    the number of ``counts`` on) get the place -1."""
+    the number of experts on) get the place -1.  ``counts`` None: the items of ``n_experts`` experts are counted on the way (packed)."""
     _need(h, "h", dims=2)
     _need(ids, "ids", torch.int32, 2)
     _need(weights, "weights", torch.float32, 2)
-    _need(counts, "counts", torch.int32, 1)
+    if counts is not None:
+        _need(counts, "counts", torch.int32, 1)
+        n_experts = counts.shape[0]
+    elif cap or not 0 < n_experts <= 1024:
+        raise KernelError(f"moe_sort: {n_experts} experts, blocks of {cap} rows need counts")
     T, width = h.shape
-    top, n_experts = ids.shape[1], counts.shape[0]
+    top = ids.shape[1]
     book = torch.empty(2 * n_experts + 1, dtype=torch.int32, device=h.device)
     offsets, cursor = book[:n_experts + 1], book[n_experts + 1:]
     place = torch.empty(T * top, dtype=torch.int32, device=h.device)

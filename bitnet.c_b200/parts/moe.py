@@ -149,14 +149,14 @@ class Moe(FeedForward):
         if self.few_fits and (ctx.decode or T * s.top <= self.FEW_ITEMS):
             return ops.moe_experts_few(h, ids, weights, self.w_gate_up, self.w_down, s.expert_limit, s.slope,
                                        s.weight_on_input, add=shared, act=self.act, add_scale=shared_scale)
-        counts = ops.moe_count(ids, s.n_experts)
         rest = dict(add_scale=shared_scale, h=h if s.identity else None)
         if self.USE_GROUPED and h.dtype == torch.bfloat16 and ops.grouped_fits(self.w_gate_up) and ops.grouped_fits(self.w_down):
-            x_sorted, place, offsets = ops.moe_sort(h, ids, weights, counts, s.weight_on_input)
+            x_sorted, place, offsets = ops.moe_sort(h, ids, weights, None, s.weight_on_input, n_experts=s.n_experts)
             up = ops.grouped_product(x_sorted, self.w_gate_up, offsets, act=0 if self.gated else ops.ACT_RELU2)
             act = self._activate(up, s.expert_limit) if self.gated else up
             y_sorted = ops.grouped_product(act, self.w_down, offsets)
             return ops.moe_gather(y_sorted, place, weights, not s.weight_on_input, add=shared, **rest)
+        counts = ops.moe_count(ids, s.n_experts)
         host_tokens = getattr(ctx, "host_tokens", None)
         if self.by_table and host_tokens is not None:
             # chosen by token id: the counts follow from the step's ids on the host, nobody waits for the device
