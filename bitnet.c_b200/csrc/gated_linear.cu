@@ -241,37 +241,44 @@ __global__ void __launch_bounds__(GL_THREADS) gated_linear_carry_kernel(const Ga
 
 // ---- one token per sequence --------------------------------------------------------------------------------
 #define GL_SEQS 8        // sequences a block takes at a time
-#define GL_CHANNELS 8    // channels per block: one per warp
+#define GL_CHANNELS 8    // channels a block takes at a time: one per warp
+#define GL_TOKEN_BLOCKS 300  // about two blocks per SM: every block convolves its whole part
 #define GL_AHEAD 8       // numbers of each row of R and I that a lane asks for before the step's inputs are there
 
-// A block per (part, 8 of its channels): the convolution of the whole part for eight sequences at a time into shared memory,
-// then a warp per channel takes its rows of R and I (w_gates [blocks][2 wb][wb], r's rows first) against all of them, and
+// Blocks share out a part's channels eight at a time: the convolution of the whole part for eight sequences at a time into
+// shared memory, then a warp per channel takes its rows of R and I (w_gates [blocks][2 wb][wb], r's rows first) against all of them, and
 // lane s does sequence s's step.
-template <typename T>
+// TAPS: the most taps the instantiation takes (their loads are all in flight together).
+template <typename T, int TAPS>
 __global__ void __launch_bounds__(256) gated_linear_token_kernel(const GatedLinearArgs a, const T* __restrict__ w_gates) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float us[];  // [GL_SEQS][wb padded to 4]
   __shared__ int seq_pos[GL_SEQS], seq_row[GL_SEQS];
   __shared__ float* seq_own[GL_SEQS];
   const int wb = a.width / a.blocks, ld = (wb + 3) / 4 * 4;
-  const int b = blockIdx.x, d0 = blockIdx.y * GL_CHANNELS;
+  const int b = blockIdx.x, first = blockIdx.y * GL_CHANNELS, step = gridDim.y * GL_CHANNELS;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const T* x = (const T*)a.x;
   T* out = (T*)a.out;
-  // the warp's channel and what of it are weights
-  const int d = d0 + warp, c = b * wb + d;
-  const bool live = d < wb;
-  const T* rr = w_gates + ((size_t)b * 2 * wb + (live ? d : 0)) * wb;
-  const T* ri = rr + (size_t)wb * wb;
-  float wr[GL_AHEAD], wi[GL_AHEAD];
+  // what of the warp's first channel are weights
+  float wr[GL_AHEAD], wi[GL_AHEAD], br = 0.f, bi = 0.f, sp = 0.f;
+  auto weights_of = [&](int d) {
+    const bool live = d < wb;
+    const T* rr = w_gates + ((size_t)b * 2 * wb + (live ? d : 0)) * wb;
+    const T* ri = rr + (size_t)wb * wb;
 #pragma unroll
-  for (int k = 0; k < GL_AHEAD; ++k) {
-    const int jj = lane + 32 * k;
-    wr[k] = jj < wb ? to_f32<T>(rr[jj]) : 0.f;
-    wi[k] = jj < wb ? to_f32<T>(ri[jj]) : 0.f;
-  }
-  const float br = live ? a.gate_b[(size_t)b * 2 * wb + d] : 0.f, bi = live ? a.gate_b[(size_t)b * 2 * wb + wb + d] : 0.f;
-  const float sp = live ? gl_softplus(a.lam[c]) : 0.f;
+    for (int k = 0; k < GL_AHEAD; ++k) {
+      const int jj = lane + 32 * k;
+      wr[k] = jj < wb ? to_f32<T>(rr[jj]) : 0.f;
+      wi[k] = jj < wb ? to_f32<T>(ri[jj]) : 0.f;
+    }
+    if (live) {
+      br = a.gate_b[(size_t)b * 2 * wb + d];
+      bi = a.gate_b[(size_t)b * 2 * wb + wb + d];
+      sp = gl_softplus(a.lam[b * wb + d]);
+    }
+  };
+  weights_of(first + warp);
   pdl_wait();
   if (a.tail > 0 && blockIdx.x == 0 && blockIdx.y == 0)
     for (int i = threadIdx.x; i < a.n_seqs * a.tail; i += blockDim.x) {
@@ -288,13 +295,17 @@ __global__ void __launch_bounds__(256) gated_linear_token_kernel(const GatedLine
       seq_own[threadIdx.x] = a.own(s);
     }
     __syncthreads();
-    // lane s: sequence s's state and output gate, on their way during the convolution
-    float S = 0.f, y = 0.f;
-    if (live && lane < ns) {
-      S = seq_own[lane][c];
-      y = to_f32<T>(((const T*)a.y)[(size_t)seq_row[lane] * a.stride + c]);
-    }
-#pragma unroll 4
+    // lane s: sequence s's state and output gate, on their way during the convolution (of the next channel: during this one's
+    // sums)
+    float S_next = 0.f, y_next = 0.f;
+    auto inputs_of = [&](int d) {
+      if (d < wb && lane < ns) {
+        S_next = seq_own[lane][b * wb + d];
+        y_next = to_f32<T>(((const T*)a.y)[(size_t)seq_row[lane] * a.stride + b * wb + d]);
+      }
+    };
+    inputs_of(first + warp);
+#pragma unroll (TAPS <= 4 ? 4 : 1)
     for (int i = threadIdx.x; i < GL_SEQS * ld; i += blockDim.x) {
       const int q = i / ld, dd = i - q * ld;
       float acc = 0.f;
@@ -304,52 +315,70 @@ __global__ void __launch_bounds__(256) gated_linear_token_kernel(const GatedLine
         const float now = to_f32<T>(x[(size_t)seq_row[q] * a.stride + cc]);
         acc = fmaf(a.conv_w[(size_t)(a.taps - 1) * a.width + cc], now, a.conv_b[cc]);
         int row = pos % a.taps;  // of this token; the token `back` before it lies `back` rows in front
-        if (a.taps > 1 && dd >= d0 && dd < d0 + GL_CHANNELS) ring[(size_t)row * a.width + cc] = now;
-        for (int back = 1; back < a.taps && back <= pos; ++back) {
+        if (a.taps > 1 && dd / GL_CHANNELS % gridDim.y == blockIdx.y) ring[(size_t)row * a.width + cc] = now;
+        float before[TAPS], w[TAPS];
+#pragma unroll
+        for (int back = 1; back < TAPS; ++back) {
           row = row == 0 ? a.taps - 1 : row - 1;
-          acc = fmaf(a.conv_w[(size_t)(a.taps - 1 - back) * a.width + cc], ring[(size_t)row * a.width + cc], acc);
+          const bool there = back < a.taps && back <= pos;
+          before[back] = there ? ring[(size_t)row * a.width + cc] : 0.f;
+          w[back] = there ? a.conv_w[(size_t)(a.taps - 1 - back) * a.width + cc] : 0.f;
         }
+#pragma unroll
+        for (int back = 1; back < TAPS; ++back) acc = fmaf(w[back], before[back], acc);
         acc = to_f32<T>(from_f32<T>(acc));
       }
       us[i] = acc;
     }
     __syncthreads();
-    if (!live) continue;
-    float zr[GL_SEQS], zi[GL_SEQS];
+    for (int d = first + warp; d < wb; d += step) {
+      const int c = b * wb + d;
+      const T* rr = w_gates + ((size_t)b * 2 * wb + d) * wb;
+      const T* ri = rr + (size_t)wb * wb;
+      const float S_old = S_next, y = y_next;
+      float zr[GL_SEQS], zi[GL_SEQS];
 #pragma unroll
-    for (int q = 0; q < GL_SEQS; ++q) zr[q] = zi[q] = 0.f;
+      for (int q = 0; q < GL_SEQS; ++q) zr[q] = zi[q] = 0.f;
 #pragma unroll
-    for (int k = 0; k < GL_AHEAD; ++k) {
-      const int j = lane + 32 * k;
-      if (j < wb) {
+      for (int k = 0; k < GL_AHEAD; ++k) {
+        const int j = lane + 32 * k;
+        if (j < wb) {
+#pragma unroll
+          for (int q = 0; q < GL_SEQS; ++q) {
+            const float v = us[q * ld + j];
+            zr[q] = fmaf(wr[k], v, zr[q]);
+            zi[q] = fmaf(wi[k], v, zi[q]);
+          }
+        }
+      }
+      for (int j = lane + 32 * GL_AHEAD; j < wb; j += 32) {
+        const float vr = to_f32<T>(rr[j]), vi = to_f32<T>(ri[j]);
 #pragma unroll
         for (int q = 0; q < GL_SEQS; ++q) {
           const float v = us[q * ld + j];
-          zr[q] = fmaf(wr[k], v, zr[q]);
-          zi[q] = fmaf(wi[k], v, zi[q]);
+          zr[q] = fmaf(vr, v, zr[q]);
+          zi[q] = fmaf(vi, v, zi[q]);
         }
       }
-    }
-    for (int j = lane + 32 * GL_AHEAD; j < wb; j += 32) {
-      const float vr = to_f32<T>(rr[j]), vi = to_f32<T>(ri[j]);
+      const float my_br = br, my_bi = bi, my_sp = sp;
+      // this channel's weights have been used: the next one's, or the first one's for the next sequences
+      const int next = d + step < wb ? d + step : first + warp;
+      if (next != d) {
+        weights_of(next);
+        if (next > d) inputs_of(next);
+      }
+      float my_r = 0.f, my_i = 0.f;
 #pragma unroll
       for (int q = 0; q < GL_SEQS; ++q) {
-        const float v = us[q * ld + j];
-        zr[q] = fmaf(vr, v, zr[q]);
-        zi[q] = fmaf(vi, v, zi[q]);
+        const float r = warp_sum(zr[q]), i = warp_sum(zi[q]);
+        if (lane == q) { my_r = r; my_i = i; }
       }
-    }
-    float my_r = 0.f, my_i = 0.f;
-#pragma unroll
-    for (int q = 0; q < GL_SEQS; ++q) {
-      const float r = warp_sum(zr[q]), i = warp_sum(zi[q]);
-      if (lane == q) { my_r = r; my_i = i; }
-    }
-    if (lane < ns) {
-      const float2 st = gl_step(my_r + br, my_i + bi, us[lane * ld + d], sp);
-      S = fmaf(expf(st.x), S, st.y);
-      seq_own[lane][c] = S;
-      out[(size_t)seq_row[lane] * a.out_stride + c] = from_f32<T>(a.scale * glu_activation(y, BN_ACT_GELU_TANH) * S);
+      if (lane < ns) {
+        const float2 st = gl_step(my_r + my_br, my_i + my_bi, us[lane * ld + d], my_sp);
+        const float S = fmaf(expf(st.x), S_old, st.y);
+        seq_own[lane][c] = S;
+        out[(size_t)seq_row[lane] * a.out_stride + c] = from_f32<T>(a.scale * glu_activation(y, BN_ACT_GELU_TANH) * S);
+      }
     }
   }
 }
@@ -437,20 +466,21 @@ extern "C" int bn_gated_linear_token(GL_PARAMS, const void* w_gates, cudaStream_
   if (!gl_fits(a) || !w_gates || !out || out_stride < width + tail || n_tokens != n_seqs) return BN_ERR_BAD_ARG;
   const int wb = width / blocks;
   const size_t smem = (size_t)GL_SEQS * ((wb + 3) / 4 * 4) * sizeof(float);
-  const dim3 grid(blocks, (wb + GL_CHANNELS - 1) / GL_CHANNELS);
-  if (smem > 200 * 1024 || grid.y > 65535) return BN_ERR_BAD_ARG;
-#define GL_TOKEN(TT)                                                                                                                   \
+  const int groups = (wb + GL_CHANNELS - 1) / GL_CHANNELS, want = (GL_TOKEN_BLOCKS + blocks - 1) / blocks;
+  const dim3 grid(blocks, groups < want ? groups : want);
+  if (smem > 200 * 1024) return BN_ERR_BAD_ARG;
+#define GL_TOKEN(TT, NN)                                                                                                               \
   do {                                                                                                                                 \
     static size_t granted = 0;                                                                                                         \
     if (smem > 48 * 1024 && smem > granted) {                                                                                          \
-      cudaError_t e = cudaFuncSetAttribute(gated_linear_token_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
+      cudaError_t e = cudaFuncSetAttribute(gated_linear_token_kernel<TT, NN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
       if (e != cudaSuccess) return BN_ERR_LAUNCH + (int)e;                                                                             \
       granted = smem;                                                                                                                  \
     }                                                                                                                                  \
-    BN_LAUNCH(gated_linear_token_kernel<TT>, grid, 256, smem, stream, a, (const TT*)w_gates);                                          \
+    BN_LAUNCH((gated_linear_token_kernel<TT, NN>), grid, 256, smem, stream, a, (const TT*)w_gates);                                    \
   } while (0)
-  if (dtype == BN_F32) GL_TOKEN(float);
-  else if (dtype == BN_BF16) GL_TOKEN(__nv_bfloat16);
+  if (dtype == BN_F32) { if (taps <= 4) GL_TOKEN(float, 4); else GL_TOKEN(float, GL_MAX_TAPS); }
+  else if (dtype == BN_BF16) { if (taps <= 4) GL_TOKEN(__nv_bfloat16, 4); else GL_TOKEN(__nv_bfloat16, GL_MAX_TAPS); }
   else return BN_ERR_BAD_ARG;
 #undef GL_TOKEN
   return BN_OK;

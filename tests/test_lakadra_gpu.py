@@ -64,7 +64,7 @@ def _step_arrays(new, at, slots):
 
 
 # ---- kernels alone -----------------------------------------------------------------------------------
-@pytest.mark.parametrize("blocks,part,taps", [(1, 8, 4), (3, 5, 2), (4, 16, 1), (2, 130, 16), (16, 128, 4), (1, 300, 3)])
+@pytest.mark.parametrize("blocks,part,taps", [(1, 8, 4), (3, 5, 2), (4, 16, 1), (2, 130, 16), (16, 128, 4), (1, 300, 3), (40, 72, 2)])
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_the_gated_recurrence_however_the_tokens_are_cut(cuda_device, blocks, part, taps, dtype):
     """Unequal sequences in scattered slots, in runs that end before, on and behind the edge of a piece, in pairs, and one
@@ -108,6 +108,32 @@ def test_the_gated_recurrence_however_the_tokens_are_cut(cuda_device, blocks, pa
             for s in live:
                 at[s] += new[s]
         assert at == LENGTHS and bool((state[1] == 7.0).all()) and bool((state[2] == 0.0).all())
+
+
+@pytest.mark.parametrize("blocks,part", [(3, 24), (60, 48), (2, 288)])
+def test_the_gated_recurrence_of_many_sequences_at_once(cuda_device, blocks, part):
+    """Nineteen sequences of unequal lengths, then one token each, three times."""
+    from bitnet_c_b200.csrc import ops
+    n, taps, S = blocks * part, 4, 19
+    rng = np.random.default_rng(n)
+    conv, conv_b, lam = f32(0.6 * rng.standard_normal((n, taps))), f32(0.3 * rng.standard_normal(n)), f32(rng.uniform(-7, 0, n))
+    ra, ri = (bf(1.5 * rng.standard_normal((blocks, part, part)) / np.sqrt(part)) for _ in range(2))
+    rb, ib = (f32(rng.standard_normal((blocks, part))) for _ in range(2))
+    lens = [1 + 5 * (s % 4) for s in range(S)]
+    xs, ys = ([bf(rng.standard_normal((m + 3, n))) for m in lens] for _ in range(2))
+    want = [pl.gelu_tanh(y) * pl.gated_linear_states(pl.causal_convolution(x, conv, conv_b), ra, rb, ri, ib, lam) for x, y in zip(xs, ys)]
+    scale = max(np.abs(a).max() for a in want)
+    state = torch.zeros((S, ops.gated_linear_floats(n, taps)), dtype=torch.float32, device="cuda")
+    at, slots = [0] * S, rng.permutation(S).tolist()
+    for new in (lens, [1] * S, [1] * S, [1] * S):
+        live, step = _step_arrays(new, at, slots)
+        cat = lambda zs: dev(np.concatenate([zs[s][at[s]:at[s] + new[s]] for s in live]))
+        out = torch.empty((sum(new), n), device="cuda")
+        ops.gated_linear(cat(xs), cat(ys), dev(conv.T.copy()), dev(conv_b), dev(np.concatenate([ra, ri], axis=1)), dev(np.concatenate([rb, ib], axis=1)),
+                         dev(lam), state, out=out, **step)
+        ref = np.concatenate([want[s][at[s]:at[s] + new[s]] for s in live])
+        assert np.abs(out.cpu().numpy() - ref).max() < 1e-4 * max(1.0, scale)
+        at = [a + c for a, c in zip(at, new)]
 
 
 def _lightning_inputs(rng, H, d, dv):
